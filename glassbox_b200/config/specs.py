@@ -163,7 +163,10 @@ class SinkAttentionSpec:
     "none"; "source": this layer's values are kept for the step, for later layers to mix in; "mixed": the values become
     (1 - lambda) v + lambda v_source (lambda a learned scalar, v_source the source layer's values of the same token) before
     they are cached. ``output_gate``: head h's output is multiplied by sigmoid(w_gate_h . x), one number per head and
-    token, from the same input as the projections. ``window`` as in ``GqaAttentionSpec``."""
+    token, from the same input as the projections; with ``gate_per`` "channel" the gate has a logit per output channel
+    instead (the concatenated heads times sigmoid(W_g x)). ``qk_norm_gain`` False: the query and key norms have no gains.
+    ``q_temp`` = (coef, every): the query at position p is multiplied by 1 + coef * ln(floor((p + 1) / every) + 1).
+    ``window`` as in ``GqaAttentionSpec``."""
     num_heads: int
     num_kv_heads: int
     head_dim: int
@@ -175,6 +178,9 @@ class SinkAttentionSpec:
     sink: bool = True
     value_mix: str = "none"
     output_gate: bool = True
+    gate_per: str = "head"
+    qk_norm_gain: bool = True
+    q_temp: Optional[Tuple[float, float]] = None
     kind: str = "sink_attention"
 
 
@@ -232,12 +238,32 @@ class HeadDeltaSpec:
 @dataclass(frozen=True)
 class ParallelMixerSpec:
     """Two mixers side by side that read the same input: the output is ``left_scale`` * left + ``right_scale`` * right.
-    Either may keep keys in pages, a state per request, or both."""
+    Either may keep keys in pages, a state per request, or both. ``output_norm``: an RMS norm spec; each side's output is
+    normed over the model width, with a gain of its own, before the sum. ``shared_projection``: the two sides' stacked input
+    matrices are one matrix (left's rows, then right's) and one product serves both."""
     left: Any
     right: Any
     left_scale: float = 1.0
     right_scale: float = 1.0
+    output_norm: Any = None
+    shared_projection: bool = False
     kind: str = "parallel"
+
+
+@dataclass(frozen=True)
+class StateSpaceSpec:
+    """A selective state-space mixer with one scalar decay per head and token: a float32 state S [state_dim, value_dim] per
+    head, S <- exp(-exp(A_log_h) dt) S + dt B x^T with dt = softplus(dt_logit + dt_bias), read as S^T C + D_h x. x, B and C
+    come through one causal convolution of ``conv_taps`` taps with bias and SiLU; heads share B and C in ``num_groups``
+    groups. The read-out times silu(z) is RMS-normed in ``norm_groups`` equal parts (``norm_eps``, a gain per channel)."""
+    num_heads: int
+    num_groups: int
+    state_dim: int
+    value_dim: int
+    conv_taps: int
+    norm_groups: int
+    norm_eps: float
+    kind: str = "state_space"
 
 
 @dataclass(frozen=True)
@@ -267,11 +293,17 @@ class RoutedExpertsSpec:
     shared_size: int = 0
     shared_gate: bool = True
     #: "sigmoid": as above. "softmax_chosen": the choice is made by the logits themselves (plus ``router_bias``, a stored
-    #: number per expert that is part of the logit) and the weights are the softmax over the chosen logits alone
+    #: number per expert that is part of the logit) and the weights are the softmax over the chosen logits alone.
+    #: "softmax": the scores are the softmax over all experts
     scoring: str = "sigmoid"
     router_bias: bool = False
+    #: what a run of neighbours scores: the sum of its two best choice scores ("top2") or its best ("best")
+    group_score: str = "top2"
+    #: the chosen experts' scores are divided by (their sum + this); None: they weigh as they are
+    renormalise: Optional[float] = None
     #: "relu2": W_down relu(W_up h)^2. "clamped_glu": the expert has a gate and an up matrix and computes
-    #: W_down (g * sigmoid(``glu_slope`` g) * (u + 1)) with g = min(W_gate h, ``limit``), u = clamp(W_up h, -limit, limit)
+    #: W_down (g * sigmoid(``glu_slope`` g) * (u + 1)) with g = min(W_gate h, ``limit``), u = clamp(W_up h, -limit, limit).
+    #: "swiglu": W_down (silu(W_gate h) * W_up h)
     activation: str = "relu2"
     limit: float = 0.0
     glu_slope: float = 1.702
@@ -330,8 +362,9 @@ class ScaledEmbeddingSpec:
 @dataclass(frozen=True)
 class PositionalEmbeddingSpec:
     """Token embedding plus a learned vector per position: the residual row of a token at position p is its row of the
-    table plus row p of a second table of ``max_position`` rows (neither scaled), summed in float32."""
+    table times ``scale`` plus row p of a second table of ``max_position`` rows (not scaled), in float32."""
     max_position: int
+    scale: float = 1.0
     kind: str = "positional_embedding"
 
 
@@ -367,6 +400,9 @@ class LayerSpec:
     ffn_post_norm: Any = None
     #: "branch_norm" norms each branch on the way out only: x += post(mixer(x)), x += post(ffn(x)); the branches read the
     #: residual itself (rounded to the activation dtype); ``mixer_norm`` and ``ffn_norm`` are None, ``ffn`` may be None
+    #: "post_norm" norms after the sum: x <- mixer_post_norm(alpha x + mixer(x)), x <- ffn_post_norm(alpha x + ffn(x)) with
+    #: alpha = ``residual_scale``; the branches read the residual itself, ``mixer_norm`` and ``ffn_norm`` are None
+    residual_scale: float = 1.0
     #: "hyper_connections": the residual is ``streams`` rows per token; each branch reads a learned mix of them through
     #: its norm and its output comes back into all of them through a learned matrix (``ModelConfig.residual_streams`` says
     #: the same number for the whole model); ``ffn`` may be None

@@ -31,12 +31,14 @@ struct DecodeAttnArgs {
     int late_release;   // let the next kernel in the stream go only after this one's own wait (else at its start)
     // Read only by the SINK instantiations (each may be nullptr): the score of a key `dist` tokens back loses
     // r1[head] * ln(1 + r2[head] * dist); the softmax's denominator also holds exp(sink[head]), which has no key and
-    // no value; the head's output is multiplied by sigmoid(gate[row * ld_gate + head]) (float32 logits).
+    // no value; the head's output is multiplied by sigmoid(gate[row * ld_gate + head]) (float32 logits), or, with
+    // gate_channels, channel c of it by sigmoid(gate[row * ld_gate + head * HD + c]).
     const float* r1;
     const float* r2;
     const float* sink;
     const float* gate;
     long long ld_gate;
+    int gate_channels;
 };
 
 constexpr float MMA_NEG_BIG = -1.0e30f;
@@ -158,8 +160,11 @@ __device__ __forceinline__ void attention_decode_mma_body(const DecodeAttnArgs& 
         }
     }
     auto sink_logit = [&](int head) { return (SINK && a.sink != nullptr) ? a.sink[head] : MMA_NEG_BIG; };
+    auto channel_gate = [&](int head, int c) {
+        return (SINK && a.gate != nullptr && a.gate_channels) ? 1.0f / (1.0f + __expf(-a.gate[(size_t)row * a.ld_gate + head * HD + c])) : 1.0f;
+    };
     auto gate_factor = [&](int head) {
-        return (SINK && a.gate != nullptr) ? 1.0f / (1.0f + __expf(-a.gate[(size_t)row * a.ld_gate + head])) : 1.0f;
+        return (SINK && a.gate != nullptr && !a.gate_channels) ? 1.0f / (1.0f + __expf(-a.gate[(size_t)row * a.ld_gate + head])) : 1.0f;
     };
 
     // This kernel's own prologue (positions, block table: step metadata that no kernel writes) runs before it waits
@@ -424,7 +429,7 @@ __device__ __forceinline__ void attention_decode_mma_body(const DecodeAttnArgs& 
             float v = 0.f;
 #pragma unroll 8
             for (int sidx = 0; sidx < S4; ++sidx) v = fmaf(pa[(size_t)sidx * (HD + 2)], w[sidx], v);
-            orow[(head0 + hi) * HD + d] = __float2bfloat16_rn(v);
+            orow[(head0 + hi) * HD + d] = __float2bfloat16_rn(SINK ? v * channel_gate(head0 + hi, d) : v);
         }
         return;
     }
@@ -467,6 +472,7 @@ __device__ __forceinline__ void attention_decode_mma_body(const DecodeAttnArgs& 
         constexpr int MAXP = 64;
         const int hi_o = tid / HD, d_o = tid % HD;
         float pv[MAXP];
+        const float gch = tid < G * HD ? channel_gate(head0 + hi_o, d_o) : 1.0f;
         if (tid < G * HD) {
             const float* pa = part_acc + ((size_t)row * nh + head0 + hi_o) * S4 * HD + d_o;
 #pragma unroll
@@ -491,7 +497,7 @@ __device__ __forceinline__ void attention_decode_mma_body(const DecodeAttnArgs& 
 #pragma unroll
             for (int sidx = 0; sidx < MAXP; ++sidx)
                 if (sidx < S4) v = fmaf(pv[sidx], w[sidx], v);
-            orow[(head0 + hi_o) * HD + d_o] = __float2bfloat16_rn(v);
+            orow[(head0 + hi_o) * HD + d_o] = __float2bfloat16_rn(SINK ? v * gch : v);
         }
         return;
     }
@@ -523,7 +529,7 @@ __device__ __forceinline__ void attention_decode_mma_body(const DecodeAttnArgs& 
             float v = 0.f;
 #pragma unroll 8
             for (int sidx = 0; sidx < S4; ++sidx) v = fmaf(__ldcg(pa + (size_t)sidx * HD), w[sidx], v);
-            orow[(head0 + h0 + hi) * HD + d] = __float2bfloat16_rn(v);
+            orow[(head0 + h0 + hi) * HD + d] = __float2bfloat16_rn(SINK ? v * channel_gate(head0 + h0 + hi, d) : v);
         }
         sync.group_barrier();
     }

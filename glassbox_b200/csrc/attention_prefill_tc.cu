@@ -111,13 +111,15 @@ __device__ __forceinline__ float at_exp2(float x) {
 
 // What the SINK instantiation reads beside the common arguments (each may be nullptr): the score of a key `dist` tokens
 // back loses r1[head] * ln(1 + r2[head] * dist); the softmax's denominator also holds exp(sink[head]), which has no key and
-// no value; the head's output is multiplied by sigmoid(gate[row * ld_gate + head]) (float32 logits).
+// no value; the head's output is multiplied by sigmoid(gate[row * ld_gate + head]) (float32 logits; with gate_channels a gate
+// per channel, gate[row * ld_gate + head * HD + c]).
 struct AtSinkTerms {
     const float* r1;
     const float* r2;
     const float* sink;
     const float* gate;
     long long ld_gate;
+    int gate_channels;
 };
 
 template <int HD, bool SINK = false>
@@ -448,7 +450,7 @@ __global__ void __launch_bounds__(AT_WARPS * 32) attention_prefill_tc_kernel(
             if constexpr (SINK) l += at_exp2(sink2 - m);
             float inv = l > 0.f ? 1.0f / l : 0.f;
             if constexpr (SINK) {
-                if (terms.gate != nullptr && q_lo + r < nrows)
+                if (terms.gate != nullptr && !terms.gate_channels && q_lo + r < nrows)
                     inv *= 1.0f / (1.0f + __expf(-terms.gate[(size_t)(row0 + q_lo + r) * terms.ld_gate + head]));
             }
             constexpr int OC = HD / 2;                 // this thread's channels: g * OC ..
@@ -468,6 +470,22 @@ __global__ void __launch_bounds__(AT_WARPS * 32) attention_prefill_tc_kernel(
             }
             if (q_lo + r < nrows) {
                 __nv_bfloat16* dst = out + (size_t)(row0 + q_lo + r) * out_stride + (size_t)head * HD + g * OC;
+                if constexpr (SINK) {
+                    if (terms.gate != nullptr && terms.gate_channels) {
+                        const float* gch = terms.gate + (size_t)(row0 + q_lo + r) * terms.ld_gate + (size_t)head * HD + g * OC;
+                        const bool vec = (((uintptr_t)gch) & 15) == 0;
+#pragma unroll
+                        for (int k = 0; k < OC; k += 4) {
+                            float4 z;
+                            if (vec) z = *reinterpret_cast<const float4*>(gch + k);
+                            else z = make_float4(gch[k], gch[k + 1], gch[k + 2], gch[k + 3]);
+                            o[k] = __fdividef(o[k], 1.0f + __expf(-z.x));
+                            o[k + 1] = __fdividef(o[k + 1], 1.0f + __expf(-z.y));
+                            o[k + 2] = __fdividef(o[k + 2], 1.0f + __expf(-z.z));
+                            o[k + 3] = __fdividef(o[k + 3], 1.0f + __expf(-z.w));
+                        }
+                    }
+                }
 #pragma unroll
                 for (int k = 0; k < OC; k += 8) {
                     uint4 w;
@@ -561,16 +579,17 @@ GB_EXPORT int gb_attention_prefill_tc(const void* q, long long q_stride, int n_r
 
 // gb_attention_prefill_tc for a softmax with a distance bias, a sink and an output gate: the score of a key `dist` tokens
 // back loses r1[head] * ln(1 + r2[head] * dist) (r1 and r2 both or neither), the denominator also holds exp(sink[head]),
-// and the head's output is multiplied by sigmoid(gate[row * ld_gate + head]). Each term may be nullptr.
+// and the head's output is multiplied by sigmoid(gate[row * ld_gate + head]) (with gate_channels: each channel by a gate of
+// its own). Each term may be nullptr.
 GB_EXPORT int gb_attention_prefill_tc_sink(const void* q, long long q_stride, int n_rows, void* out, long long out_stride,
                                            const void* kcache, const void* vcache, const int* block_tables, int max_pages,
                                            const int* seq_first_row, const int* seq_start_pos, int num_seqs,
                                            int max_rows_per_seq, int nh, int nkv, int hd, int page_size, long long num_pages,
                                            float scale, int window, int* status, const float* r1, const float* r2,
-                                           const float* sink, const float* gate, long long ld_gate, cudaStream_t stream) {
+                                           const float* sink, const float* gate, long long ld_gate, int gate_channels, cudaStream_t stream) {
     GB_REQUIRE((r1 == nullptr) == (r2 == nullptr), "gb_attention_prefill_tc_sink: the distance bias needs r1 and r2");
-    GB_REQUIRE(gate == nullptr || ld_gate >= nh, "gb_attention_prefill_tc_sink: rows of gate logits are too short");
-    const AtSinkTerms terms = {r1, r2, sink, gate, ld_gate};
+    GB_REQUIRE(gate == nullptr || ld_gate >= (long long)nh * (gate_channels ? hd : 1), "gb_attention_prefill_tc_sink: rows of gate logits are too short");
+    const AtSinkTerms terms = {r1, r2, sink, gate, ld_gate, gate_channels};
     return prefill_tc_launch<true>(q, q_stride, n_rows, out, out_stride, kcache, vcache, block_tables, max_pages, seq_first_row,
                                    seq_start_pos, num_seqs, max_rows_per_seq, nh, nkv, hd, page_size, num_pages, scale, window,
                                    status, stream, terms);

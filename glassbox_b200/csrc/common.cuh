@@ -60,6 +60,16 @@ __device__ __forceinline__ float gb_gelu_tanh_fast(float z) {
     return __fdividef(z, 1.0f + __expf(-1.5957691216057308f * (z + 0.044715f * z * z * z)));
 }
 
+// ln(1 + e^z), accurate for any z (also as a factor: no cancellation where e^z is small).
+__device__ __forceinline__ float gb_softplus(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
+
+// One gated unit, told apart by its two numbers: a negative slope selects gelu_tanh(gate) * up, a slope of zero
+// silu(gate) * up (neither clamps anything), a positive one the clamped unit.
+__device__ __forceinline__ float gb_gated_unit(float gate, float up, float limit, float slope) {
+    if (slope > 0.f) return gb_clamped_unit(gate, up, limit, slope);
+    return slope < 0.f ? gb_gelu_tanh(gate) * up : gate / (1.0f + expf(-gate)) * up;
+}
+
 __device__ __forceinline__ float gb_warp_sum(float v) {
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);

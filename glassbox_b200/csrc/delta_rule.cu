@@ -126,13 +126,17 @@ struct ChannelDeltaArgs {
     int* status;
     int decay_channels;     // dk: a decay per head and key channel (a, dt_bias: heads * dk); 1: one per head (a, dt_bias: heads)
     int flags;              // CD_* below
+    int q_at, k_at, v_at;   // where a row's queries, keys and values start
+    const float* skip;      // CD_SSD: [heads], how much of a token's own value joins its read-out
 };
 // CD_SILU_INPUTS: q, k and v pass SiLU as they are read (a mixer without convolutions in front).
 // CD_PLAIN: linear attention with a fixed decay per head, S <- decay_h S + k v^T, o = S^T q: no beta, no correction towards
 //           the value, no unit vectors, no factor on q; `a_log` then holds the decays themselves, a, beta and dt_bias are not read.
+// CD_SSD: (with CD_PLAIN) a state-space mixer, S <- exp(-exp(a_log) dt) S + dt k v^T, o = S^T q + skip v with a step
+//           dt = softplus(a + dt_bias) per head and token: the decays come from a and dt_bias after all.
 // CD_GATE_SILU: the decoding form's output gate is silu(gate) instead of sigmoid(gate).
 // CD_NO_NORM: the decoding form leaves the read-out as it is (float32, no norm, no gate), for a norm that spans the heads.
-enum { CD_SILU_INPUTS = 1, CD_PLAIN = 2, CD_GATE_SILU = 4, CD_NO_NORM = 8 };
+enum { CD_SILU_INPUTS = 1, CD_PLAIN = 2, CD_GATE_SILU = 4, CD_NO_NORM = 8, CD_SSD = 16 };
 __device__ __forceinline__ float cd_silu(float v) { return v / (1.0f + expf(-v)); }
 
 template <int DPT, int NS>
@@ -160,8 +164,9 @@ __global__ void __launch_bounds__(CD_THREADS) channel_delta_kernel(ChannelDeltaA
     const int buf_floats = TC * per_token;
     // one buffer: q [TC][row_w], k [TC][row_w], g [TC][row_w], v [TC][cols], scalars [TC][4] = (beta, 1/|q| / sqrt(dk), 1/|k|, -)
     const int n_chunks = (r1 - r0 + TC - 1) / TC;
-    const bool plain = p.flags & CD_PLAIN, silu_in = p.flags & CD_SILU_INPUTS;
-    const float decay_rate = plain ? 0.f : expf(p.a_log[head]);
+    const bool plain = p.flags & CD_PLAIN, silu_in = p.flags & CD_SILU_INPUTS, ssd = p.flags & CD_SSD;
+    const float decay_rate = plain && !ssd ? 0.f : expf(p.a_log[head]);
+    const float skip = ssd ? p.skip[head] : 0.f;
     const float fixed_decay = plain ? p.a_log[head] : 1.f;
     const float q_scale = plain ? 1.0f : 1.0f / sqrtf((float)dk);
     const float corr = plain ? 0.f : 1.f;               // how much of S^T k is taken off the value
@@ -178,10 +183,11 @@ __global__ void __launch_bounds__(CD_THREADS) channel_delta_kernel(ChannelDeltaA
         const int vidx = wt, vt_ = vidx >> cols_shift, vcl = vidx & (cols - 1), vcc = blockIdx.z * cols + vcl;
         float vv = 0.f, bb = 0.f;
         if (vidx < nt * cols && vcc < dv) {
-            vv = p.qkv[(size_t)(c0 + vt_) * p.ldq + (size_t)2 * p.kv_heads * dk + (size_t)head * dv + vcc];
+            vv = p.qkv[(size_t)(c0 + vt_) * p.ldq + p.v_at + (size_t)head * dv + vcc];
             if (silu_in) vv = cd_silu(vv);
         }
         if (wt < nt && !plain) bb = p.beta[(size_t)(c0 + wt) * p.ldb + head];
+        if (wt < nt && ssd) bb = gb_softplus(p.a[(size_t)(c0 + wt) * p.lda + head] + p.dt_bias[head]);
         constexpr int U = 8;
         for (int base = wt; base < total; base += CD_STAGERS * U) {
             float qv[U], kv[U], zv[U];
@@ -193,9 +199,9 @@ __global__ void __launch_bounds__(CD_THREADS) channel_delta_kernel(ChannelDeltaA
                 zv[u] = -1e30f;
                 if (idx < total && d < dk) {
                     const size_t row = (size_t)(c0 + t);
-                    qv[u] = p.qkv[row * p.ldq + (size_t)kvh * dk + d];
-                    kv[u] = p.qkv[row * p.ldq + (size_t)(p.kv_heads + kvh) * dk + d];
-                    if (!plain) {
+                    qv[u] = p.qkv[row * p.ldq + p.q_at + (size_t)kvh * dk + d];
+                    kv[u] = p.qkv[row * p.ldq + p.k_at + (size_t)kvh * dk + d];
+                    if (!plain || ssd) {
                         const size_t ai = (size_t)head * dc + (dc > 1 ? d : 0);
                         zv[u] = p.a[row * p.lda + ai] + p.dt_bias[ai];
                     }
@@ -211,7 +217,8 @@ __global__ void __launch_bounds__(CD_THREADS) channel_delta_kernel(ChannelDeltaA
                     const float sp = zv[u] > 15.f ? zv[u] : __logf(1.0f + __expf(zv[u]));     // (padding channels: sp = 0, g = 1)
                     qs[at] = qv[u];
                     ks[at] = kv[u];
-                    gs[at] = (plain && d < dk) ? fixed_decay : __expf(-decay_rate * sp);
+                    gs[at] = ssd ? (d < dk ? expf(-decay_rate * gb_softplus(zv[u])) : 1.f)
+                                 : (plain && d < dk) ? fixed_decay : __expf(-decay_rate * sp);
                 }
             }
         }
@@ -219,10 +226,10 @@ __global__ void __launch_bounds__(CD_THREADS) channel_delta_kernel(ChannelDeltaA
         for (int idx = wt + CD_STAGERS; idx < nt * cols; idx += CD_STAGERS) {     // (more than 256 values: few splits, many columns)
             const int t = idx >> cols_shift, cl = idx & (cols - 1);
             const int cc = blockIdx.z * cols + cl;
-            float val = cc < dv ? p.qkv[(size_t)(c0 + t) * p.ldq + (size_t)2 * p.kv_heads * dk + (size_t)head * dv + cc] : 0.f;
+            float val = cc < dv ? p.qkv[(size_t)(c0 + t) * p.ldq + p.v_at + (size_t)head * dv + cc] : 0.f;
             vs[idx] = silu_in ? cd_silu(val) : val;
         }
-        if (wt < nt) sc[wt * 4] = plain ? 1.0f : 1.0f / (1.0f + __expf(-bb));
+        if (wt < nt) sc[wt * 4] = ssd ? bb : plain ? 1.0f : 1.0f / (1.0f + __expf(-bb));
         asm volatile("bar.sync 1, 256;" ::: "memory");         // the stagers among themselves
         const int lane = wt & 31;
         for (int t = wt >> 5; t < nt; t += CD_STAGERS / 32) {
@@ -332,6 +339,7 @@ __global__ void __launch_bounds__(CD_THREADS) channel_delta_kernel(ChannelDeltaA
                     a3 = fmaf(S[4 * i + 3], q.w, a3);
                 }
                 o_part = ((a0 + a1) + (a2 + a3)) * scal.y;
+                if (split == 0) o_part = fmaf(skip, vt, o_part);
                 o_row = c0 + t;
             }
         }
@@ -351,17 +359,9 @@ __global__ void __launch_bounds__(CD_THREADS) channel_delta_kernel(ChannelDeltaA
     }
 }
 
-GB_EXPORT int gb_channel_delta(const float* qkv, long long ldq, const float* beta, long long ldb, const float* a, long long lda,
-                               const float* dt_bias, const float* a_log, float* state, long long state_stride, float* out,
-                               const int* seq_first_row, const int* seq_start_pos, const int* seq_slots, int S, int heads,
-                               int kv_heads, int dk, int dv, int num_slots, int write_state, int* status, int decay_channels,
-                               int flags, cudaStream_t stream) {
-    GB_REQUIRE(S >= 0 && heads > 0 && kv_heads > 0 && heads % kv_heads == 0, "gb_channel_delta: heads %d must be a multiple of key heads %d",
-               heads, kv_heads);
-    GB_REQUIRE(decay_channels == 1 || decay_channels == dk, "gb_channel_delta: %d decays per head (one, or one per key channel)",
-               decay_channels);
-    GB_REQUIRE(dk > 0 && dk <= 1024 && dv > 0, "gb_channel_delta: a key size of %d is outside 1..1024", dk);
-    if (S == 0) return 0;
+// How many splits of the key dimension and how many tokens a chunk take, then the launch.
+static int channel_delta_launch(ChannelDeltaArgs p, int S, cudaStream_t stream) {
+    const int dk = p.dk, heads = p.heads, dv = p.dv;
     const int dpt = dk <= 128 ? 16 : 32;
     int ns = 1;
     while (ns * dpt < dk) ns *= 2;
@@ -370,8 +370,8 @@ GB_EXPORT int gb_channel_delta(const float* qkv, long long ldq, const float* bet
     int tc = (64 * 1024) / (2 * per_token);      // two buffers
     if (tc > 16) tc = 16;
     if (tc < 1) tc = 1;
-    ChannelDeltaArgs p = {qkv, ldq, beta, ldb, a, lda, dt_bias, a_log, state, state_stride, out, seq_first_row, seq_start_pos,
-                          seq_slots, heads, kv_heads, dk, dv, ns, tc, num_slots, write_state, status, decay_channels, flags};
+    p.ns = ns;
+    p.tc = tc;
     dim3 grid(S, heads, gb_ceil_div(dv, cols));
     const size_t smem = (size_t)2 * tc * per_token;
     bool launched = false;
@@ -389,6 +389,40 @@ GB_EXPORT int gb_channel_delta(const float* qkv, long long ldq, const float* bet
 #undef CD_CASE
     GB_REQUIRE(launched, "gb_channel_delta: no kernel for a key size of %d", dk);
     return gb_check_launch("gb_channel_delta");
+}
+
+GB_EXPORT int gb_channel_delta(const float* qkv, long long ldq, const float* beta, long long ldb, const float* a, long long lda,
+                               const float* dt_bias, const float* a_log, float* state, long long state_stride, float* out,
+                               const int* seq_first_row, const int* seq_start_pos, const int* seq_slots, int S, int heads,
+                               int kv_heads, int dk, int dv, int num_slots, int write_state, int* status, int decay_channels,
+                               int flags, cudaStream_t stream) {
+    GB_REQUIRE(S >= 0 && heads > 0 && kv_heads > 0 && heads % kv_heads == 0, "gb_channel_delta: heads %d must be a multiple of key heads %d",
+               heads, kv_heads);
+    GB_REQUIRE(decay_channels == 1 || decay_channels == dk, "gb_channel_delta: %d decays per head (one, or one per key channel)",
+               decay_channels);
+    GB_REQUIRE(dk > 0 && dk <= 1024 && dv > 0, "gb_channel_delta: a key size of %d is outside 1..1024", dk);
+    if (S == 0) return 0;
+    ChannelDeltaArgs p = {qkv, ldq, beta, ldb, a, lda, dt_bias, a_log, state, state_stride, out, seq_first_row, seq_start_pos,
+                          seq_slots, heads, kv_heads, dk, dv, 0, 0, num_slots, write_state, status, decay_channels, flags,
+                          0, kv_heads * dk, 2 * kv_heads * dk, nullptr};
+    return channel_delta_launch(p, S, stream);
+}
+
+// The state-space recurrence on the same walk: per head S <- exp(-exp(a_log) dt) S + dt B x^T, y = S^T C + skip x with
+// dt = softplus(dt_raw + dt_bias); heads share B and C in `groups`. xbc float32 rows [x: heads * dv | B: groups * dk | C: groups * dk],
+// dt_raw float32 [n, heads] (row stride ld_dt), y float32 [n, heads * dv].
+GB_EXPORT int gb_ssd_walk(const float* xbc, long long ldx, const float* dt_raw, long long ld_dt, const float* dt_bias, const float* a_log,
+                          const float* skip, float* state, long long state_stride, float* y, const int* seq_first_row,
+                          const int* seq_start_pos, const int* seq_slots, int S, int heads, int groups, int dk, int dv, int num_slots,
+                          int write_state, int* status, cudaStream_t stream) {
+    GB_REQUIRE(S >= 0 && heads > 0 && groups > 0 && heads % groups == 0, "gb_ssd_walk: heads %d must be a multiple of groups %d", heads, groups);
+    GB_REQUIRE(dk > 0 && dk <= 1024 && dv > 0, "gb_ssd_walk: a state size of %d is outside 1..1024", dk);
+    if (S == 0) return 0;
+    const int inner = heads * dv;
+    ChannelDeltaArgs p = {xbc, ldx, nullptr, 0, dt_raw, ld_dt, dt_bias, a_log, state, state_stride, y, seq_first_row, seq_start_pos,
+                          seq_slots, heads, groups, dk, dv, 0, 0, num_slots, write_state, status, 1, CD_PLAIN | CD_SSD,
+                          inner + groups * dk, inner, 0, skip};
+    return channel_delta_launch(p, S, stream);
 }
 
 // ----------------------------------------------------------------------------------------------
@@ -792,7 +826,8 @@ GB_EXPORT int gb_channel_delta_decode(const float* qkv, long long ldq, const flo
                "gb_channel_delta_decode: the fused form takes low ranks up to %d in all", CD_MAX_LOW_RANK);
     if (S == 0) return 0;
     ChannelDeltaArgs p = {qkv, ldq, beta, ldb, a, lda, dt_bias, a_log, state, state_stride, nullptr, seq_first_row, seq_start_pos,
-                          seq_slots, heads, kv_heads, dk, dv, 0, 0, num_slots, write_state, status, decay_channels, flags};
+                          seq_slots, heads, kv_heads, dk, dv, 0, 0, num_slots, write_state, status, decay_channels, flags,
+                          0, kv_heads * dk, 2 * kv_heads * dk, nullptr};
     if (flags & CD_NO_NORM) p.out = (float*)att;
     DeltaDecodeFusion f = {proj, ldp, conv_w, conv_state_off, taps, 2 * kv_heads * dk + heads * dv, a1_at, ra, rg, w_a2, w_g2};
     dim3 grid(S, heads);

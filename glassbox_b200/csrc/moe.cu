@@ -8,8 +8,11 @@
 //                    renormalised. Also the gate of a shared expert, sigmoid(w_gate . h), one number per row.
 //                    With softmax_chosen the scores are the logits themselves (plus a stored bias per expert), the `top`
 //                    largest are taken and their weights are the softmax over the chosen logits alone.
-//                    An expert is either W_down relu(W_up h)^2 or (UNIT) W_down unit(W_gate h, W_up h) with the clamped
-//                    gated unit g * sigmoid(slope g) * (u + 1), g = min(gate, limit), u = clamp(up, -limit, limit); its
+//                    With softmax scores s = softmax(logits) over all experts; a run's score is the largest in it (run_best
+//                    1; else the sum of its two largest), and with renorm_eps >= 0 the chosen scores are divided by
+//                    (their sum + renorm_eps).
+//                    An expert is either W_down relu(W_up h)^2 or (UNIT) W_down unit(W_gate h, W_up h) with one of the gated
+//                    units of gb_gated_unit (the clamped one, gelu_tanh(gate) * up or silu(gate) * up); its
 //                    up matrix then holds gate row f and up row f as rows 2f and 2f + 1.
 //   moe_expert_rows  one block per (row, chosen expert): act = relu(W_up[e] h)^2 in shared memory, then W_down[e] act,
 //                    written as float32 per (row, choice). Reads the two matrices of one expert once per block: the
@@ -20,6 +23,7 @@
 #include <math.h>
 
 constexpr int MOE_MAX_EXPERTS = 512;
+enum { MOE_SIGMOID = 0, MOE_SOFTMAX_CHOSEN = 1, MOE_SOFTMAX = 2 };      // how logits become scores and weights
 constexpr int MOE_ROUTE_THREADS = 1024;      // at most; the launch takes a warp per expert (and one for the shared gate)
 
 __device__ __forceinline__ float moe_sigmoid(float v) { return 1.0f / (1.0f + expf(-v)); }
@@ -85,7 +89,8 @@ __device__ __forceinline__ int moe_warp_argmax(const float* v, int count, int la
 // The choice for one row, by one warp: `score`, `choice` (score + correction), `run_score` and `kept` are the row's arrays.
 __device__ __forceinline__ void moe_choose(const float* score, float* choice, float* run_score, unsigned char* kept, int E, int top,
                                            int groups, int keep, float route_scale, int* choice_out, float* weight_out, int lane,
-                                           bool softmax_chosen = false) {
+                                           int scoring, int run_best, float renorm_eps) {
+    const bool softmax_chosen = scoring == MOE_SOFTMAX_CHOSEN;
     if (groups > 1 && keep < groups) {
         const int per = E / groups;
         for (int g = lane; g < groups; g += 32) {
@@ -94,7 +99,7 @@ __device__ __forceinline__ void moe_choose(const float* score, float* choice, fl
                 const float c = choice[g * per + i];
                 if (c > a) { b = a; a = c; } else if (c > b) { b = c; }
             }
-            run_score[g] = per > 1 ? a + b : a;
+            run_score[g] = per > 1 && !run_best ? a + b : a;
             kept[g] = 0;
         }
         __syncwarp();
@@ -133,7 +138,13 @@ __device__ __forceinline__ void moe_choose(const float* score, float* choice, fl
             const float inv = 1.0f / sum;
             for (int k = 0; k < top; ++k) weight_out[k] = run_score[k] * inv;
         } else {
-            for (int k = 0; k < top; ++k) weight_out[k] = run_score[k];
+            float f = 1.0f;
+            if (renorm_eps >= 0.f) {
+                float sum = renorm_eps;
+                for (int k = 0; k < top; ++k) sum += run_score[k];
+                f = 1.0f / sum;
+            }
+            for (int k = 0; k < top; ++k) weight_out[k] = run_score[k] * f;
         }
     }
 }
@@ -146,7 +157,7 @@ __global__ void __launch_bounds__(RB > 1 ? MOE_ROUTE_THREADS / 2 : MOE_ROUTE_THR
     const T* __restrict__ h, int d, const float* __restrict__ w_router, const float* __restrict__ correction,
     const float* __restrict__ w_gate, const int* __restrict__ positions, int n, int E, int top, int groups, int keep,
     float route_scale, int* __restrict__ choice_out, float* __restrict__ weight_out, float* __restrict__ gate_out,
-    const float* __restrict__ router_bias, int softmax_chosen) {
+    const float* __restrict__ router_bias, int scoring, int run_best, float renorm_eps) {
     extern __shared__ __align__(16) float moe_smem[];
     float* hx = moe_smem;                       // RB rows of d numbers (rows start 16-byte aligned: ldh is a multiple of 4)
     const int ldh = (d + 3) & ~3;
@@ -196,7 +207,7 @@ __global__ void __launch_bounds__(RB > 1 ? MOE_ROUTE_THREADS / 2 : MOE_ROUTE_THR
             const int row = row0 + r;
             if (lane == 0 && row < n && positions[row] >= 0) {
                 const float sg = moe_sigmoid(z);
-                if (e < E && softmax_chosen) {
+                if (e < E && scoring != MOE_SIGMOID) {
                     score[r][e] = choice[r][e] = z + (router_bias ? router_bias[e] : 0.f);
                 } else if (e < E) {
                     score[r][e] = sg;
@@ -210,16 +221,28 @@ __global__ void __launch_bounds__(RB > 1 ? MOE_ROUTE_THREADS / 2 : MOE_ROUTE_THR
     __syncthreads();
     for (int r = warp; r < RB; r += warps) {
         const int row = row0 + r;
-        if (row < n && positions[row] >= 0)
-            moe_choose(score[r], choice[r], run_score[r], kept[r], E, top, groups, keep, softmax_chosen ? 1.0f : route_scale,
-                       choice_out + (size_t)row * top, weight_out + (size_t)row * top, lane, softmax_chosen != 0);
+        if (row < n && positions[row] >= 0) {
+            if (scoring == MOE_SOFTMAX) {        // the row's logits become its softmax over all experts, by this row's warp
+                float m = -INFINITY, sum = 0.f;
+                for (int e = lane; e < E; e += 32) m = fmaxf(m, score[r][e]);
+                m = gb_warp_max(m);
+                for (int e = lane; e < E; e += 32) sum += expf(score[r][e] - m);
+                sum = gb_warp_sum(sum);
+                for (int e = lane; e < E; e += 32) score[r][e] = choice[r][e] = expf(score[r][e] - m) / sum;
+                __syncwarp();
+            }
+            moe_choose(score[r], choice[r], run_score[r], kept[r], E, top, groups, keep,
+                       scoring == MOE_SOFTMAX_CHOSEN ? 1.0f : route_scale, choice_out + (size_t)row * top,
+                       weight_out + (size_t)row * top, lane, scoring, run_best, renorm_eps);
+        }
     }
 }
 
 template <typename T, int RB, int EMAX>
 static void moe_route_launch(const void* h, int d, const float* w_router, const float* correction, const float* w_gate,
                              const int* positions, int n, int E, int top, int groups, int keep, float route_scale, int* choice_out,
-                             float* weight_out, float* gate_out, const float* router_bias, int softmax_chosen, cudaStream_t stream) {
+                             float* weight_out, float* gate_out, const float* router_bias, int scoring, int run_best, float renorm_eps,
+                             cudaStream_t stream) {
     const size_t smem = (size_t)RB * ((d + 3) & ~3) * 4;
     int warps = E + (w_gate ? 1 : 0);
     const int most = (RB > 1 ? MOE_ROUTE_THREADS / 2 : MOE_ROUTE_THREADS) / 32, least = RB > 4 ? RB : 4;
@@ -227,13 +250,16 @@ static void moe_route_launch(const void* h, int d, const float* w_router, const 
     if (smem > 32 * 1024) cudaFuncSetAttribute(moe_route_kernel<T, RB, EMAX>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     gb_launch(GB_PDL_ELEMENTWISE, moe_route_kernel<T, RB, EMAX>, dim3(gb_ceil_div(n, RB)), dim3(32 * warps), smem, stream, (const T*)h, d,
               w_router, correction, w_gate, positions, n, E, top, groups, keep, route_scale, choice_out, weight_out, gate_out, router_bias,
-              softmax_chosen);
+              scoring, run_best, renorm_eps);
 }
 
 GB_EXPORT int gb_moe_route(const void* h, int h_dtype, int d, const float* w_router, const float* correction, const float* w_gate,
                            const int* positions, int n, int E, int top, int groups, int keep, float route_scale, int* choice_out,
-                           float* weight_out, float* gate_out, const float* router_bias, int softmax_chosen, cudaStream_t stream) {
-    GB_REQUIRE(!softmax_chosen || (groups == 1 && correction == nullptr), "gb_moe_route: softmax over the chosen logits goes with neither groups nor a correction");
+                           float* weight_out, float* gate_out, const float* router_bias, int scoring, int run_best, float renorm_eps,
+                           cudaStream_t stream) {
+    GB_REQUIRE(scoring >= MOE_SIGMOID && scoring <= MOE_SOFTMAX, "gb_moe_route: unknown scoring %d", scoring);
+    GB_REQUIRE(scoring == MOE_SIGMOID || correction == nullptr, "gb_moe_route: a choice correction goes with sigmoid scores");
+    GB_REQUIRE(scoring != MOE_SOFTMAX_CHOSEN || groups == 1, "gb_moe_route: softmax over the chosen logits goes without groups");
     GB_REQUIRE(n >= 0 && d > 0 && E > 0 && E <= MOE_MAX_EXPERTS && top > 0 && top <= E, "gb_moe_route: bad sizes (experts %d, top %d)", E,
                top);
     GB_REQUIRE(groups >= 1 && E % groups == 0 && keep >= 1 && keep <= groups, "gb_moe_route: %d experts in %d groups, %d kept", E, groups,
@@ -247,10 +273,10 @@ GB_EXPORT int gb_moe_route(const void* h, int h_dtype, int d, const float* w_rou
 #define MOE_ROUTE_GO(T)                                                                                                              \
     if (many)                                                                                                                        \
         moe_route_launch<T, 8, 128>(h, d, w_router, correction, w_gate, positions, n, E, top, groups, keep, route_scale, choice_out,  \
-                                    weight_out, gate_out, router_bias, softmax_chosen, stream);                                      \
+                                    weight_out, gate_out, router_bias, scoring, run_best, renorm_eps, stream);                       \
     else                                                                                                                             \
         moe_route_launch<T, 1, MOE_MAX_EXPERTS>(h, d, w_router, correction, w_gate, positions, n, E, top, groups, keep, route_scale,  \
-                                                choice_out, weight_out, gate_out, router_bias, softmax_chosen, stream);
+                                                choice_out, weight_out, gate_out, router_bias, scoring, run_best, renorm_eps, stream);
     if (h_dtype == GB_F32) { MOE_ROUTE_GO(float) } else { MOE_ROUTE_GO(__nv_bfloat16) }
 #undef MOE_ROUTE_GO
     return gb_check_launch("gb_moe_route");
@@ -385,7 +411,7 @@ __global__ void __launch_bounds__(256) moe_half_rows_kernel(const void* __restri
     if (wrow == nullptr) return;
     float v = moe_warp_dot<T>(wrow, x, K, lane);
     if (UP && unit) {
-        v = gb_clamped_unit(v, moe_warp_dot<T>(wrow + K, x, K, lane), limit, slope);
+        v = gb_gated_unit(v, moe_warp_dot<T>(wrow + K, x, K, lane), limit, slope);
     } else if (UP) {
         v = fmaxf(v, 0.f);
         v *= v;
@@ -590,7 +616,7 @@ __global__ void __launch_bounds__(MG_THREADS) moe_grouped_gemm_kernel(const __nv
                 float v0 = acc[i][j][half * 2], v1 = acc[i][j][half * 2 + 1];
                 if (UP && unit) {
                     // neighbouring outputs are the gate sum and the up sum of one unit: N / 2 units per row
-                    if (col + 1 < N) ((__nv_bfloat16*)C)[(size_t)out_row * ldc + (col >> 1)] = __float2bfloat16_rn(gb_clamped_unit(v0, v1, limit, slope));
+                    if (col + 1 < N) ((__nv_bfloat16*)C)[(size_t)out_row * ldc + (col >> 1)] = __float2bfloat16_rn(gb_gated_unit(v0, v1, limit, slope));
                 } else if (UP) {
                     v0 = fmaxf(v0, 0.f); v0 *= v0;
                     v1 = fmaxf(v1, 0.f); v1 *= v1;

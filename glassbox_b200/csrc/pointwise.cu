@@ -10,6 +10,8 @@
 //   gated_head_norm  out[r, h, :] = w * o[r, h, :] / sqrt(mean_v(o[r, h, :]^2) + eps) * sigmoid(gate[r, h, :])  (or * silu(gate))
 //   gelu_glu      act[r, f] = gelu_tanh(gate[r, f]) * up[r, f]
 //   scaled_sum    out (+)= a * x + b * y
+//   post_norm     x[r, :] <- gain * t / rms(t), t = alpha * x[r, :] + y[r, :] (y stored, or a weighted sum, or two normed branches)
+//   gate_group_norm  u = y * silu(z), each of equal parts of the row normed by its own root mean square, times a gain
 #include "common.cuh"
 
 // ----------------------------------------------------------------------------------------------
@@ -383,4 +385,294 @@ GB_EXPORT int gb_scaled_sum(const float* x, const float* y, float a, float b, fl
     if (count == 0) return 0;
     gb_launch(GB_PDL_ELEMENTWISE, scaled_sum_kernel, dim3(gb_ceil_div(count, 256)), dim3(256), 0, stream, x, y, a, b, out, count, accumulate);
     return gb_check_launch("gb_scaled_sum");
+}
+
+// ----------------------------------------------------------------------------------------------
+// A residual that is normed after the sum: x[r, :] <- gain * t / sqrt(mean(t^2) + eps) with t = alpha * x[r, :] + y[r, :], and
+// optionally a copy of the new row in the activation dtype. y comes as one of
+//   rows     y[r, :] as it is stored
+//   weighted sum_k weight[r, k] * pair[r, k, :] (+ gate[r] * shared[r, :]): a routed feed-forward's output in its parts
+//   pair     a_scale * (ga * a[r, :] / rms(a[r, :])) + b_scale * (gb * b[r, :] / rms(b[r, :])): two branches side by side, each
+//            normed over the row before they join
+// so that a branch costs one launch beside its own. One block per row; float32 throughout; padding rows are skipped.
+// ----------------------------------------------------------------------------------------------
+struct PostNormArgs {
+    float* x;
+    long long ldx;
+    const float* gain;
+    float alpha, eps;
+    const float* y;             // rows: y; pair: a
+    const float* b;             // pair: b
+    const float* ga;
+    const float* gb;
+    float a_scale, b_scale, pair_eps;
+    const float* weighted;      // weighted: [n, top * d]
+    const float* weight;
+    const float* shared;
+    const float* gate;
+    int top;
+    void* copy;
+    const int* positions;
+    int n, d;
+};
+enum { PN_ROWS = 0, PN_WEIGHTED = 1, PN_PAIR = 2 };
+constexpr int PN_THREADS = 256, PN_VMAX = 4;
+
+__device__ __forceinline__ float2 pn_block_sum2(float a, float b, float2* partial) {
+    a = gb_warp_sum(a);
+    b = gb_warp_sum(b);
+    __syncthreads();                 // (an earlier use of `partial` is over)
+    if ((threadIdx.x & 31) == 0) partial[threadIdx.x >> 5] = make_float2(a, b);
+    __syncthreads();
+    float2 t = make_float2(0.f, 0.f);
+#pragma unroll
+    for (int w = 0; w < PN_THREADS / 32; ++w) {
+        t.x += partial[w].x;
+        t.y += partial[w].y;
+    }
+    return t;
+}
+
+template <int MODE, int VMAX, typename T>
+__global__ void __launch_bounds__(PN_THREADS) post_norm_kernel(PostNormArgs p) {
+    __shared__ float2 partial[PN_THREADS / 32];
+    gb_pdl_launch_dependents();
+    gb_pdl_wait();
+    const int r = blockIdx.x;
+    if (r >= p.n || (p.positions != nullptr && p.positions[r] < 0)) return;
+    const int d = p.d, top = p.top;
+    float* x = p.x + (size_t)r * p.ldx;
+    T* cp = p.copy ? (T*)p.copy + (size_t)r * d : nullptr;
+    const float* y = p.y ? p.y + (size_t)r * d : nullptr;
+    const float* b = MODE == PN_PAIR ? p.b + (size_t)r * d : nullptr;
+    const float* rows = MODE == PN_WEIGHTED ? p.weighted + (size_t)r * top * d : nullptr;
+    const float* wt = MODE == PN_WEIGHTED ? p.weight + (size_t)r * top : nullptr;
+    const float* sh = MODE == PN_WEIGHTED && p.shared ? p.shared + (size_t)r * d : nullptr;
+    const float shg = MODE == PN_WEIGHTED && p.gate ? p.gate[r] : 1.0f;
+    if constexpr (VMAX > 0) {            // rows of whole 16-byte pieces that fit the block's registers: one trip to memory
+        float4 t[VMAX], v[VMAX], u[MODE == PN_PAIR ? VMAX : 1];
+#pragma unroll
+        for (int i = 0; i < VMAX; ++i) {
+            const int j = (i * PN_THREADS + threadIdx.x) * 4;
+            const bool in = j < d;
+            t[i] = in ? *reinterpret_cast<const float4*>(x + j) : make_float4(0.f, 0.f, 0.f, 0.f);
+            if constexpr (MODE != PN_WEIGHTED) v[i] = in ? *reinterpret_cast<const float4*>(y + j) : make_float4(0.f, 0.f, 0.f, 0.f);
+            if constexpr (MODE == PN_PAIR) u[i] = in ? *reinterpret_cast<const float4*>(b + j) : make_float4(0.f, 0.f, 0.f, 0.f);
+        }
+        if constexpr (MODE == PN_WEIGHTED) {
+#pragma unroll
+            for (int i = 0; i < VMAX; ++i) {
+                const int j = (i * PN_THREADS + threadIdx.x) * 4;
+                v[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+                if (j < d) {
+#pragma unroll 4
+                    for (int k = 0; k < top; ++k) {
+                        const float w = wt[k];
+                        const float4 q = *reinterpret_cast<const float4*>(rows + (size_t)k * d + j);
+                        v[i].x = fmaf(w, q.x, v[i].x); v[i].y = fmaf(w, q.y, v[i].y);
+                        v[i].z = fmaf(w, q.z, v[i].z); v[i].w = fmaf(w, q.w, v[i].w);
+                    }
+                    if (sh) {
+                        const float4 q = *reinterpret_cast<const float4*>(sh + j);
+                        v[i].x = fmaf(shg, q.x, v[i].x); v[i].y = fmaf(shg, q.y, v[i].y);
+                        v[i].z = fmaf(shg, q.z, v[i].z); v[i].w = fmaf(shg, q.w, v[i].w);
+                    }
+                }
+            }
+        }
+        if constexpr (MODE == PN_PAIR) {
+            float sa = 0.f, sb = 0.f;
+#pragma unroll
+            for (int i = 0; i < VMAX; ++i) {
+                sa = fmaf(v[i].x, v[i].x, sa); sa = fmaf(v[i].y, v[i].y, sa); sa = fmaf(v[i].z, v[i].z, sa); sa = fmaf(v[i].w, v[i].w, sa);
+                sb = fmaf(u[i].x, u[i].x, sb); sb = fmaf(u[i].y, u[i].y, sb); sb = fmaf(u[i].z, u[i].z, sb); sb = fmaf(u[i].w, u[i].w, sb);
+            }
+            const float2 s = pn_block_sum2(sa, sb, partial);
+            const float fa = p.a_scale / sqrtf(s.x / (float)d + p.pair_eps), fb = p.b_scale / sqrtf(s.y / (float)d + p.pair_eps);
+#pragma unroll
+            for (int i = 0; i < VMAX; ++i) {
+                const int j = (i * PN_THREADS + threadIdx.x) * 4;
+                if (j < d) {
+                    const float4 g = *reinterpret_cast<const float4*>(p.ga + j), h = *reinterpret_cast<const float4*>(p.gb + j);
+                    v[i].x = fmaf(g.x * fa, v[i].x, h.x * fb * u[i].x); v[i].y = fmaf(g.y * fa, v[i].y, h.y * fb * u[i].y);
+                    v[i].z = fmaf(g.z * fa, v[i].z, h.z * fb * u[i].z); v[i].w = fmaf(g.w * fa, v[i].w, h.w * fb * u[i].w);
+                }
+            }
+        }
+        float ss = 0.f;
+#pragma unroll
+        for (int i = 0; i < VMAX; ++i) {
+            t[i].x = fmaf(p.alpha, t[i].x, v[i].x); t[i].y = fmaf(p.alpha, t[i].y, v[i].y);
+            t[i].z = fmaf(p.alpha, t[i].z, v[i].z); t[i].w = fmaf(p.alpha, t[i].w, v[i].w);
+            ss = fmaf(t[i].x, t[i].x, ss); ss = fmaf(t[i].y, t[i].y, ss); ss = fmaf(t[i].z, t[i].z, ss); ss = fmaf(t[i].w, t[i].w, ss);
+        }
+        const float s = 1.0f / sqrtf(pn_block_sum2(ss, 0.f, partial).x / (float)d + p.eps);
+#pragma unroll
+        for (int i = 0; i < VMAX; ++i) {
+            const int j = (i * PN_THREADS + threadIdx.x) * 4;
+            if (j < d) {
+                const float4 g = *reinterpret_cast<const float4*>(p.gain + j);
+                const float4 w = make_float4(g.x * (t[i].x * s), g.y * (t[i].y * s), g.z * (t[i].z * s), g.w * (t[i].w * s));
+                *reinterpret_cast<float4*>(x + j) = w;
+                if (cp != nullptr) {
+                    cp[j] = gb_from_float<T>(w.x); cp[j + 1] = gb_from_float<T>(w.y);
+                    cp[j + 2] = gb_from_float<T>(w.z); cp[j + 3] = gb_from_float<T>(w.w);
+                }
+            }
+        }
+    } else {                             // any other row: a value is formed again in every pass
+        float fa = 0.f, fb = 0.f;
+        if constexpr (MODE == PN_PAIR) {
+            float sa = 0.f, sb = 0.f;
+            for (int j = threadIdx.x; j < d; j += PN_THREADS) {
+                sa = fmaf(y[j], y[j], sa);
+                sb = fmaf(b[j], b[j], sb);
+            }
+            const float2 s = pn_block_sum2(sa, sb, partial);
+            fa = p.a_scale / sqrtf(s.x / (float)d + p.pair_eps);
+            fb = p.b_scale / sqrtf(s.y / (float)d + p.pair_eps);
+        }
+        auto value = [&](int j) {
+            float v;
+            if constexpr (MODE == PN_ROWS) v = y[j];
+            if constexpr (MODE == PN_PAIR) v = fmaf(p.ga[j] * fa, y[j], p.gb[j] * fb * b[j]);
+            if constexpr (MODE == PN_WEIGHTED) {
+                v = 0.f;
+                for (int k = 0; k < top; ++k) v = fmaf(wt[k], rows[(size_t)k * d + j], v);
+                if (sh) v = fmaf(shg, sh[j], v);
+            }
+            return fmaf(p.alpha, x[j], v);
+        };
+        float ss = 0.f;
+        for (int j = threadIdx.x; j < d; j += PN_THREADS) {
+            const float t = value(j);
+            ss = fmaf(t, t, ss);
+        }
+        const float s = 1.0f / sqrtf(pn_block_sum2(ss, 0.f, partial).x / (float)d + p.eps);
+        for (int j = threadIdx.x; j < d; j += PN_THREADS) {
+            const float w = p.gain[j] * (value(j) * s);
+            x[j] = w;
+            if (cp != nullptr) cp[j] = gb_from_float<T>(w);
+        }
+    }
+}
+
+template <int MODE, typename T>
+static void post_norm_launch(const PostNormArgs& p, bool vec, cudaStream_t stream) {
+    const int pieces = gb_ceil_div(p.d, PN_THREADS * 4);
+    if (!vec || pieces > PN_VMAX) gb_launch(GB_PDL_ELEMENTWISE, post_norm_kernel<MODE, 0, T>, dim3(p.n), dim3(PN_THREADS), 0, stream, p);
+    else if (pieces == 1) gb_launch(GB_PDL_ELEMENTWISE, post_norm_kernel<MODE, 1, T>, dim3(p.n), dim3(PN_THREADS), 0, stream, p);
+    else if (pieces == 2) gb_launch(GB_PDL_ELEMENTWISE, post_norm_kernel<MODE, 2, T>, dim3(p.n), dim3(PN_THREADS), 0, stream, p);
+    else gb_launch(GB_PDL_ELEMENTWISE, post_norm_kernel<MODE, 4, T>, dim3(p.n), dim3(PN_THREADS), 0, stream, p);
+}
+
+// mode 0: y [n, d]; 1: weighted [n, top * d], weight [n, top], shared [n, d] or nullptr, gate [n] or nullptr; 2: y and b [n, d] with
+// gains ga, gb [d]. All rows of y, b, weighted and shared are contiguous. copy: [n, d] of copy_dtype or nullptr.
+GB_EXPORT int gb_post_norm(float* x, long long ldx, const float* gain, float alpha, float eps, int mode, const float* y, const float* b,
+                           const float* ga, const float* gb, float a_scale, float b_scale, float pair_eps, const float* weighted,
+                           const float* weight, int top, const float* shared, const float* gate, void* copy, int copy_dtype,
+                           const int* positions, int n, int d, cudaStream_t stream) {
+    GB_REQUIRE(n >= 0 && d > 0 && ldx >= d, "gb_post_norm: bad sizes n=%d d=%d", n, d);
+    GB_REQUIRE(mode == PN_ROWS ? y != nullptr : mode == PN_WEIGHTED ? (weighted != nullptr && weight != nullptr && top > 0)
+                                              : (mode == PN_PAIR && y != nullptr && b != nullptr && ga != nullptr && gb != nullptr),
+               "gb_post_norm: mode %d lacks its operands", mode);
+    GB_REQUIRE(copy == nullptr || copy_dtype == GB_F32 || copy_dtype == GB_BF16, "gb_post_norm: unsupported dtype %d", copy_dtype);
+    if (n == 0) return 0;
+    PostNormArgs p = {x, ldx, gain, alpha, eps, y, b, ga, gb, a_scale, b_scale, pair_eps, weighted, weight, shared, gate, top, copy,
+                      positions, n, d};
+    const uintptr_t all = (uintptr_t)x | (uintptr_t)gain | (uintptr_t)y | (uintptr_t)b | (uintptr_t)ga | (uintptr_t)gb | (uintptr_t)weighted |
+                          (uintptr_t)shared;
+    const bool vec = d % 4 == 0 && ldx % 4 == 0 && (all & 15) == 0;
+    const bool half = copy != nullptr && copy_dtype == GB_BF16;
+#define PN_GO(M)                                                                \
+    if (mode == M) {                                                            \
+        if (half) post_norm_launch<M, __nv_bfloat16>(p, vec, stream);           \
+        else post_norm_launch<M, float>(p, vec, stream);                        \
+    }
+    PN_GO(PN_ROWS) PN_GO(PN_WEIGHTED) PN_GO(PN_PAIR)
+#undef PN_GO
+    return gb_check_launch("gb_post_norm");
+}
+
+// ----------------------------------------------------------------------------------------------
+// A gate in front of a norm over equal parts of a row: u = y * silu(z), out = w * u / sqrt(mean over the part of u^2 + eps).
+// y float32 [n, groups * size], z float32 logits (row stride ldz), w float32 [groups * size]. One block per (row, part).
+// ----------------------------------------------------------------------------------------------
+template <int THREADS, typename T>
+__global__ void __launch_bounds__(THREADS) gate_group_norm_kernel(const float* __restrict__ y, const float* __restrict__ z, long long ldz,
+                                                                  const float* __restrict__ w, T* __restrict__ out,
+                                                                  const int* __restrict__ positions, int groups, int size, float eps,
+                                                                  int vec) {
+    __shared__ float partial[THREADS / 32];
+    gb_pdl_launch_dependents();
+    gb_pdl_wait();
+    const int row = blockIdx.x / groups, g = blockIdx.x % groups;
+    if (positions != nullptr && positions[row] < 0) return;
+    const size_t at = (size_t)blockIdx.x * size;
+    const float* src = y + at;
+    const float* gz = z + (size_t)row * ldz + (size_t)g * size;
+    const float* gw = w + (size_t)g * size;
+    T* dst = out + at;
+    constexpr int VMAX = 4;
+    float4 u[VMAX];
+    float ss = 0.f;
+    const bool quick = vec && size <= THREADS * 4 * VMAX;
+    auto gated = [](float a, float b) { return a * (b / (1.0f + expf(-b))); };
+    if (quick) {
+        float4 q[VMAX];
+#pragma unroll
+        for (int i = 0; i < VMAX; ++i) {
+            const int j = (i * THREADS + threadIdx.x) * 4;
+            u[i] = j < size ? *reinterpret_cast<const float4*>(src + j) : make_float4(0.f, 0.f, 0.f, 0.f);
+            q[i] = j < size ? *reinterpret_cast<const float4*>(gz + j) : make_float4(0.f, 0.f, 0.f, 0.f);
+        }
+#pragma unroll
+        for (int i = 0; i < VMAX; ++i) {
+            u[i] = make_float4(gated(u[i].x, q[i].x), gated(u[i].y, q[i].y), gated(u[i].z, q[i].z), gated(u[i].w, q[i].w));
+            ss = fmaf(u[i].x, u[i].x, ss); ss = fmaf(u[i].y, u[i].y, ss); ss = fmaf(u[i].z, u[i].z, ss); ss = fmaf(u[i].w, u[i].w, ss);
+        }
+    } else {
+        for (int j = threadIdx.x; j < size; j += THREADS) {
+            const float t = gated(src[j], gz[j]);
+            ss = fmaf(t, t, ss);
+        }
+    }
+    ss = gb_warp_sum(ss);
+    if ((threadIdx.x & 31) == 0) partial[threadIdx.x >> 5] = ss;
+    __syncthreads();
+    ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < THREADS / 32; ++i) ss += partial[i];
+    const float s = 1.0f / sqrtf(ss / (float)size + eps);
+    if (quick) {
+#pragma unroll
+        for (int i = 0; i < VMAX; ++i) {
+            const int j = (i * THREADS + threadIdx.x) * 4;
+            if (j < size) {
+                const float4 g4 = *reinterpret_cast<const float4*>(gw + j);
+                dst[j] = gb_from_float<T>(g4.x * (u[i].x * s)); dst[j + 1] = gb_from_float<T>(g4.y * (u[i].y * s));
+                dst[j + 2] = gb_from_float<T>(g4.z * (u[i].z * s)); dst[j + 3] = gb_from_float<T>(g4.w * (u[i].w * s));
+            }
+        }
+    } else {
+        for (int j = threadIdx.x; j < size; j += THREADS) dst[j] = gb_from_float<T>(gw[j] * (gated(src[j], gz[j]) * s));
+    }
+}
+
+GB_EXPORT int gb_gate_group_norm(const float* y, const float* z, long long ldz, const float* w, void* out, int out_dtype,
+                                 const int* positions, int n, int groups, int size, float eps, cudaStream_t stream) {
+    GB_REQUIRE(n >= 0 && groups > 0 && size > 0 && ldz >= (long long)groups * size, "gb_gate_group_norm: bad sizes");
+    GB_REQUIRE(out_dtype == GB_F32 || out_dtype == GB_BF16, "gb_gate_group_norm: unsupported output dtype %d", out_dtype);
+    if (n == 0) return 0;
+    const int vec = size % 4 == 0 && ldz % 4 == 0 && (((uintptr_t)y | (uintptr_t)z | (uintptr_t)w) & 15) == 0;
+#define GGN_GO(TH, T)                                                                                                            \
+    gb_launch(GB_PDL_ELEMENTWISE, gate_group_norm_kernel<TH, T>, dim3(n * groups), dim3(TH), 0, stream, y, z, ldz, w, (T*)out,   \
+              positions, groups, size, eps, vec)
+    if (size <= 512) {
+        if (out_dtype == GB_F32) GGN_GO(64, float); else GGN_GO(64, __nv_bfloat16);
+    } else {
+        if (out_dtype == GB_F32) GGN_GO(256, float); else GGN_GO(256, __nv_bfloat16);
+    }
+#undef GGN_GO
+    return gb_check_launch("gb_gate_group_norm");
 }

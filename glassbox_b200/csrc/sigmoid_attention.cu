@@ -8,7 +8,9 @@
 //                        (2i, 2i+1) by the angle float32(position) * inv_freq[i], q to the query buffer, k and v into the
 //                        cache at the row's slot. Input: the float32 sums of the stacked projection q | k | v. Optionally
 //                        the values are mixed on the way: values_in given, v <- (1 - lambda) v + lambda values_in[row]
-//                        (lambda one float32 number on the device); values_out given, it receives the row's (mixed) v.
+//                        (lambda one float32 number on the device); values_out given, it receives the row's (mixed) v. A norm
+//                        may lack its gains (unit_norm), and queries may carry a temperature: q at position p is multiplied
+//                        by 1 + temp_coef * ln(floor((p + 1) / temp_every) + 1) (temp_every 0: none), in float32.
 //   sigmoid_attention_rows  one warp per (row, head), any row (prompt portion or single token), both dtypes: 32 keys at a
 //                        time from the first visible one, a lane per key for the scores, a lane per channel for the sum.
 #include "common.cuh"
@@ -22,7 +24,7 @@ __global__ void __launch_bounds__(512) qk_norm_rope_write_kernel(
     const float* __restrict__ inv_freq, const int* __restrict__ positions, const int* __restrict__ slots, T* __restrict__ q_out,
     T* __restrict__ kcache, T* __restrict__ vcache, int n, int H, int G, int D, int V, int rot, float eps, int page_size,
     long long num_slots, int write_kv, int* __restrict__ status, float* __restrict__ values_out, const float* __restrict__ values_in,
-    long long ld_values, const float* __restrict__ value_mix) {
+    long long ld_values, const float* __restrict__ value_mix, int unit_norm, float temp_coef, float temp_every) {
     gb_pdl_launch_dependents();
     gb_pdl_wait();
     const int row = blockIdx.x;
@@ -40,18 +42,20 @@ __global__ void __launch_bounds__(512) qk_norm_rope_write_kernel(
     const long long page = slot / page_size;
     const int off = (int)(slot % page_size);
     const int pairs = D / 2;          // (an odd last channel is handled apart)
+    const float temp = temp_every > 0.f ? 1.0f + temp_coef * logf(floorf(__fdiv_rn((float)(pos + 1), temp_every)) + 1.0f) : 1.0f;
     for (int head = warp; head < H + G; head += warps) {
         const bool is_q = head < H;
         if (!is_q && !store) continue;
         const float* x = src + (size_t)head * D;     // q heads, then k heads: contiguous in the stacked row
-        const float* gain = is_q ? q_gain : k_gain;      // nullptr: the heads are not normed
+        const float* gain = is_q ? q_gain : k_gain;      // nullptr: the heads are not normed, or (unit_norm) normed without a gain
         float r = 1.f;
-        if (gain != nullptr) {
+        if (gain != nullptr || unit_norm) {
             float ss = 0.f;
             for (int i = lane; i < D; i += 32) ss = fmaf(x[i], x[i], ss);
             ss = gb_warp_sum(ss);
             r = 1.0f / sqrtf(ss / (float)D + eps);
         }
+        if (is_q) r *= temp;
         T* dst = is_q ? q_out + ((size_t)row * H + head) * D
                       : kcache + ((page * G + (head - H)) * page_size + off) * D;
         for (int i = lane; i < pairs; i += 32) {
@@ -89,7 +93,8 @@ GB_EXPORT int gb_qk_norm_rope_write(const float* qkv, long long ld, const float*
                                     const int* positions, const int* slots, void* q_out, void* kcache, void* vcache, int dtype, int n,
                                     int H, int G, int D, int V, int rot, float eps, int page_size, long long num_slots, int write_kv,
                                     int* status, float* values_out, const float* values_in, long long ld_values,
-                                    const float* value_mix, cudaStream_t stream) {
+                                    const float* value_mix, int unit_norm, float temp_coef, float temp_every, cudaStream_t stream) {
+    GB_REQUIRE(temp_every >= 0.f, "gb_qk_norm_rope_write: the query temperature's step must be positive (0: none)");
     GB_REQUIRE(n >= 0 && H > 0 && G > 0 && D > 0 && V > 0, "gb_qk_norm_rope_write: bad sizes");
     GB_REQUIRE(values_in == nullptr || value_mix != nullptr, "gb_qk_norm_rope_write: values to mix in need their weight");
     GB_REQUIRE((values_in == nullptr && values_out == nullptr) || ld_values >= (long long)G * V, "gb_qk_norm_rope_write: rows of values are too short");
@@ -100,11 +105,11 @@ GB_EXPORT int gb_qk_norm_rope_write(const float* qkv, long long ld, const float*
     if (dtype == GB_F32)
         gb_launch(GB_PDL_ELEMENTWISE, qk_norm_rope_write_kernel<float>, dim3(n), block, 0, stream, qkv, ld, q_gain, k_gain, inv_freq,
                   positions, slots, (float*)q_out, (float*)kcache, (float*)vcache, n, H, G, D, V, rot, eps, page_size, num_slots,
-                  write_kv, status, values_out, values_in, ld_values, value_mix);
+                  write_kv, status, values_out, values_in, ld_values, value_mix, unit_norm, temp_coef, temp_every);
     else if (dtype == GB_BF16)
         gb_launch(GB_PDL_ELEMENTWISE, qk_norm_rope_write_kernel<__nv_bfloat16>, dim3(n), block, 0, stream, qkv, ld, q_gain, k_gain,
                   inv_freq, positions, slots, (__nv_bfloat16*)q_out, (__nv_bfloat16*)kcache, (__nv_bfloat16*)vcache, n, H, G, D, V,
-                  rot, eps, page_size, num_slots, write_kv, status, values_out, values_in, ld_values, value_mix);
+                  rot, eps, page_size, num_slots, write_kv, status, values_out, values_in, ld_values, value_mix, unit_norm, temp_coef, temp_every);
     else
         GB_REQUIRE(false, "gb_qk_norm_rope_write: unsupported dtype %d", dtype);
     return gb_check_launch("gb_qk_norm_rope_write");

@@ -3,6 +3,7 @@
 //     s_j = q . k_j * scale - r1[head] * ln(1 + r2[head] * (p - j))                 (r1 == nullptr: no bias)
 //     w_j = exp(s_j - m) / (sum_j' exp(s_j' - m) + exp(sink[head] - m))             (sink == nullptr: a plain softmax)
 //     out = sum_j w_j v_j * sigmoid(gate[row, head])                                (gate == nullptr: no gate)
+// With gate_channels the gate has a logit per output channel: out[c] *= sigmoid(gate[row, head * V + c]).
 // The sink has no key and no value: it only takes its share of the weights. The row sees keys max(0, p - window + 1) .. p
 // (window 0: all of them). Query heads share key/value heads in groups; the key size (dim) and the value size (vdim) may
 // differ. Distances, logarithms, scores, weights, sums and the gate are float32. gate holds logits, float32 [n, ld_gate].
@@ -28,7 +29,7 @@ __global__ void __launch_bounds__(SK_WARPS * 32) sink_attention_rows_kernel(
     const int* __restrict__ block_tables, int max_pages, const int* __restrict__ row_seq, const int* __restrict__ positions,
     const float* __restrict__ r1, const float* __restrict__ r2, const float* __restrict__ sink, const float* __restrict__ gate,
     long long ld_gate, int n, int H, int G, int D, int V, int page_size, long long num_pages, float scale, int window,
-    int* __restrict__ status) {
+    int gate_channels, int* __restrict__ status) {
     __shared__ float qs[SK_WARPS][SA_MAX_DIM];
     gb_pdl_launch_dependents();
     gb_pdl_wait();
@@ -90,12 +91,13 @@ __global__ void __launch_bounds__(SK_WARPS * 32) sink_attention_rows_kernel(
         }
     }
     float f = l > 0.f ? 1.0f / l : 0.f;
-    if (gate) f *= sk_sigmoid(gate[(size_t)row * ld_gate + head]);
+    if (gate && !gate_channels) f *= sk_sigmoid(gate[(size_t)row * ld_gate + head]);
+    const float* gch = gate && gate_channels ? gate + (size_t)row * ld_gate + (size_t)head * V : nullptr;
     T* orow = out + ((size_t)row * H + head) * V;
 #pragma unroll
     for (int j = 0; j < SA_MAX_DIM / 32; ++j) {
         const int i = lane + 32 * j;
-        if (i < V) orow[i] = gb_from_float<T>(acc[j] * f);
+        if (i < V) orow[i] = gb_from_float<T>(gch ? acc[j] * f * sk_sigmoid(gch[i]) : acc[j] * f);
     }
 }
 
@@ -104,23 +106,25 @@ __global__ void __launch_bounds__(SK_WARPS * 32) sink_attention_rows_kernel(
     GB_REQUIRE(D > 0 && D <= SA_MAX_DIM && V > 0 && V <= SA_MAX_DIM, name ": head sizes %d / %d are outside 1..%d", D, V, SA_MAX_DIM);  \
     GB_REQUIRE(page_size > 0 && max_pages > 0 && window >= 0, name ": bad page geometry or window");                                    \
     GB_REQUIRE((r1 == nullptr) == (r2 == nullptr), name ": the distance bias needs both of its numbers per head");                      \
-    GB_REQUIRE(gate == nullptr || ld_gate >= H, name ": rows of gate logits are too short");
+    GB_REQUIRE(gate == nullptr || ld_gate >= (long long)H * (gate_channels ? V : 1), name ": rows of gate logits are too short");
 
 GB_EXPORT int gb_sink_attention_rows(const void* q, void* out, int dtype, const void* kcache, const void* vcache, const int* block_tables,
                                      int max_pages, const int* row_seq, const int* positions, const float* r1, const float* r2,
                                      const float* sink, const float* gate, long long ld_gate, int n, int H, int G, int D, int V,
-                                     int page_size, long long num_pages, float scale, int window, int* status, cudaStream_t stream) {
+                                     int page_size, long long num_pages, float scale, int window, int gate_channels, int* status,
+                                     cudaStream_t stream) {
     SK_COMMON_CHECKS("gb_sink_attention_rows")
     if (n == 0) return 0;
     const int blocks = gb_ceil_div((long long)n * H, SK_WARPS);
     if (dtype == GB_F32)
         gb_launch(GB_PDL_ATTENTION, sink_attention_rows_kernel<float>, dim3(blocks), dim3(SK_WARPS * 32), 0, stream, (const float*)q,
                   (float*)out, (const float*)kcache, (const float*)vcache, block_tables, max_pages, row_seq, positions, r1, r2, sink, gate,
-                  ld_gate, n, H, G, D, V, page_size, num_pages, scale, window, status);
+                  ld_gate, n, H, G, D, V, page_size, num_pages, scale, window, gate_channels, status);
     else if (dtype == GB_BF16)
         gb_launch(GB_PDL_ATTENTION, sink_attention_rows_kernel<__nv_bfloat16>, dim3(blocks), dim3(SK_WARPS * 32), 0, stream,
                   (const __nv_bfloat16*)q, (__nv_bfloat16*)out, (const __nv_bfloat16*)kcache, (const __nv_bfloat16*)vcache, block_tables,
-                  max_pages, row_seq, positions, r1, r2, sink, gate, ld_gate, n, H, G, D, V, page_size, num_pages, scale, window, status);
+                  max_pages, row_seq, positions, r1, r2, sink, gate, ld_gate, n, H, G, D, V, page_size, num_pages, scale, window, gate_channels,
+                  status);
     else
         GB_REQUIRE(false, "gb_sink_attention_rows: unsupported dtype %d", dtype);
     return gb_check_launch("gb_sink_attention_rows");
@@ -145,7 +149,7 @@ __global__ void __launch_bounds__(SKD_WARPS * 32) sink_attention_decode_kernel(
     const int* __restrict__ block_tables, int max_pages, const int* __restrict__ row_seq, const int* __restrict__ positions,
     const float* __restrict__ r1, const float* __restrict__ r2, const float* __restrict__ sink, const float* __restrict__ gate,
     long long ld_gate, int n, int H, int G, int D, int V, int page_size, long long num_pages, float scale, int window,
-    int* __restrict__ status) {
+    int gate_channels, int* __restrict__ status) {
     constexpr int PN = SadPiece<T>::N;          // channels in a 16-byte piece
     constexpr int KPI = 32 / LPK;               // keys that one warp-wide load fetches
     __shared__ __align__(16) float qs[R * SA_MAX_DIM];        // the R heads' queries, D apart
@@ -267,7 +271,7 @@ __global__ void __launch_bounds__(SKD_WARPS * 32) sink_attention_decode_kernel(
             den = fmaf(part_l[w][r], c, den);
         }
         float f = den > 0.f ? 1.0f / den : 0.f;
-        if (gate) f *= sk_sigmoid(gate[(size_t)row * ld_gate + head + r]);
+        if (gate) f *= sk_sigmoid(gate[(size_t)row * ld_gate + (gate_channels ? (size_t)head * V + i : (size_t)(head + r))]);
         out[((size_t)row * H + head) * V + i] = gb_from_float<T>(t * f);
     }
 }
@@ -281,7 +285,7 @@ template <typename T>
 static int skd_launch(const void* q, void* out, const void* kcache, const void* vcache, const int* block_tables, int max_pages,
                       const int* row_seq, const int* positions, const float* r1, const float* r2, const float* sink, const float* gate,
                       long long ld_gate, int n, int H, int G, int D, int V, int page_size, long long num_pages, float scale, int window,
-                      int* status, cudaStream_t stream) {
+                      int gate_channels, int* status, cudaStream_t stream) {
     const int lpk = V * (int)sizeof(T) / 16;
     // With enough (row, key/value head) pairs to fill the GPU, the query heads of a group go four at a time through one
     // block, which then reads the group's keys and values once for the four; with few rows every head gets its own block.
@@ -291,7 +295,7 @@ static int skd_launch(const void* q, void* out, const void* kcache, const void* 
     if (lpk == L && (together ? 4 : 1) == RR)                                                                                            \
         gb_launch(GB_PDL_ATTENTION, sink_attention_decode_kernel<T, L, RR>, dim3(n, H / RR), dim3(SKD_WARPS * 32), 0, stream,            \
                   (const T*)q, (T*)out, (const T*)kcache, (const T*)vcache, block_tables, max_pages, row_seq, positions, r1, r2, sink,   \
-                  gate, ld_gate, n, H, G, D, V, page_size, num_pages, scale, window, status);
+                  gate, ld_gate, n, H, G, D, V, page_size, num_pages, scale, window, gate_channels, status);
     SKD_CASE(4, 1) SKD_CASE(8, 1) SKD_CASE(16, 1) SKD_CASE(32, 1) SKD_CASE(4, 4) SKD_CASE(8, 4) SKD_CASE(16, 4)
 #undef SKD_CASE
     return gb_check_launch("gb_sink_attention_decode");
@@ -300,7 +304,7 @@ static int skd_launch(const void* q, void* out, const void* kcache, const void* 
 GB_EXPORT int gb_sink_attention_decode(const void* q, void* out, int dtype, const void* kcache, const void* vcache,
                                        const int* block_tables, int max_pages, const int* row_seq, const int* positions, const float* r1,
                                        const float* r2, const float* sink, const float* gate, long long ld_gate, int n, int H, int G,
-                                       int D, int V, int page_size, long long num_pages, float scale, int window, int* status,
+                                       int D, int V, int page_size, long long num_pages, float scale, int window, int gate_channels, int* status,
                                        cudaStream_t stream) {
     SK_COMMON_CHECKS("gb_sink_attention_decode")
     GB_REQUIRE(dtype == GB_F32 || dtype == GB_BF16, "gb_sink_attention_decode: unsupported dtype %d", dtype);
@@ -310,9 +314,9 @@ GB_EXPORT int gb_sink_attention_decode(const void* q, void* out, int dtype, cons
     if (n == 0) return 0;
     if (dtype == GB_F32)
         return skd_launch<float>(q, out, kcache, vcache, block_tables, max_pages, row_seq, positions, r1, r2, sink, gate, ld_gate, n, H, G,
-                                 D, V, page_size, num_pages, scale, window, status, stream);
+                                 D, V, page_size, num_pages, scale, window, gate_channels, status, stream);
     return skd_launch<__nv_bfloat16>(q, out, kcache, vcache, block_tables, max_pages, row_seq, positions, r1, r2, sink, gate, ld_gate, n,
-                                     H, G, D, V, page_size, num_pages, scale, window, status, stream);
+                                     H, G, D, V, page_size, num_pages, scale, window, gate_channels, status, stream);
 }
 
 // ----------------------------------------------------------------------------------------------
@@ -322,7 +326,8 @@ GB_EXPORT int gb_sink_attention_decode(const void* q, void* out, int dtype, cons
 // m16n8k16; in float32 and in the base-2 domain t = S * (scale * log2 e) - r1 * log2(1 + r2 * distance), the window and the
 // causal edge per element, a running maximum per row that starts at the sink's logit, weights 2^(t - m) rounded to
 // bfloat16 as the A operand of O += P V (float32 sums), O rescaled when the maximum moves. At the end the sink's share
-// joins the denominator and the gate multiplies the row. Head sizes 32, 64 or 128 for keys and for values.
+// joins the denominator and the gate multiplies the row. Head sizes 32, 64 or 128 for keys and for values, and 48, 80 or 96
+// for both.
 // ----------------------------------------------------------------------------------------------
 constexpr int SKT_BM = 64, SKT_BN = 64;
 constexpr float SK_LOG2E = 1.4426950408889634f;
@@ -333,7 +338,7 @@ __global__ void __launch_bounds__(128) sink_attention_tiles_kernel(
     const __nv_bfloat16* __restrict__ vcache, const int* __restrict__ block_tables, int max_pages, const int* __restrict__ seq_first_row,
     const int* __restrict__ seq_start_pos, const float* __restrict__ r1, const float* __restrict__ r2, const float* __restrict__ sink,
     const float* __restrict__ gate, long long ld_gate, int num_seqs, int tiles_per_seq, int H, int G, int page_size, long long num_pages,
-    float scale, int window, int* __restrict__ status) {
+    float scale, int window, int gate_channels, int* __restrict__ status) {
     constexpr int LDK = D + 8, LDV = V + 8;          // rows padded by 16 bytes: ldmatrix meets no bank twice
     extern __shared__ __align__(16) unsigned char skt_smem[];
     __nv_bfloat16* sq = reinterpret_cast<__nv_bfloat16*>(skt_smem);             // [64][LDK]
@@ -519,37 +524,44 @@ __global__ void __launch_bounds__(128) sink_attention_tiles_kernel(
         const int r = warp * 16 + (lane >> 2) + half * 8;
         if (r >= rows) continue;
         float f = den > 0.f ? 1.0f / den : 0.f;
-        if (gate) f *= sk_sigmoid(gate[(size_t)(row0 + r) * ld_gate + head]);
+        if (gate && !gate_channels) f *= sk_sigmoid(gate[(size_t)(row0 + r) * ld_gate + head]);
         __nv_bfloat16* dst = out + ((size_t)(row0 + r) * H + head) * V;
 #pragma unroll
-        for (int j = 0; j < V / 8; ++j)
-            *reinterpret_cast<__nv_bfloat162*>(dst + j * 8 + (lane & 3) * 2) = __floats2bfloat162_rn(o[j][half * 2] * f, o[j][half * 2 + 1] * f);
+        for (int j = 0; j < V / 8; ++j) {
+            float a = o[j][half * 2] * f, b = o[j][half * 2 + 1] * f;
+            if (gate && gate_channels) {
+                const float* gch = gate + (size_t)(row0 + r) * ld_gate + (size_t)head * V + j * 8 + (lane & 3) * 2;
+                a *= sk_sigmoid(gch[0]);
+                b *= sk_sigmoid(gch[1]);
+            }
+            *reinterpret_cast<__nv_bfloat162*>(dst + j * 8 + (lane & 3) * 2) = __floats2bfloat162_rn(a, b);
+        }
     }
 }
 
 GB_EXPORT int gb_sink_attention_tiles_supported(int D, int V) {
-    return (D == 32 || D == 64 || D == 128) && (V == 32 || V == 64 || V == 128) ? 1 : 0;
+    return ((D == 32 || D == 64 || D == 128) && (V == 32 || V == 64 || V == 128)) || (D == V && (D == 48 || D == 80 || D == 96)) ? 1 : 0;
 }
 
 template <int D, int V>
 static int skt_launch(const void* q, void* out, const void* kcache, const void* vcache, const int* block_tables, int max_pages,
                       const int* seq_first_row, const int* seq_start_pos, const float* r1, const float* r2, const float* sink,
                       const float* gate, long long ld_gate, int num_seqs, int tiles_per_seq, int H, int G, int page_size,
-                      long long num_pages, float scale, int window, int* status, cudaStream_t stream) {
+                      long long num_pages, float scale, int window, int gate_channels, int* status, cudaStream_t stream) {
     const size_t smem = ((size_t)3 * SKT_BM * (D + 8) + (size_t)2 * SKT_BN * (V + 8)) * 2;
     cudaFuncSetAttribute(sink_attention_tiles_kernel<D, V>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     gb_launch(GB_PDL_ATTENTION, sink_attention_tiles_kernel<D, V>, dim3(num_seqs * tiles_per_seq, H), dim3(128), smem, stream,
               (const __nv_bfloat16*)q, (__nv_bfloat16*)out, (const __nv_bfloat16*)kcache, (const __nv_bfloat16*)vcache, block_tables,
               max_pages, seq_first_row, seq_start_pos, r1, r2, sink, gate, ld_gate, num_seqs, tiles_per_seq, H, G, page_size, num_pages,
-              scale, window, status);
+              scale, window, gate_channels, status);
     return gb_check_launch("gb_sink_attention_tiles");
 }
 
 GB_EXPORT int gb_sink_attention_tiles(const void* q, void* out, const void* kcache, const void* vcache, const int* block_tables,
                                       int max_pages, const int* seq_first_row, const int* seq_start_pos, const float* r1, const float* r2,
                                       const float* sink, const float* gate, long long ld_gate, int num_seqs, int max_rows_per_seq, int H,
-                                      int G, int D, int V, int page_size, long long num_pages, float scale, int window, int* status,
-                                      cudaStream_t stream) {
+                                      int G, int D, int V, int page_size, long long num_pages, float scale, int window, int gate_channels,
+                                      int* status, cudaStream_t stream) {
     const int n = num_seqs;
     SK_COMMON_CHECKS("gb_sink_attention_tiles")
     GB_REQUIRE(gb_sink_attention_tiles_supported(D, V), "gb_sink_attention_tiles: head sizes %d / %d are not built", D, V);
@@ -559,9 +571,9 @@ GB_EXPORT int gb_sink_attention_tiles(const void* q, void* out, const void* kcac
 #define SKT_CASE(DD, VV)                                                                                                              \
     if (D == DD && V == VV)                                                                                                           \
         return skt_launch<DD, VV>(q, out, kcache, vcache, block_tables, max_pages, seq_first_row, seq_start_pos, r1, r2, sink, gate,   \
-                                  ld_gate, num_seqs, tiles, H, G, page_size, num_pages, scale, window, status, stream);
+                                  ld_gate, num_seqs, tiles, H, G, page_size, num_pages, scale, window, gate_channels, status, stream);
     SKT_CASE(32, 32) SKT_CASE(32, 64) SKT_CASE(32, 128) SKT_CASE(64, 32) SKT_CASE(64, 64) SKT_CASE(64, 128) SKT_CASE(128, 32)
-    SKT_CASE(128, 64) SKT_CASE(128, 128)
+    SKT_CASE(128, 64) SKT_CASE(128, 128) SKT_CASE(48, 48) SKT_CASE(80, 80) SKT_CASE(96, 96)
 #undef SKT_CASE
     GB_REQUIRE(false, "gb_sink_attention_tiles: head sizes %d / %d are not built", D, V);
 }

@@ -139,6 +139,9 @@ class StepContext:
         # ... and takes a branch output that is a weighted sum of rows as its parts (kernels.WeightedRows), if the part offers
         self.accepts_weighted_rows = False
         self.weighted_rows = None
+        # ... or one that is a sum of two normed rows (kernels.NormedPair)
+        self.accepts_normed_pair = False
+        self.normed_pair = None
 
     def scratch(self, name: str, shape, dtype: Optional[torch.dtype] = None, grow: bool = False) -> torch.Tensor:
         return (self._grow if grow else self._scratch).get(name, shape, dtype, grow)

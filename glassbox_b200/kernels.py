@@ -22,6 +22,8 @@ _DT = {torch.float32: F32, torch.bfloat16: BF16}
 GATED_EPILOGUES = ("silu", "gelu_tanh")
 #: how the unit epilogues are told to form gelu_tanh(gate) * up instead of the clamped unit: (limit, slope)
 GELU_UNIT = (3.0e38, -1.0)
+#: the same for silu(gate) * up, where a kernel takes a unit by these two numbers (the routed experts)
+SILU_UNIT = (3.0e38, 0.0)
 
 STATUS_BITS = {1: "a token id outside the vocabulary", 2: "a cache slot or page id outside the pool",
                4: "a position outside the rotary table or beyond a block table", 8: "a bounded wait inside a kernel gave up"}
@@ -56,7 +58,7 @@ _SIGNATURES = {
     "gb_attention_decode_mma_pdl": [_P, _LL, _P, _LL, _P, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _LL, _F, _I, _I, _P, _P,
                                     _P, _P, _I, _I, _I, _P],
     "gb_attention_decode_mma_sink": [_P, _LL, _P, _LL, _P, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _LL, _F, _I, _I, _P, _P,
-                                     _P, _P, _I, _I, _I, _P, _P, _P, _P, _LL, _P],
+                                     _P, _P, _I, _I, _I, _P, _P, _P, _P, _LL, _I, _P],
     "gb_attention_decode_mma": [_P, _LL, _P, _LL, _P, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _LL, _F, _I, _I, _P, _P, _P,
                                 _P, _P],
     "gb_attention_decode_mma_supported": [_I, _I, _I],
@@ -69,7 +71,7 @@ _SIGNATURES = {
     "gb_gemm_tcgen05_qkv_supported": [_I],
     "gb_attention_prefill_tc": [_P, _LL, _I, _P, _LL, _P, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _I, _LL, _F, _I, _P, _P],
     "gb_attention_prefill_tc_sink": [_P, _LL, _I, _P, _LL, _P, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _I, _LL, _F, _I, _P, _P, _P,
-                                     _P, _P, _LL, _P],
+                                     _P, _P, _LL, _I, _P],
     "gb_attention_prefill_tc_supported": [_I, _I, _I, _I],
     "gb_gemm_tcgen05": [_P, _P, _P, _I, _I, _I, _I, _LL, _LL, _LL, _P, _P, _P, _P, _LL, _P, _P, _I, _F],
     "gb_gemm_tcgen05_column_tiles": [_I, _I, _I],
@@ -100,7 +102,7 @@ _SIGNATURES = {
                                 _P, _P],
     "gb_head_linear_supported": [_P, _LL, _LL, _P, _P, _LL, _LL, _I, _I],
     "gb_head_linear": [_P, _LL, _LL, _P, _P, _LL, _LL, _I, _I, _I, _I, _P],
-    "gb_embed_positions": [_P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _P, _P],
+    "gb_embed_positions": [_P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _F, _P, _P],
     "gb_residual_conv": [_P, _I, _P, _I, _P, _P, _LL, _LL, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _P, _P],
     "gb_gelu_glu": [_P, _I, _LL, _P, _I, _I, _I, _P],
     "gb_scaled_sum": [_P, _P, _F, _F, _P, _LL, _I, _P],
@@ -121,25 +123,33 @@ _SIGNATURES = {
     "gb_streams_broadcast": [_P, _P, _I, _I, _I, _P],
     "gb_streams_step": [_P, _I, _I, _P, _LL, _P, _P, _I, _P, _LL, _P, _P, _P, _P, _P, _P, _F, _P, _I, _P, _P, _P, _I, _I, _P],
     "gb_qk_norm_rope_write": [_P, _LL, _P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _F, _I, _LL, _I, _P, _P, _P, _LL,
-                              _P, _P],
-    "gb_sink_attention_rows": [_P, _P, _I, _P, _P, _P, _I, _P, _P, _P, _P, _P, _P, _LL, _I, _I, _I, _I, _I, _I, _LL, _F, _I, _P, _P],
-    "gb_sink_attention_decode": [_P, _P, _I, _P, _P, _P, _I, _P, _P, _P, _P, _P, _P, _LL, _I, _I, _I, _I, _I, _I, _LL, _F, _I, _P, _P],
+                              _P, _I, _F, _F, _P],
+    "gb_sink_attention_rows": [_P, _P, _I, _P, _P, _P, _I, _P, _P, _P, _P, _P, _P, _LL, _I, _I, _I, _I, _I, _I, _LL, _F, _I, _I, _P, _P],
+    "gb_sink_attention_decode": [_P, _P, _I, _P, _P, _P, _I, _P, _P, _P, _P, _P, _P, _LL, _I, _I, _I, _I, _I, _I, _LL, _F, _I, _I, _P, _P],
     "gb_sink_attention_decode_supported": [_I],
     "gb_sink_attention_tiles_supported": [_I, _I],
-    "gb_sink_attention_tiles": [_P, _P, _P, _P, _P, _I, _P, _P, _P, _P, _P, _P, _LL, _I, _I, _I, _I, _I, _I, _I, _LL, _F, _I, _P, _P],
+    "gb_sink_attention_tiles": [_P, _P, _P, _P, _P, _I, _P, _P, _P, _P, _P, _P, _LL, _I, _I, _I, _I, _I, _I, _I, _LL, _F, _I, _I, _P, _P],
     "gb_sigmoid_attention_rows": [_P, _P, _I, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _LL, _F, _I, _P, _P],
     "gb_sigmoid_attention_decode": [_P, _P, _I, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _LL, _F, _I, _P, _P],
     "gb_sigmoid_attention_decode_supported": [_I],
     "gb_sigmoid_attention_tiles_supported": [_I, _I],
     "gb_sigmoid_attention_tiles": [_P, _P, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _LL, _F, _I, _P, _P],
     "gb_mingru_scan": [_P, _LL, _P, _P, _P, _LL, _LL, _P, _LL, _I, _P, _P, _P, _I, _I, _I, _I, _I, _P, _P],
-    "gb_moe_route": [_P, _I, _I, _P, _P, _P, _P, _I, _I, _I, _I, _I, _F, _P, _P, _P, _P, _I, _P],
+    "gb_moe_route": [_P, _I, _I, _P, _P, _P, _P, _I, _I, _I, _I, _I, _F, _P, _P, _P, _P, _I, _I, _F, _P],
     "gb_moe_expert_rows": [_P, _I, _I, _P, _P, _I, _P, _P, _I, _I, _I, _P, _P],
     "gb_moe_expert_halves": [_P, _I, _I, _P, _P, _I, _P, _P, _I, _I, _I, _P, _P, _I, _F, _F, _P],
     "gb_moe_sort": [_P, _P, _I, _I, _I, _P, _P, _P, _P],
     "gb_moe_grouped_supported": [_I, _I],
     "gb_moe_grouped_gemm": [_P, _LL, _P, _I, _I, _P, _P, _P, _I, _I, _I, _P, _LL, _I, _I, _F, _F, _P],
     "gb_moe_combine": [_P, _P, _I, _P, _LL, _P, _P, _P, _LL, _I, _I, _I, _P],
+    "gb_post_norm": [_P, _LL, _P, _F, _F, _I, _P, _P, _P, _P, _F, _F, _F, _P, _P, _I, _P, _P, _P, _I, _P, _I, _I, _P],
+    "gb_gate_group_norm": [_P, _P, _LL, _P, _P, _I, _P, _I, _I, _I, _F, _P],
+    "gb_ring_conv": [_P, _LL, _P, _P, _P, _I, _LL, _P, _LL, _LL, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P, _P],
+    "gb_ssd_decode": [_P, _LL, _P, _LL, _P, _P, _P, _P, _P, _P, _LL, _LL, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P, _P],
+    "gb_ssd_walk": [_P, _LL, _P, _LL, _P, _P, _P, _P, _LL, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P, _P],
+    "gb_ssd_chunk_rows": [],
+    "gb_ssd_chunks_supported": [_I, _I],
+    "gb_ssd_chunks": [_P, _LL, _P, _LL, _P, _P, _P, _P, _LL, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _P, _P, _P, _P],
     "gb_program_op_bytes": [],
     "gb_program_max_rows": [],
 }
@@ -375,14 +385,14 @@ def embed(table: torch.Tensor, tokens: torch.Tensor, x: torch.Tensor, status: to
 
 
 def embed_positions(table: torch.Tensor, pos_table: torch.Tensor, tokens: torch.Tensor, positions: torch.Tensor, x: torch.Tensor,
-                    status: torch.Tensor) -> None:
-    """x[i, :] = table[tokens[i], :] + pos_table[positions[i], :], summed in float32; padding rows (position < 0) are cleared."""
+                    status: torch.Tensor, scale: float = 1.0) -> None:
+    """x[i, :] = table[tokens[i], :] * scale + pos_table[positions[i], :], in float32; padding rows (position < 0) are cleared."""
     _cuda(table, pos_table, tokens, positions, x, status)
     n, d = x.shape
     assert table.dtype == pos_table.dtype and table.shape[1] == pos_table.shape[1] == d and x.dtype == torch.float32
     assert table.is_contiguous() and pos_table.is_contiguous() and x.is_contiguous() and tokens.shape[0] >= n and positions.shape[0] >= n
     _call("gb_embed_positions", _ptr(table), _ptr(pos_table), _dt(table), _ptr(tokens), _ptr(positions), _ptr(x), n, d, table.shape[0],
-          pos_table.shape[0], _ptr(status), _stream())
+          pos_table.shape[0], float(scale), _ptr(status), _stream())
 
 
 def rmsnorm(x: torch.Tensor, gain: torch.Tensor, out: torch.Tensor, eps: float,
@@ -826,10 +836,11 @@ def attention_decode_mma(q: torch.Tensor, out: torch.Tensor, kcache: torch.Tenso
             prog.flush()
         r1, r2, sink, gate = sink_terms
         _cuda(r1, r2, sink, gate)
+        terms, by_channel = _sink_args(r1, r2, sink, gate, nh, hd)
         _call("gb_attention_decode_mma_sink", _ptr(q), q.stride(0), _ptr(out), out.stride(0), _ptr(kcache), _ptr(vcache),
               _ptr(block_tables), block_tables.shape[1], _ptr(row_seq), _ptr(positions), n, nh, nkv, hd, page_size,
               kcache.shape[0], float(scale), int(window or 0), int(splits), _ptr(part_acc), _ptr(part_ml), _ptr(counters),
-              _ptr(status), 1 if USE_PDL else 0, int(block_keys), int(warps), *_sink_args(r1, r2, sink, gate, nh), _stream())
+              _ptr(status), 1 if USE_PDL else 0, int(block_keys), int(warps), *terms, by_channel, _stream())
         return
     if prog is not None and prog.takes_rows(n):
         if not prog.takes_attention(hd, block_keys):
@@ -875,10 +886,11 @@ def attention_prefill_tc(q: torch.Tensor, out: torch.Tensor, kcache: torch.Tenso
     if sink_terms is not None:
         r1, r2, sink, gate = sink_terms
         _cuda(r1, r2, sink, gate)
+        terms, by_channel = _sink_args(r1, r2, sink, gate, nh, hd)
         _call("gb_attention_prefill_tc_sink", _ptr(q), q.stride(0), q.shape[0], _ptr(out), out.stride(0), _ptr(kcache),
               _ptr(vcache), _ptr(block_tables), block_tables.shape[1], _ptr(seq_first_row), _ptr(seq_start_pos), S,
               int(max_rows_per_seq), nh, nkv, hd, page_size, kcache.shape[0], float(scale), int(window or 0), _ptr(status),
-              *_sink_args(r1, r2, sink, gate, nh), _stream())
+              *terms, by_channel, _stream())
         return
     _call("gb_attention_prefill_tc", _ptr(q), q.stride(0), q.shape[0], _ptr(out), out.stride(0), _ptr(kcache),
           _ptr(vcache), _ptr(block_tables), block_tables.shape[1], _ptr(seq_first_row), _ptr(seq_start_pos), S,
@@ -1124,6 +1136,153 @@ def latent_attention_mma(q: torch.Tensor, out: torch.Tensor, cache: torch.Tensor
           block_tables.shape[1], _ptr(seq_first_row), _ptr(seq_start_pos), _ptr(positions), _ptr(sink), n, S,
           int(max_rows_per_seq), heads, c, r, page_size, num_pages, float(scale), int(window) if window else 0,
           1 if decode else 0, int(splits), _ptr(status), _stream())
+
+
+class NormedPair:
+    """A branch output that exists only as its parts: a_scale * rms(a[r], gain_a) + b_scale * rms(b[r], gain_b), two branches that
+    share an input and are each normed over the row before they join. ``post_norm`` takes it in the place of a stored y."""
+    __slots__ = ("a", "b", "gain_a", "gain_b", "a_scale", "b_scale", "eps")
+
+    def __init__(self, a, b, gain_a, gain_b, a_scale: float, b_scale: float, eps: float):
+        self.a, self.b, self.gain_a, self.gain_b = a, b, gain_a, gain_b
+        self.a_scale, self.b_scale, self.eps = float(a_scale), float(b_scale), float(eps)
+
+
+def post_norm(x: torch.Tensor, gain: torch.Tensor, alpha: float, eps: float, branch, positions: Optional[torch.Tensor] = None,
+              copy: Optional[torch.Tensor] = None) -> None:
+    """x[r, :] <- gain * t / sqrt(mean(t^2) + eps) with t = alpha * x[r, :] + y[r, :]; everything float32. ``branch`` is y itself
+    (float32 [n, d], contiguous), a ``WeightedRows`` or a ``NormedPair``, whose y is formed on the way. ``copy`` ([n, d], float32
+    or bfloat16, contiguous) receives the new x; rows whose position is below zero are left alone."""
+    n, d = x.shape
+    _cuda(x, gain, positions, copy)
+    assert x.dtype == gain.dtype == torch.float32 and x.stride(1) == 1 and gain.numel() == d and gain.is_contiguous()
+    assert copy is None or (copy.shape == (n, d) and copy.is_contiguous())
+    mode, y, b, ga, gb, sa, sb, pe, pair, weight, top, shared, gate = 0, None, None, None, None, 0.0, 0.0, 0.0, None, None, 0, None, None
+    if isinstance(branch, WeightedRows):
+        mode, pair, weight, shared, gate = 1, branch.pair, branch.weight, branch.shared, branch.gate
+        top = weight.shape[1]
+        _cuda(pair, weight, shared, gate)
+        assert pair.dtype == weight.dtype == torch.float32 and pair.shape == (n, top * d) and pair.is_contiguous() and weight.is_contiguous()
+        assert shared is None or (shared.dtype == torch.float32 and shared.shape == (n, d) and shared.is_contiguous())
+        assert gate is None or (gate.dtype == torch.float32 and gate.numel() >= n)
+    elif isinstance(branch, NormedPair):
+        mode, y, b, ga, gb = 2, branch.a, branch.b, branch.gain_a, branch.gain_b
+        sa, sb, pe = branch.a_scale, branch.b_scale, branch.eps
+        _cuda(y, b, ga, gb)
+        for t in (y, b):
+            assert t.dtype == torch.float32 and t.shape == (n, d) and t.is_contiguous()
+        for t in (ga, gb):
+            assert t.dtype == torch.float32 and t.numel() == d and t.is_contiguous()
+    else:
+        y = branch
+        _cuda(y)
+        assert y.dtype == torch.float32 and y.shape == (n, d) and y.is_contiguous()
+    _call("gb_post_norm", _ptr(x), x.stride(0), _ptr(gain), float(alpha), float(eps), mode, _ptr(y), _ptr(b), _ptr(ga), _ptr(gb), sa, sb, pe,
+          _ptr(pair), _ptr(weight), top, _ptr(shared), _ptr(gate), _ptr(copy), _dt(copy) if copy is not None else F32, _ptr(positions), n, d,
+          _stream())
+
+
+def gate_group_norm(y: torch.Tensor, z: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, groups: int, eps: float,
+                    positions: Optional[torch.Tensor] = None) -> None:
+    """u = y * silu(z), each of ``groups`` equal parts of a row divided by its own root mean square (eps inside the root), times
+    ``weight`` per channel. y, z, weight float32 (z may be a column slice), out in any activation dtype."""
+    _cuda(y, z, weight, out, positions)
+    n, width = y.shape
+    assert y.dtype == z.dtype == weight.dtype == torch.float32 and y.is_contiguous() and out.is_contiguous() and width % groups == 0
+    assert z.shape == (n, width) and z.stride(1) == 1 and out.shape == (n, width) and weight.numel() == width and weight.is_contiguous()
+    _call("gb_gate_group_norm", _ptr(y), _ptr(z), z.stride(0), _ptr(weight), _ptr(out), _dt(out), _ptr(positions), n, groups,
+          width // groups, float(eps), _stream())
+
+
+# ------------------------------------------------------------------------------------- state-space mixers
+def ring_conv(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], y: torch.Tensor, state: torch.Tensor, state_off: int,
+              row_seq: torch.Tensor, positions: torch.Tensor, seq_first_row: torch.Tensor, seq_start_pos: torch.Tensor,
+              seq_slots: torch.Tensor, update_state: bool, status: torch.Tensor, first_row: int = 0, first_seq: int = 0) -> None:
+    """y[t, c] = silu(bias[c] + sum_j w[c, j] * x[t - (taps - 1) + j, c]) along each request's rows (x, w, bias float32, y in any
+    activation dtype). Inputs from before the step come from a ring of ``taps`` rows at ``state_off`` of the request's slot of
+    ``state`` [slots, numbers]: the input of position p lies in row p mod taps; with ``update_state`` the step's last inputs go
+    there afterwards. Rows before ``first_row`` and requests before ``first_seq`` are left alone."""
+    _cuda(x, w, bias, y, state, row_seq, positions, seq_first_row, seq_start_pos, seq_slots, status)
+    n, C = x.shape
+    taps = w.shape[1]
+    assert x.dtype == w.dtype == state.dtype == torch.float32 and x.stride(1) == 1 and y.stride(1) == 1 and y.shape == (n, C)
+    assert w.shape == (C, taps) and w.is_contiguous() and (bias is None or (bias.dtype == torch.float32 and bias.numel() == C))
+    assert state.dim() == 2 and state.is_contiguous() and state_off + taps * C <= state.shape[1]
+    _call("gb_ring_conv", _ptr(x), x.stride(0), _ptr(w), _ptr(bias), _ptr(y), _dt(y), y.stride(0), _ptr(state), state.stride(0), state_off,
+          _ptr(row_seq), _ptr(positions), _ptr(seq_first_row), _ptr(seq_start_pos), _ptr(seq_slots), first_row, n, first_seq,
+          seq_start_pos.shape[0], C, taps, state.shape[0], 1 if update_state else 0, _ptr(status), _stream())
+    global launch_count
+    launch_count += 1 if update_state else 0
+
+
+def _ssd_check(xbc, dt_raw, dt_bias, a_log, skip, state, y, heads, groups, n_state, vdim):
+    n = xbc.shape[0]
+    assert xbc.shape[1] == heads * vdim + 2 * groups * n_state and xbc.stride(1) == 1
+    assert dt_raw.dtype == torch.float32 and dt_raw.shape == (n, heads) and dt_raw.stride(1) == 1
+    for t in (dt_bias, a_log, skip):
+        assert t.dtype == torch.float32 and t.numel() == heads and t.is_contiguous()
+    assert state.dtype == torch.float32 and state.dim() == 2 and state.is_contiguous() and state.shape[1] >= heads * n_state * vdim
+    assert y.dtype == torch.float32 and y.shape == (n, heads * vdim) and y.is_contiguous()
+
+
+def ssd_decode(xbc: torch.Tensor, dt_raw: torch.Tensor, conv_w: torch.Tensor, conv_b: torch.Tensor, dt_bias: torch.Tensor,
+               a_log: torch.Tensor, skip: torch.Tensor, state: torch.Tensor, conv_off: int, y: torch.Tensor, seq_first_row: torch.Tensor,
+               seq_start_pos: torch.Tensor, seq_slots: torch.Tensor, heads: int, groups: int, n_state: int, vdim: int,
+               write_state: bool, status: torch.Tensor) -> None:
+    """One token per request (requests 0 .. len(seq_start_pos) - 1): the convolution of x | B | C (``xbc`` float32 [n, channels], the
+    projection's sums) over the ring at ``conv_off`` of the request's slot, dt = softplus(dt_raw + dt_bias), S <- exp(-exp(a_log)
+    dt) S + dt B x^T, y = S^T C + skip x, all float32; S [heads, n_state, vdim] lies at the start of the slot and is read and
+    written once, the ring receives the token's inputs."""
+    _cuda(xbc, dt_raw, conv_w, conv_b, dt_bias, a_log, skip, state, y, seq_first_row, seq_start_pos, seq_slots, status)
+    _ssd_check(xbc, dt_raw, dt_bias, a_log, skip, state, y, heads, groups, n_state, vdim)
+    C, taps = conv_w.shape
+    assert xbc.dtype == conv_w.dtype == conv_b.dtype == torch.float32 and C == xbc.shape[1] == conv_b.numel() and conv_w.is_contiguous()
+    assert conv_off + taps * C <= state.shape[1]
+    _call("gb_ssd_decode", _ptr(xbc), xbc.stride(0), _ptr(dt_raw), dt_raw.stride(0), _ptr(conv_w), _ptr(conv_b), _ptr(dt_bias), _ptr(a_log),
+          _ptr(skip), _ptr(state), state.stride(0), conv_off, _ptr(y), _ptr(seq_first_row), _ptr(seq_start_pos), _ptr(seq_slots),
+          seq_start_pos.shape[0], heads, groups, n_state, vdim, taps, state.shape[0], 1 if write_state else 0, _ptr(status), _stream())
+
+
+def ssd_walk(xbc: torch.Tensor, dt_raw: torch.Tensor, dt_bias: torch.Tensor, a_log: torch.Tensor, skip: torch.Tensor, state: torch.Tensor,
+             y: torch.Tensor, seq_first_row: torch.Tensor, seq_start_pos: torch.Tensor, seq_slots: torch.Tensor, heads: int, groups: int,
+             n_state: int, vdim: int, write_state: bool, status: torch.Tensor) -> None:
+    """The recurrence of ``ssd_decode`` token by token along each request's rows; ``xbc`` float32 after its convolution."""
+    _cuda(xbc, dt_raw, dt_bias, a_log, skip, state, y, seq_first_row, seq_start_pos, seq_slots, status)
+    _ssd_check(xbc, dt_raw, dt_bias, a_log, skip, state, y, heads, groups, n_state, vdim)
+    assert xbc.dtype == torch.float32
+    _call("gb_ssd_walk", _ptr(xbc), xbc.stride(0), _ptr(dt_raw), dt_raw.stride(0), _ptr(dt_bias), _ptr(a_log), _ptr(skip), _ptr(state),
+          state.stride(0), _ptr(y), _ptr(seq_first_row), _ptr(seq_start_pos), _ptr(seq_slots), seq_start_pos.shape[0], heads, groups,
+          n_state, vdim, state.shape[0], 1 if write_state else 0, _ptr(status), _stream())
+
+
+def ssd_chunks_supported(dtype: torch.dtype, n_state: int, vdim: int) -> bool:
+    return dtype == torch.bfloat16 and bool(lib().gb_ssd_chunks_supported(n_state, vdim))
+
+
+def ssd_chunks_needed(n: int, num_seqs: int) -> int:
+    """How many chunks ``ssd_chunks`` may need for a step of ``n`` rows in ``num_seqs`` sequences."""
+    return n // lib().gb_ssd_chunk_rows() + num_seqs
+
+
+def ssd_chunks(xbc: torch.Tensor, dt_raw: torch.Tensor, dt_bias: torch.Tensor, a_log: torch.Tensor, skip: torch.Tensor,
+               state: torch.Tensor, y: torch.Tensor, seq_first_row: torch.Tensor, seq_start_pos: torch.Tensor, seq_slots: torch.Tensor,
+               max_rows_per_seq: int, heads: int, groups: int, n_state: int, vdim: int, write_state: bool, status: torch.Tensor,
+               chunk_state: torch.Tensor, chunk_decay: torch.Tensor) -> None:
+    """``ssd_walk`` in chunks that run side by side on the tensor cores; ``xbc`` bfloat16 after its convolution. The chunks' own
+    sums are chained afterwards (float32), then every chunk's read-outs are formed. ``chunk_state`` float32 [chunks, heads *
+    n_state * vdim] and ``chunk_decay`` float32 [chunks, heads] are scratch, chunks = ``ssd_chunks_needed``."""
+    _cuda(xbc, dt_raw, dt_bias, a_log, skip, state, y, seq_first_row, seq_start_pos, seq_slots, status, chunk_state, chunk_decay)
+    _ssd_check(xbc, dt_raw, dt_bias, a_log, skip, state, y, heads, groups, n_state, vdim)
+    n, S, chunks = xbc.shape[0], seq_start_pos.shape[0], chunk_state.shape[0]
+    assert xbc.dtype == torch.bfloat16 and chunk_state.dtype == chunk_decay.dtype == torch.float32
+    assert chunk_state.shape == (chunks, heads * n_state * vdim) and chunk_state.is_contiguous() and chunk_decay.is_contiguous()
+    assert chunk_decay.numel() >= chunks * heads and chunks >= ssd_chunks_needed(n, S)
+    _call("gb_ssd_chunks", _ptr(xbc), xbc.stride(0), _ptr(dt_raw), dt_raw.stride(0), _ptr(dt_bias), _ptr(a_log), _ptr(skip), _ptr(state),
+          state.stride(0), _ptr(y), _ptr(seq_first_row), _ptr(seq_start_pos), _ptr(seq_slots), S, n, max(int(max_rows_per_seq), 1), heads,
+          groups, n_state, vdim, state.shape[0], 1 if write_state else 0, chunks, _ptr(chunk_state), _ptr(chunk_decay), _ptr(status),
+          _stream())
+    global launch_count
+    launch_count += 2
 
 
 # ------------------------------------------------------------------------------------- recurrent state mixers
@@ -1412,12 +1571,14 @@ def qk_norm_rope_write(qkv: torch.Tensor, q_gain: Optional[torch.Tensor], k_gain
                        positions: torch.Tensor, slots: torch.Tensor, q_out: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor,
                        heads: int, kv_heads: int, dim: int, vdim: int, rot: int, eps: float, page_size: int, write_kv: bool,
                        status: torch.Tensor, values_out: Optional[torch.Tensor] = None, values_in: Optional[torch.Tensor] = None,
-                       value_mix: Optional[torch.Tensor] = None) -> None:
+                       value_mix: Optional[torch.Tensor] = None, unit_norm: bool = False, q_temp=None) -> None:
     """From the float32 sums of the stacked projection q | k | v: RMS norm of every query and key head over ``dim`` (one
     gain for the query heads, one for the key heads; None: no norm), rotation of the first ``rot`` channels in neighbouring pairs by
     float32(position) * inv_freq[i], q into ``q_out`` [n, heads * dim], k and v into the paged cache at each row's slot.
     With ``values_in`` (float32 [n, kv_heads * vdim]) a row's v becomes (1 - value_mix) v + value_mix values_in[row] first
-    (``value_mix`` one float32 number on the device); ``values_out`` (same shape) receives the row's v as it is stored."""
+    (``value_mix`` one float32 number on the device); ``values_out`` (same shape) receives the row's v as it is stored.
+    ``unit_norm``: heads without a gain are normed all the same; ``q_temp`` = (coef, every): the query at position p is
+    multiplied by 1 + coef * ln(floor((p + 1) / every) + 1)."""
     _cuda(qkv, q_gain, k_gain, inv_freq, positions, slots, q_out, kcache, vcache, status, values_out, values_in, value_mix)
     for t in (values_out, values_in):
         assert t is None or (t.dtype == torch.float32 and t.shape == (qkv.shape[0], kv_heads * vdim) and t.stride(1) == 1)
@@ -1434,7 +1595,8 @@ def qk_norm_rope_write(qkv: torch.Tensor, q_gain: Optional[torch.Tensor], k_gain
     _call("gb_qk_norm_rope_write", _ptr(qkv), qkv.stride(0), _ptr(q_gain), _ptr(k_gain), _ptr(inv_freq), _ptr(positions), _ptr(slots),
           _ptr(q_out), _ptr(kcache), _ptr(vcache), _dt(q_out), n, heads, kv_heads, dim, vdim, rot, float(eps), page_size,
           kcache.shape[0] * page_size, 1 if write_kv else 0, _ptr(status), _ptr(values_out), _ptr(values_in), ld_values,
-          _ptr(value_mix) if values_in is not None else 0, _stream())
+          _ptr(value_mix) if values_in is not None else 0, 1 if unit_norm else 0, float(q_temp[0]) if q_temp else 0.0,
+          float(q_temp[1]) if q_temp else 0.0, _stream())
 
 
 def sigmoid_attention_rows(q: torch.Tensor, out: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor, block_tables: torch.Tensor,
@@ -1494,12 +1656,15 @@ def sigmoid_attention_tiles(q: torch.Tensor, out: torch.Tensor, kcache: torch.Te
 
 
 # ------------------------------------------------------- softmax attention with a distance bias, a sink and an output gate
-def _sink_args(r1, r2, sink, gate, heads):
+def _sink_args(r1, r2, sink, gate, heads, vdim):
+    """The four terms for the launchers, and whether the gate has a logit per output channel (heads * vdim columns) instead
+    of one per head."""
     assert (r1 is None) == (r2 is None)
     for t in (r1, r2, sink):
         assert t is None or (t.dtype == torch.float32 and t.numel() == heads)
-    assert gate is None or (gate.dtype == torch.float32 and gate.shape[1] == heads and gate.stride(1) == 1)
-    return _ptr(r1), _ptr(r2), _ptr(sink), _ptr(gate), gate.stride(0) if gate is not None else 0
+    assert gate is None or (gate.dtype == torch.float32 and gate.shape[1] in (heads, heads * vdim) and gate.stride(1) == 1)
+    return (_ptr(r1), _ptr(r2), _ptr(sink), _ptr(gate), gate.stride(0) if gate is not None else 0), \
+        1 if gate is not None and gate.shape[1] != heads else 0
 
 
 def sink_attention_rows(q: torch.Tensor, out: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor, block_tables: torch.Tensor,
@@ -1508,15 +1673,17 @@ def sink_attention_rows(q: torch.Tensor, out: torch.Tensor, kcache: torch.Tensor
                         page_size: int, scale: float, window: Optional[int], status: torch.Tensor) -> None:
     """out[row, head, :] = sigmoid(gate[row, head]) * sum over the row's visible keys j of w_j v_j, the weights a softmax of
     s_j = q . k_j * scale - r1[head] * ln(1 + r2[head] * distance) whose denominator also holds exp(sink[head]). ``r1``/``r2``,
-    ``sink`` (float32 [heads]) and ``gate`` (float32 logits [n, heads], rows may be strided) are each optional. One warp per
+    ``sink`` (float32 [heads]) and ``gate`` (float32 logits [n, heads], or [n, heads * vdim] for a gate per output channel; rows
+    may be strided) are each optional. One warp per
     (row, head); any row, both dtypes."""
     _cuda(q, out, kcache, vcache, block_tables, row_seq, positions, r1, r2, sink, gate, status)
     n = q.shape[0]
     assert q.shape == (n, heads * dim) and out.shape == (n, heads * vdim) and q.is_contiguous() and out.is_contiguous()
     assert q.dtype == out.dtype == kcache.dtype == vcache.dtype and block_tables.is_contiguous()
+    terms, by_channel = _sink_args(r1, r2, sink, gate, heads, vdim)
     _call("gb_sink_attention_rows", _ptr(q), _ptr(out), _dt(q), _ptr(kcache), _ptr(vcache), _ptr(block_tables), block_tables.shape[1],
-          _ptr(row_seq), _ptr(positions), *_sink_args(r1, r2, sink, gate, heads), n, heads, kv_heads, dim, vdim, page_size,
-          kcache.shape[0], float(scale), int(window) if window else 0, _ptr(status), _stream())
+          _ptr(row_seq), _ptr(positions), *terms, n, heads, kv_heads, dim, vdim, page_size,
+          kcache.shape[0], float(scale), int(window) if window else 0, by_channel, _ptr(status), _stream())
 
 
 def sink_attention_decode_supported(dtype: torch.dtype, vdim: int) -> bool:
@@ -1534,9 +1701,10 @@ def sink_attention_decode(q: torch.Tensor, out: torch.Tensor, kcache: torch.Tens
     n = q.shape[0]
     assert q.shape == (n, heads * dim) and out.shape == (n, heads * vdim) and q.is_contiguous() and out.is_contiguous()
     assert q.dtype == out.dtype == kcache.dtype == vcache.dtype and block_tables.is_contiguous()
+    terms, by_channel = _sink_args(r1, r2, sink, gate, heads, vdim)
     _call("gb_sink_attention_decode", _ptr(q), _ptr(out), _dt(q), _ptr(kcache), _ptr(vcache), _ptr(block_tables),
-          block_tables.shape[1], _ptr(row_seq), _ptr(positions), *_sink_args(r1, r2, sink, gate, heads), n, heads, kv_heads, dim, vdim,
-          page_size, kcache.shape[0], float(scale), int(window) if window else 0, _ptr(status), _stream())
+          block_tables.shape[1], _ptr(row_seq), _ptr(positions), *terms, n, heads, kv_heads, dim, vdim,
+          page_size, kcache.shape[0], float(scale), int(window) if window else 0, by_channel, _ptr(status), _stream())
 
 
 def sink_attention_tiles_supported(dtype: torch.dtype, dim: int, vdim: int) -> bool:
@@ -1555,10 +1723,11 @@ def sink_attention_tiles(q: torch.Tensor, out: torch.Tensor, kcache: torch.Tenso
     assert q.dtype == out.dtype == kcache.dtype == vcache.dtype == torch.bfloat16
     assert q.shape == (n, heads * dim) and out.shape == (n, heads * vdim) and q.is_contiguous() and out.is_contiguous()
     assert block_tables.is_contiguous() and seq_first_row.shape[0] == seq_start_pos.shape[0] + 1
+    terms, by_channel = _sink_args(r1, r2, sink, gate, heads, vdim)
     _call("gb_sink_attention_tiles", _ptr(q), _ptr(out), _ptr(kcache), _ptr(vcache), _ptr(block_tables), block_tables.shape[1],
-          _ptr(seq_first_row), _ptr(seq_start_pos), *_sink_args(r1, r2, sink, gate, heads), seq_start_pos.shape[0],
+          _ptr(seq_first_row), _ptr(seq_start_pos), *terms, seq_start_pos.shape[0],
           max(int(max_rows_per_seq), 1), heads, kv_heads, dim, vdim, page_size, kcache.shape[0], float(scale),
-          int(window) if window else 0, _ptr(status), _stream())
+          int(window) if window else 0, by_channel, _ptr(status), _stream())
 
 
 # ------------------------------------------------------------------------------------------------ minGRU
@@ -1583,13 +1752,15 @@ def mingru_scan(proj: torch.Tensor, bias_z: torch.Tensor, bias_x: torch.Tensor, 
 def moe_route(h: torch.Tensor, w_router: torch.Tensor, correction: Optional[torch.Tensor], w_gate: Optional[torch.Tensor],
               positions: torch.Tensor, top: int, groups: int, keep: int, route_scale: float, choice: torch.Tensor,
               weight: torch.Tensor, gate: Optional[torch.Tensor], router_bias: Optional[torch.Tensor] = None,
-              softmax_chosen: bool = False) -> None:
+              softmax_chosen: bool = False, softmax: bool = False, group_best: bool = False, renorm_eps: Optional[float] = None) -> None:
     """Per row: float32 router logits, sigmoid scores, the ``top`` experts by score + correction among the ``keep`` best of
     ``groups`` runs of neighbouring experts, weights score * route_scale; ``gate`` = sigmoid(w_gate . h) per row. With
     ``softmax_chosen`` the ``top`` largest logits (plus ``router_bias``, float32 [experts]) win and the weights are the
-    softmax over the chosen logits alone."""
+    softmax over the chosen logits alone. ``softmax``: the scores are the softmax over all experts. ``group_best``: a run scores
+    its largest score, not the sum of its two largest. ``renorm_eps``: the chosen scores are divided by (their sum + it)."""
+    assert not (softmax_chosen and softmax)
     _cuda(h, w_router, correction, w_gate, positions, choice, weight, gate, router_bias)
-    assert router_bias is None or (softmax_chosen and router_bias.dtype == torch.float32 and router_bias.numel() == w_router.shape[0])
+    assert router_bias is None or ((softmax_chosen or softmax) and router_bias.dtype == torch.float32 and router_bias.numel() == w_router.shape[0])
     n, d = h.shape
     E = w_router.shape[0]
     assert h.is_contiguous() and w_router.dtype == torch.float32 and w_router.shape == (E, d) and w_router.is_contiguous()
@@ -1599,7 +1770,9 @@ def moe_route(h: torch.Tensor, w_router: torch.Tensor, correction: Optional[torc
     assert weight.dtype == torch.float32 and weight.shape == (n, top) and weight.is_contiguous()
     assert gate is None or (gate.dtype == torch.float32 and gate.numel() >= n)
     _call("gb_moe_route", _ptr(h), _dt(h), d, _ptr(w_router), _ptr(correction), _ptr(w_gate), _ptr(positions), n, E, top, groups, keep,
-          float(route_scale), _ptr(choice), _ptr(weight), _ptr(gate), _ptr(router_bias), 1 if softmax_chosen else 0, _stream())
+          float(route_scale), _ptr(choice), _ptr(weight), _ptr(gate), _ptr(router_bias),
+          1 if softmax_chosen else 2 if softmax else 0, 1 if group_best else 0, float(renorm_eps) if renorm_eps is not None else -1.0,
+          _stream())
 
 
 def moe_expert_rows(h: torch.Tensor, w_up: torch.Tensor, w_down: torch.Tensor, experts: int, choice: torch.Tensor,

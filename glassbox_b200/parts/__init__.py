@@ -2,7 +2,7 @@
 from .base import (FeedForward, Mixer, Norm, OutputHead, PagedKvSpec, Part, Position, StateSpec, TokenEmbedding, build_part,
                    register_part, registered)
 from . import (attention, block, delta_rule, embedding, latent_attention, linear_attention, mingru, mlp, moe, norm, parallel, rope,
-               sigmoid_attention, sink_attention, talking_attention)  # noqa: F401  (registration)
+               sigmoid_attention, sink_attention, state_space, talking_attention)  # noqa: F401  (registration)
 from .block import build_block
 from .embedding import Embedding, LmHead
 

@@ -152,6 +152,20 @@ class Norm(Part):
             copy.copy_(x)
 
 
+    def renorm(self, ctx, x, alpha: float, branch, copy=None) -> None:
+        """x <- norm(alpha * x + branch), float32 [n, d]: a residual that is normed after the sum. ``branch`` is the branch's
+        output, or its parts (``kernels.WeightedRows``, ``kernels.NormedPair``) for norms that say ``renorms_parts``; ``copy``
+        (activation dtype [n, d], optional) receives the new x. The default goes through ``forward``."""
+        tmp = ctx.scratch("residual_sum", tuple(x.shape), torch.float32)
+        torch.add(branch, x, alpha=alpha, out=tmp)
+        self.forward(ctx, tmp, x)
+        if copy is not None:
+            copy.copy_(x)
+
+    #: whether ``renorm`` takes a branch in its parts
+    renorms_parts = False
+
+
 class PreparedNorm:
     """What the product that last added into the residual ``x`` left behind for the norm that reads ``x`` next
     (``ctx.next_norm``, a hint from whoever wires the parts): ``pre`` = bfloat16(x * gain) and the scale that
@@ -212,6 +226,15 @@ class Mixer(Part):
     #: residual stream it sets that flag, and the part's last product then stores instead of adding (the buffer need
     #: not be cleared first). Parts that leave this False always add, into a buffer the wiring has cleared.
     can_overwrite_output = False
+    #: set by parts whose first step is one stacked product of their input into float32 (parameter ``w_in``): whoever owns
+    #: such a part may set ``projected_input`` before its parameters are collected. The part then declares no ``w_in``, and
+    #: ``forward`` receives the product's columns in the place of ``h``. ``input_pieces`` lists the rows of the tensors
+    #: that are stacked in ``w_in``.
+    can_take_projected_input = False
+    projected_input = False
+
+    def input_pieces(self) -> Tuple[int, ...]:
+        raise NotImplementedError
 
     def cache_spec(self):
         return None

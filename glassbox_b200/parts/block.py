@@ -3,10 +3,11 @@
 "pre_norm" is x += mixer(norm(x)); x += ffn(norm(x)), with no norms after the parts
 (crates/glassbox-core/src/model.rs:251-348; a layer may lack the feed-forward). "sandwich_norm" norms each branch on the
 way out as well: x += post(mixer(norm(x))); x += post(ffn(norm(x))). "branch_norm" norms them on the way out only: the
-branches read the residual itself, x += post(mixer(x)); x += post(ffn(x)). "hyper_connections" keeps the residual as several
+branches read the residual itself, x += post(mixer(x)); x += post(ffn(x)). "post_norm" norms after the sum: x <- norm(alpha x +
+mixer(x)); x <- norm(alpha x + ffn(x)). "hyper_connections" keeps the residual as several
 streams x_1 .. x_S per token: a branch reads u = sum_s read[s] x_s through its norm, and its output y comes back into all
 streams at once, x_t <- sum_s mix[s, t] x_s + write[t] y. The arrangement is looked up by name, so another
-wiring (post-norm, parallel branches) is another registered class.
+wiring is another registered class.
 """
 from __future__ import annotations
 
@@ -127,9 +128,9 @@ class BranchNormBlock(Part):
     def __init__(self, spec, *, hidden_size: int):
         super().__init__(spec)
         if spec.mixer_post_norm is None or (spec.ffn is not None and spec.ffn_post_norm is None):
-            raise ValueError("a branch_norm layer needs a norm behind its mixer and behind its feed-forward")
+            raise ValueError(f"a {spec.arrangement} layer needs a norm behind its mixer and behind its feed-forward")
         if spec.mixer_norm is not None or spec.ffn_norm is not None:
-            raise ValueError("a branch_norm layer has no norm in front of its branches")
+            raise ValueError(f"a {spec.arrangement} layer has no norm in front of its branches")
         self.hidden_size = hidden_size
         self.entry = ResidualItself(hidden_size=hidden_size)
         self.mixer = build_part("mixer", spec.mixer, hidden_size=hidden_size)
@@ -188,6 +189,38 @@ class BranchNormBlock(Part):
         if self.ffn is not None:
             self._branch(ctx, self.ffn, self.ffn_post_norm, x, lambda h, out: self.ffn.forward(ctx, h, out),
                          copy_after=next_reads_as_is)
+
+
+class PostNormBlock(BranchNormBlock):
+    """x <- mixer_post_norm(alpha * x + mixer(x)), then x <- ffn_post_norm(alpha * x + ffn(x)) (the second half only if the layer
+    has a feed-forward): the branches read the residual itself and the residual is normed after the sum. One kernel per branch
+    forms the sum, norms the row and writes it twice, as the float32 residual and in the activation dtype for the next
+    reader; a branch that is a weighted sum of rows or a pair of normed rows is formed by that kernel from its parts."""
+
+    def __init__(self, spec, *, hidden_size: int):
+        super().__init__(spec, hidden_size=hidden_size)
+        self.alpha = float(spec.residual_scale)
+
+    def _branch(self, ctx, part, post, x, run, copy_after: bool) -> None:
+        h = self._input(ctx, x)
+        branch = ctx.scratch("branch", tuple(x.shape), torch.float32)
+        ctx.overwrite_output = bool(part.can_overwrite_output)
+        if not ctx.overwrite_output:
+            branch.zero_()
+        ctx.accepts_weighted_rows = ctx.accepts_normed_pair = post.renorms_parts
+        ctx.weighted_rows = ctx.normed_pair = None
+        try:
+            run(h, branch)
+        finally:
+            ctx.overwrite_output = ctx.accepts_weighted_rows = ctx.accepts_normed_pair = False
+        for parts in (ctx.weighted_rows, ctx.normed_pair):
+            branch = parts if parts is not None else branch
+        ctx.weighted_rows = ctx.normed_pair = None
+        copy = ctx.scratch("h", tuple(x.shape)) if copy_after and x.dtype != ctx.dtype else None
+        post.renorm(ctx, x, self.alpha, branch, copy=copy)
+        ctx.prepared_norm = None         # x has changed behind the back of whatever was prepared from it
+        if copy is not None:
+            ctx.residual_copy = (x.data_ptr(), x.shape[0], copy)
 
 
 class StreamMixing(Part):
@@ -353,6 +386,8 @@ def collapse_streams(ctx, xs, streams: int, norm, out, rows=None, total=None) ->
 
 register_part("arrangement", "hyper_connections",
               lambda kind, *, layer_spec, hidden_size: HyperConnectionBlock(layer_spec, hidden_size=hidden_size), replace=True)
+register_part("arrangement", "post_norm",
+              lambda kind, *, layer_spec, hidden_size: PostNormBlock(layer_spec, hidden_size=hidden_size), replace=True)
 register_part("arrangement", "branch_norm",
               lambda kind, *, layer_spec, hidden_size: BranchNormBlock(layer_spec, hidden_size=hidden_size), replace=True)
 register_part("arrangement", "sandwich_norm",

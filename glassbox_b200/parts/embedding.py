@@ -41,14 +41,15 @@ class LmHead(OutputHead):
 
 
 class PositionalEmbedding(Embedding):
-    """x[i, :] = E[token_i, :] + P[position_i, :]: a learned vector per position, neither table scaled, the sum in float32."""
+    """x[i, :] = E[token_i, :] * scale + P[position_i, :]: a learned vector per position (not scaled), in float32."""
 
     def param_specs(self):
         return {"weight": ParamSpec((self.vocab_size, self.hidden_size)),
                 "positions": ParamSpec((self.spec.max_position, self.hidden_size))}
 
     def forward(self, ctx, tokens, x) -> None:
-        kernels.embed_positions(self.params["weight"], self.params["positions"], tokens, ctx.positions, x, ctx.status)
+        kernels.embed_positions(self.params["weight"], self.params["positions"], tokens, ctx.positions, x, ctx.status,
+                                scale=self.spec.scale)
 
 
 class ScaledEmbedding(Embedding):

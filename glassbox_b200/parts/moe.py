@@ -10,8 +10,12 @@ choice scores win, the lowest index among equals. The weights are not renormalis
 With `scoring` "softmax_chosen" the router is plainer: logits = W_router h + router_bias in float32, the `top_k` largest
 logits win (the lowest index among equals), and the weights are the softmax over the chosen logits alone.
 
+With `scoring` "softmax" the scores are the softmax over all experts; `group_score` "best" scores a run by its largest score, and
+`renormalise` divides the chosen scores by (their sum + that number).
+
 Expert: W_down relu(W_up h)^2, no biases; or, with `activation` "clamped_glu", W_down (g * sigmoid(slope * g) * (u + 1)) with
-g = min(W_gate h, limit), u = clamp(W_up h, -limit, limit): the up parameter then holds, per expert, gate row f and up row
+g = min(W_gate h, limit), u = clamp(W_up h, -limit, limit), or, with "swiglu", W_down (silu(W_gate h) * W_up h): for these the up
+parameter then holds, per expert, gate row f and up row
 f as neighbours (rows 2f and 2f + 1), so that a product's neighbouring outputs are the two inputs of one unit. Output: sum over the chosen experts of weight * expert(h), plus, if there is a
 shared expert, sigmoid(w_gate . h) * shared(h) (one gate number per token; without a gate the shared output is added as
 it is). The experts' matrices are stacked by rows into two parameters, so a kernel finds expert e at row e * size.
@@ -44,15 +48,20 @@ class RoutedExperts(FeedForward):
             raise ValueError(f"{s.num_experts} experts do not form {s.num_groups} equal groups of which {s.keep_groups} are kept")
         if s.keep_groups * (s.num_experts // s.num_groups) < s.top_k:
             raise ValueError(f"{s.keep_groups} groups of {s.num_experts // s.num_groups} experts cannot supply {s.top_k} per token")
-        if s.scoring not in ("sigmoid", "softmax_chosen") or s.activation not in ("relu2", "clamped_glu"):
+        if s.scoring not in ("sigmoid", "softmax_chosen", "softmax") or s.activation not in ("relu2", "clamped_glu", "swiglu"):
             raise ValueError(f"scoring {s.scoring!r} / activation {s.activation!r} are not known")
+        if s.group_score not in ("top2", "best"):
+            raise ValueError(f"group_score {s.group_score!r} must be 'top2' or 'best'")
+        if s.scoring == "softmax" and s.correction:
+            raise ValueError("a choice correction goes with sigmoid scores")
         if s.scoring == "softmax_chosen" and (s.num_groups != 1 or s.correction):
             raise ValueError("softmax weights over the chosen logits go with neither groups nor a choice correction")
         if s.activation == "clamped_glu" and not s.limit > 0:
             raise ValueError(f"limit {s.limit} must be positive")
         self.hidden_size = hidden_size
         self.E, self.top, self.ff, self.shared = s.num_experts, s.top_k, s.expert_size, s.shared_size
-        self.glu = s.activation == "clamped_glu"
+        self.glu = s.activation != "relu2"          # the expert has a gate and an up matrix
+        self.unit = {"relu2": None, "clamped_glu": (s.limit, s.glu_slope), "swiglu": kernels.SILU_UNIT}[s.activation]
 
     def param_specs(self):
         d, E, ff = self.hidden_size, self.E, self.ff
@@ -81,13 +90,14 @@ class RoutedExperts(FeedForward):
     def forward(self, ctx, h, residual) -> None:
         n, d, s = h.shape[0], self.hidden_size, self.spec
         p = self.params
-        unit = (s.limit, s.glu_slope) if self.glu else None
+        unit = self.unit
         choice = ctx.scratch("moe_choice", (n, self.top), torch.int32)
         weight = ctx.scratch("moe_weight", (n, self.top), torch.float32)
         gate = ctx.scratch("moe_gate", (n, 1), torch.float32) if "shared_gate" in p else None
         kernels.moe_route(h, p["router"], p.get("correction"), p.get("shared_gate"), ctx.positions, self.top, s.num_groups,
                           s.keep_groups, s.route_scale, choice, weight, gate, router_bias=p.get("router_bias"),
-                          softmax_chosen=s.scoring == "softmax_chosen")
+                          softmax_chosen=s.scoring == "softmax_chosen", softmax=s.scoring == "softmax",
+                          group_best=s.group_score == "best", renorm_eps=s.renormalise)
         shared_out = None
         if self.shared:
             # the shared expert is a dense squared-ReLU feed-forward: the framework's products, activation in the epilogue

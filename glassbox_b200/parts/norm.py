@@ -9,6 +9,7 @@ from .base import Norm, register_part
 
 class RmsNorm(Norm):
     launches_through_kernels_only = True
+    renorms_parts = True
 
     def __init__(self, spec, *, hidden_size: int):
         super().__init__(spec)
@@ -26,6 +27,10 @@ class RmsNorm(Norm):
 
     def add_normed(self, ctx, y, x, bias=None, copy=None) -> None:
         kernels.rmsnorm_add(y, self.params["weight"], x, self.eps, bias=bias, copy=copy)
+
+
+    def renorm(self, ctx, x, alpha, branch, copy=None) -> None:
+        kernels.post_norm(x, self.params["weight"], alpha, self.eps, branch, positions=ctx.positions, copy=copy)
 
 
 class UnitOffsetRmsNorm(RmsNorm):

@@ -1,16 +1,21 @@
-"""Two mixers side by side: both read the same input, and the output is left_scale * left + right_scale * right.
+"""Two mixers side by side: both read the same input, and the output is left_scale * left + right_scale * right, each side
+optionally normed over the model width first (an RMS norm with a gain of its own).
 
 Either mixer may be any registered one; their caches share the layer's cache layer (at most one of them may keep pages, any
 may keep a state per request: ``combine_cache_specs``). Each writes its output into a float32 buffer of its own (as under
 a wiring that norms a branch: ``ctx.overwrite_output``); one small kernel forms the weighted sum and stores it or adds it
-into the residual, in float32.
+into the residual, in float32. A wiring that norms the branch may take a normed pair over in its parts
+(``ctx.accepts_normed_pair`` / ``ctx.normed_pair``) and form the sum on its way over the rows. Where both sides begin with one
+stacked product of their input, the two matrices may be one (``shared_projection``): one product then serves both.
 """
 from __future__ import annotations
 
 import torch
 
 from .. import kernels
+from ..weights.binding import ParamSpec
 from .base import Mixer, build_part, combine_cache_specs, register_part, sub_view
+from .linear import linear
 
 
 class ParallelMixer(Mixer):
@@ -22,9 +27,27 @@ class ParallelMixer(Mixer):
         self.hidden_size = hidden_size
         self.left = build_part("mixer", spec.left, hidden_size=hidden_size)
         self.right = build_part("mixer", spec.right, hidden_size=hidden_size)
+        self.left_norm = self.right_norm = None
+        if spec.output_norm is not None:
+            self.left_norm = build_part("norm", spec.output_norm, hidden_size=hidden_size)
+            self.right_norm = build_part("norm", spec.output_norm, hidden_size=hidden_size)
+        if spec.shared_projection:
+            for part in (self.left, self.right):
+                if not part.can_take_projected_input:
+                    raise ValueError(f"a mixer of kind {part.spec.kind!r} cannot share its input projection")
+                part.projected_input = True
+            self.left_cols, self.in_cols = self.left.in_cols, self.left.in_cols + self.right.in_cols
 
     def sub_parts(self):
-        return {"left": self.left, "right": self.right}
+        parts = {"left": self.left, "right": self.right}
+        if self.left_norm is not None:
+            parts.update({"left_norm": self.left_norm, "right_norm": self.right_norm})
+        return parts
+
+    def param_specs(self):
+        if not self.spec.shared_projection:
+            return {}
+        return {"w_in": ParamSpec((self.in_cols, self.hidden_size), pieces=self.left.input_pieces() + self.right.input_pieces())}
 
     def recordable(self, decode_only: bool) -> bool:
         return True
@@ -35,6 +58,17 @@ class ParallelMixer(Mixer):
     def forward(self, ctx, h, residual, cache, writes_cache: bool) -> None:
         n, d = residual.shape
         overwrite = getattr(ctx, "overwrite_output", False)
+        takes_pair = getattr(ctx, "accepts_normed_pair", False)
+        # what the wiring offers to take over is this mixer's output, not that of either side
+        offers = {name: getattr(ctx, name, False) for name in ("accepts_output_bias", "accepts_weighted_rows", "accepts_normed_pair")}
+        for name in offers:
+            setattr(ctx, name, False)
+        inputs = {"left": h, "right": h}
+        if self.spec.shared_projection:
+            ld = -(-self.in_cols // 4) * 4
+            proj = ctx.scratch("parallel_proj", (n, ld), torch.float32)[:, :self.in_cols]
+            linear(ctx, h, self.params["w_in"], proj)
+            inputs = {"left": proj[:, :self.left_cols], "right": proj[:, self.left_cols:]}
         outs = []
         for name, part in (("left", self.left), ("right", self.right)):
             y = ctx.scratch("parallel_" + name, (n, d), torch.float32)
@@ -42,11 +76,23 @@ class ParallelMixer(Mixer):
             if not ctx.overwrite_output:
                 y.zero_()
             try:
-                part.forward(ctx, h, y, sub_view(cache, name, part.cache_spec()), writes_cache)
+                part.forward(ctx, inputs[name], y, sub_view(cache, name, part.cache_spec()), writes_cache)
             finally:
                 ctx.overwrite_output = overwrite
             outs.append(y)
-        kernels.scaled_sum(outs[0], outs[1], self.spec.left_scale, self.spec.right_scale, residual, accumulate=not overwrite)
+        for name, was in offers.items():
+            setattr(ctx, name, was)
+        s = self.spec
+        if self.left_norm is not None:
+            lrms, rrms = self.left_norm.as_rms(), self.right_norm.as_rms()
+            if overwrite and takes_pair and lrms is not None and rrms is not None and lrms[1] == rrms[1]:
+                ctx.normed_pair = kernels.NormedPair(outs[0], outs[1], lrms[0], rrms[0], s.left_scale, s.right_scale, lrms[1])
+                return
+            for i, norm in enumerate((self.left_norm, self.right_norm)):
+                normed = ctx.scratch("parallel_normed_%d" % i, (n, d), torch.float32)
+                norm.forward(ctx, outs[i], normed)
+                outs[i] = normed
+        kernels.scaled_sum(outs[0], outs[1], s.left_scale, s.right_scale, residual, accumulate=not overwrite)
 
 
 register_part("mixer", "parallel", ParallelMixer, replace=True)

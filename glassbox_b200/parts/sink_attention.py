@@ -1,12 +1,14 @@
 """Causal grouped-query softmax attention whose positions enter as a bias on the distance, with a sink in the softmax.
 
 x -> one stacked product gives q (heads x head_dim), k (kv heads x head_dim), v (kv heads x value_dim) and one gate logit
-per head as float32 sums -> every query and key head is RMS-normed over head_dim (one gain shared by the query heads, one by
-the key heads); nothing is rotated -> values: a "source" layer leaves its v rows in a float32 buffer that lives for the
+per head (or per output channel) as float32 sums -> every query and key head is RMS-normed over head_dim (one gain shared by
+the query heads, one by the key heads, or no gains); nothing is rotated; queries may carry a temperature that grows with the
+logarithm of the position -> values: a "source" layer leaves its v rows in a float32 buffer that lives for the
 step, a "mixed" layer replaces its v by (1 - lambda) v + lambda v_source of the same token; k and the (mixed) v go into the
 paged cache at the row's slot (all rows of the step before any attention) -> per (row, head), over the row's visible keys j
 of its own request: s_j = q . k_j * scale - r1_h * ln(1 + r2_h * (i - j)), weights exp(s_j - m) / (sum_j exp(s_j - m) +
-exp(sink_h - m)): the sink adds to the denominator and to nothing else -> the head's output times sigmoid(gate logit) ->
+exp(sink_h - m)): the sink adds to the denominator and to nothing else (bias and sink are each optional) -> the head's output
+times sigmoid(gate logit) ->
 residual += out Wo^T. A window w lets position p see keys p-w+1 .. p; pages behind the window of every future query go
 back to the pool, as for any windowed paged group. Norms, distances, logarithms, scores, weights, the sums over keys, the
 value mix and the gate are float32 whatever the activation dtype; the cache holds the activation dtype.
@@ -27,6 +29,7 @@ VALUE_SOURCE = "value_mix_source"
 class SinkAttention(Mixer):
     launches_through_kernels_only = True
     can_overwrite_output = True
+    can_take_projected_input = True
 
     def __init__(self, spec, *, hidden_size: int):
         super().__init__(spec)
@@ -39,16 +42,26 @@ class SinkAttention(Mixer):
             raise ValueError(f"window {s.window} must be positive")
         if s.value_mix not in ("none", "source", "mixed"):
             raise ValueError(f"value_mix {s.value_mix!r} must be 'none', 'source' or 'mixed'")
+        if s.gate_per not in ("head", "channel"):
+            raise ValueError(f"gate_per {s.gate_per!r} must be 'head' or 'channel'")
+        if s.q_temp is not None and not s.q_temp[1] > 0:
+            raise ValueError(f"the query temperature grows every {s.q_temp[1]} positions: must be positive")
         self.hidden_size = hidden_size
         self.H, self.G, self.D, self.V = s.num_heads, s.num_kv_heads, s.head_dim, s.value_dim
         self.gate_col = (self.H + self.G) * self.D + self.G * self.V
-        self.in_cols = self.gate_col + (self.H if s.output_gate else 0)
+        self.gate_cols = 0 if not s.output_gate else self.H if s.gate_per == "head" else self.H * self.V
+        self.in_cols = self.gate_col + self.gate_cols
+
+    def input_pieces(self):
+        pieces = (self.H * self.D, self.G * self.D, self.G * self.V)
+        return pieces + ((self.gate_cols,) if self.gate_cols else ())
 
     def param_specs(self):
         d, s = self.hidden_size, self.spec
-        pieces = (self.H * self.D, self.G * self.D, self.G * self.V) + ((self.H,) if s.output_gate else ())
-        specs = {"w_in": ParamSpec((self.in_cols, d), pieces=pieces), "wo": ParamSpec((d, self.H * self.V))}
-        if s.qk_norm_eps is not None:
+        specs = {"wo": ParamSpec((d, self.H * self.V))}
+        if not self.projected_input:
+            specs["w_in"] = ParamSpec((self.in_cols, d), pieces=self.input_pieces())
+        if s.qk_norm_eps is not None and s.qk_norm_gain:
             specs["q_norm"] = ParamSpec((self.D,), role="gain")
             specs["k_norm"] = ParamSpec((self.D,), role="gain")
         if s.distance_bias:
@@ -65,16 +78,20 @@ class SinkAttention(Mixer):
 
     def forward(self, ctx, h, residual, cache, writes_cache: bool) -> None:
         n, s = h.shape[0], self.spec
-        ld = -(-self.in_cols // 4) * 4                      # rows of the float32 buffer start 16-byte aligned
-        proj = ctx.scratch("sk_proj", (n, ld), torch.float32)[:, :self.in_cols]
-        linear(ctx, h, self.params["w_in"], proj)
+        if self.projected_input:
+            proj = h
+        else:
+            ld = -(-self.in_cols // 4) * 4                  # rows of the float32 buffer start 16-byte aligned
+            proj = ctx.scratch("sk_proj", (n, ld), torch.float32)[:, :self.in_cols]
+            linear(ctx, h, self.params["w_in"], proj)
         q = ctx.scratch("sk_q", (n, self.H * self.D))
         source = ctx.scratch(VALUE_SOURCE, (n, self.G * self.V), torch.float32) if s.value_mix != "none" else None
         kernels.qk_norm_rope_write(proj[:, :self.gate_col], self.params.get("q_norm"), self.params.get("k_norm"), None, ctx.positions,
                                    cache.slots, q, cache.k, cache.v, self.H, self.G, self.D, self.V, 0, s.qk_norm_eps or 0.0,
                                    cache.page_size, writes_cache, ctx.status,
                                    values_out=source if s.value_mix == "source" else None,
-                                   values_in=source if s.value_mix == "mixed" else None, value_mix=self.params.get("value_mix"))
+                                   values_in=source if s.value_mix == "mixed" else None, value_mix=self.params.get("value_mix"),
+                                   unit_norm=s.qk_norm_eps is not None and not s.qk_norm_gain, q_temp=s.q_temp)
         att = ctx.scratch("att", (n, self.H * self.V))
         self.attend(ctx, q, att, cache, proj[:, self.gate_col:] if s.output_gate else None)
         linear(ctx, att, self.params["wo"], residual, accumulate=not getattr(ctx, "overwrite_output", False))
