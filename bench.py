@@ -588,6 +588,55 @@ def babotar_workload(args):
     return out
 
 
+# ------------------------------------------------------------------------------------------------ Felovik beside its neighbours
+#: layer sizes that resemble real models' (random weights): a Felovik model whose layers are all the pair of gated attention
+#: and a state-space mixer (inner width twice the model's), the feed-forwards in turn a dense clamped gated unit of width
+#: ``ff`` and a mixture of 16 SwiGLU experts of width ``ff / 4`` of which four per token (as many multiply-adds per token as
+#: the dense one). Beside it Babotar (the framework's other model of attention and a recurrence side by side), Tagenex (its
+#: other model of gated attention and routed gated experts) and the Llama decoder, all of the same width, depth and
+#: feed-forward width.
+FELOVIK_SIZES = {
+    "w1024": dict(left=dict(heads=16, kv_heads=4, dim=64, vdim=64), right=dict(heads=32, groups=2, vdim=64, state=128, conv=4, norm_groups=2),
+                  moe=dict(experts=16, top=4, ff=1024, groups=(4, 2))),
+    "w2048": dict(left=dict(heads=32, kv_heads=8, dim=64, vdim=64), right=dict(heads=64, groups=4, vdim=64, state=128, conv=4, norm_groups=4),
+                  moe=dict(experts=16, top=4, ff=2048, groups=(4, 2))),
+}
+
+
+def felovik_raw(size: dict, own: dict, max_positions: int = 8192) -> dict:
+    from glassbox_b200.models.felovik import make_felovik_raw_config
+    layers = []
+    for i in range(size["layers"]):
+        lf = dict(own["left"])
+        lf.update(scale=lf["dim"] ** -0.5, q_temp={"coef": 0.1, "every": 1024})
+        if i % 2:
+            e = own["moe"]
+            mlp = {"kind": "moe", "expert": {"ff": e["ff"]}, "router": {"experts": e["experts"], "top": e["top"],
+                                                                        "groups": {"count": e["groups"][0], "keep": e["groups"][1]}}}
+        else:
+            mlp = {"kind": "dense", "ff": size["ff"], "limit": 7.0}
+        layers.append({"type": "parallel", "mixer": {"left": lf, "right": dict(own["right"])}, "mlp": mlp})
+    return make_felovik_raw_config(vocab=size["vocab"], width=size["width"], max_positions=max_positions, layers=layers, alpha=2.0,
+                                   embedding_scale=4.0)
+
+
+def felovik_workload(args):
+    """Prefill and decode throughput of Felovik models beside Babotar, Tagenex and the Llama decoder of equal width, depth and
+    feed-forward width; one JSON line. Decode steps end at the context length; three timed regions per point."""
+    T, ctx, K, W = 2048, args.context, min(args.steps, 128), max(args.warmup, 3)
+    out = {"workload": "felovik", "dtype": args.dtype, "context": ctx, "prefill_tokens": T, "decode_steps": K, "sizes": {}}
+    for name, size in ZURERAX_SIZES.items():
+        llama = dict(num_hidden_layers=size["layers"], hidden_size=size["width"], intermediate_size=size["ff"],
+                     vocab_size=size["vocab"], rope_theta=10000.0, rms_norm_eps=1e-5, tie_word_embeddings=False,
+                     max_position_embeddings=8192, **size["llama"])
+        arms = (("felovik", dict(raw=felovik_raw(size, FELOVIK_SIZES[name], max(8192, ctx)))),
+                ("babotar", dict(raw=babotar_raw(size, BABOTAR_SIZES[name], max(8192, ctx)))),
+                ("tagenex", dict(raw=tagenex_raw(size, TAGENEX_SIZES[name]))), ("llama", dict(shape=llama)))
+        out["sizes"][name] = {label: measure_arm(f"{label}-{name}", args, T, ctx, K, W, **kw) for label, kw in arms
+                              if not args.only or label in args.only.split(",")}
+    return out
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -602,14 +651,15 @@ def main():
     ap.add_argument("--no-points", action="store_true", help="only the headline region: no other batches, prefill or e2e")
     ap.add_argument("--no-others", action="store_true",
                     help="skip the other model sizes, the serving workload, the 32-bit path and the CPU baseline")
-    ap.add_argument("--workload", default="decode", choices=["decode", "serving", "zurerax", "lonorax", "tagenex", "babotar"],
+    ap.add_argument("--workload", default="decode", choices=["decode", "serving", "zurerax", "lonorax", "tagenex", "babotar", "felovik"],
                     help="serving: the mixed workload of the 360M configuration (64 requests, prompts 32-2048, outputs "
                          "32-512, prompt portions of 512, a quarter of the requests sharing a 384-token prefix) through "
                          "the scheduler; prints its own JSON line. zurerax: prefill and decode throughput of Zurerax models "
                          "at two widths beside the Llama decoder of equal size; prints its own JSON line. lonorax: the same for "
                          "Lonorax models beside Zurerax and Llama of equal size; tagenex: the same for Tagenex models beside Llama "
-                         "and Lonorax of equal size; babotar: the same for Babotar models beside Zurerax and Llama of equal size")
-    ap.add_argument("--only", default="", help="with --workload lonorax, tagenex or babotar: the arms to run (babotar,tagenex,lonorax,zurerax,llama), with commas")
+                         "and Lonorax of equal size; babotar: the same for Babotar models beside Zurerax and Llama of equal size; "
+                         "felovik: the same for Felovik models beside Babotar, Tagenex and Llama of equal size")
+    ap.add_argument("--only", default="", help="with --workload lonorax, tagenex, babotar or felovik: the arms to run (felovik,babotar,tagenex,lonorax,zurerax,llama), with commas")
     args = ap.parse_args()
 
     if args.impl == "reference":
@@ -636,6 +686,9 @@ def main():
         return 0
     if args.workload == "babotar":
         print(json.dumps(babotar_workload(args)))
+        return 0
+    if args.workload == "felovik":
+        print(json.dumps(felovik_workload(args)))
         return 0
     K, W, B, CTX = args.steps, max(args.warmup, 3), args.batch, args.context
     pk = peaks()

@@ -433,6 +433,13 @@ __device__ __forceinline__ float2 pn_block_sum2(float a, float b, float2* partia
     return t;
 }
 
+// four neighbours at once (the address is a multiple of four elements)
+__device__ __forceinline__ void pn_store4(float* at, float4 v) { *reinterpret_cast<float4*>(at) = v; }
+__device__ __forceinline__ void pn_store4(__nv_bfloat16* at, float4 v) {
+    const __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+    *reinterpret_cast<uint2*>(at) = make_uint2(*reinterpret_cast<const unsigned*>(&lo), *reinterpret_cast<const unsigned*>(&hi));
+}
+
 template <int MODE, int VMAX, typename T>
 __global__ void __launch_bounds__(PN_THREADS) post_norm_kernel(PostNormArgs p) {
     __shared__ float2 partial[PN_THREADS / 32];
@@ -514,10 +521,7 @@ __global__ void __launch_bounds__(PN_THREADS) post_norm_kernel(PostNormArgs p) {
                 const float4 g = *reinterpret_cast<const float4*>(p.gain + j);
                 const float4 w = make_float4(g.x * (t[i].x * s), g.y * (t[i].y * s), g.z * (t[i].z * s), g.w * (t[i].w * s));
                 *reinterpret_cast<float4*>(x + j) = w;
-                if (cp != nullptr) {
-                    cp[j] = gb_from_float<T>(w.x); cp[j + 1] = gb_from_float<T>(w.y);
-                    cp[j + 2] = gb_from_float<T>(w.z); cp[j + 3] = gb_from_float<T>(w.w);
-                }
+                if (cp != nullptr) pn_store4(cp + j, w);
             }
         }
     } else {                             // any other row: a value is formed again in every pass
@@ -581,7 +585,7 @@ GB_EXPORT int gb_post_norm(float* x, long long ldx, const float* gain, float alp
     PostNormArgs p = {x, ldx, gain, alpha, eps, y, b, ga, gb, a_scale, b_scale, pair_eps, weighted, weight, shared, gate, top, copy,
                       positions, n, d};
     const uintptr_t all = (uintptr_t)x | (uintptr_t)gain | (uintptr_t)y | (uintptr_t)b | (uintptr_t)ga | (uintptr_t)gb | (uintptr_t)weighted |
-                          (uintptr_t)shared;
+                          (uintptr_t)shared | (uintptr_t)copy;
     const bool vec = d % 4 == 0 && ldx % 4 == 0 && (all & 15) == 0;
     const bool half = copy != nullptr && copy_dtype == GB_BF16;
 #define PN_GO(M)                                                                \
@@ -598,11 +602,10 @@ GB_EXPORT int gb_post_norm(float* x, long long ldx, const float* gain, float alp
 // A gate in front of a norm over equal parts of a row: u = y * silu(z), out = w * u / sqrt(mean over the part of u^2 + eps).
 // y float32 [n, groups * size], z float32 logits (row stride ldz), w float32 [groups * size]. One block per (row, part).
 // ----------------------------------------------------------------------------------------------
-template <int THREADS, typename T>
+template <int THREADS, int VMAX, typename T>
 __global__ void __launch_bounds__(THREADS) gate_group_norm_kernel(const float* __restrict__ y, const float* __restrict__ z, long long ldz,
                                                                   const float* __restrict__ w, T* __restrict__ out,
-                                                                  const int* __restrict__ positions, int groups, int size, float eps,
-                                                                  int vec) {
+                                                                  const int* __restrict__ positions, int groups, int size, float eps) {
     __shared__ float partial[THREADS / 32];
     gb_pdl_launch_dependents();
     gb_pdl_wait();
@@ -613,12 +616,14 @@ __global__ void __launch_bounds__(THREADS) gate_group_norm_kernel(const float* _
     const float* gz = z + (size_t)row * ldz + (size_t)g * size;
     const float* gw = w + (size_t)g * size;
     T* dst = out + at;
-    constexpr int VMAX = 4;
-    float4 u[VMAX];
+    // VMAX pieces of four numbers per thread in registers (rows of whole 16-byte pieces); VMAX 0: any row, in two passes
+    float4 u[VMAX > 0 ? VMAX : 1];
     float ss = 0.f;
-    const bool quick = vec && size <= THREADS * 4 * VMAX;
-    auto gated = [](float a, float b) { return a * (b / (1.0f + expf(-b))); };
-    if (quick) {
+    auto gated = [](float a, float b) {
+        if constexpr (sizeof(T) == 4) return a * (b / (1.0f + expf(-b)));
+        else return __fdividef(a * b, 1.0f + __expf(-b));       // (the result is rounded to 16 bits in the end)
+    };
+    if constexpr (VMAX > 0) {
         float4 q[VMAX];
 #pragma unroll
         for (int i = 0; i < VMAX; ++i) {
@@ -644,14 +649,13 @@ __global__ void __launch_bounds__(THREADS) gate_group_norm_kernel(const float* _
 #pragma unroll
     for (int i = 0; i < THREADS / 32; ++i) ss += partial[i];
     const float s = 1.0f / sqrtf(ss / (float)size + eps);
-    if (quick) {
+    if constexpr (VMAX > 0) {
 #pragma unroll
         for (int i = 0; i < VMAX; ++i) {
             const int j = (i * THREADS + threadIdx.x) * 4;
             if (j < size) {
                 const float4 g4 = *reinterpret_cast<const float4*>(gw + j);
-                dst[j] = gb_from_float<T>(g4.x * (u[i].x * s)); dst[j + 1] = gb_from_float<T>(g4.y * (u[i].y * s));
-                dst[j + 2] = gb_from_float<T>(g4.z * (u[i].z * s)); dst[j + 3] = gb_from_float<T>(g4.w * (u[i].w * s));
+                pn_store4(dst + j, make_float4(g4.x * (u[i].x * s), g4.y * (u[i].y * s), g4.z * (u[i].z * s), g4.w * (u[i].w * s)));
             }
         }
     } else {
@@ -664,15 +668,22 @@ GB_EXPORT int gb_gate_group_norm(const float* y, const float* z, long long ldz, 
     GB_REQUIRE(n >= 0 && groups > 0 && size > 0 && ldz >= (long long)groups * size, "gb_gate_group_norm: bad sizes");
     GB_REQUIRE(out_dtype == GB_F32 || out_dtype == GB_BF16, "gb_gate_group_norm: unsupported output dtype %d", out_dtype);
     if (n == 0) return 0;
-    const int vec = size % 4 == 0 && ldz % 4 == 0 && (((uintptr_t)y | (uintptr_t)z | (uintptr_t)w) & 15) == 0;
-#define GGN_GO(TH, T)                                                                                                            \
-    gb_launch(GB_PDL_ELEMENTWISE, gate_group_norm_kernel<TH, T>, dim3(n * groups), dim3(TH), 0, stream, y, z, ldz, w, (T*)out,   \
-              positions, groups, size, eps, vec)
-    if (size <= 512) {
-        if (out_dtype == GB_F32) GGN_GO(64, float); else GGN_GO(64, __nv_bfloat16);
-    } else {
-        if (out_dtype == GB_F32) GGN_GO(256, float); else GGN_GO(256, __nv_bfloat16);
+    const bool vec = size % 4 == 0 && ldz % 4 == 0 && (((uintptr_t)y | (uintptr_t)z | (uintptr_t)w | (uintptr_t)out) & 15) == 0;
+#define GGN_GO(TH, VM)                                                                                                               \
+    {                                                                                                                                \
+        if (out_dtype == GB_F32)                                                                                                     \
+            gb_launch(GB_PDL_ELEMENTWISE, gate_group_norm_kernel<TH, VM, float>, dim3(n * groups), dim3(TH), 0, stream, y, z, ldz, w, \
+                      (float*)out, positions, groups, size, eps);                                                                    \
+        else                                                                                                                         \
+            gb_launch(GB_PDL_ELEMENTWISE, gate_group_norm_kernel<TH, VM, __nv_bfloat16>, dim3(n * groups), dim3(TH), 0, stream, y, z, \
+                      ldz, w, (__nv_bfloat16*)out, positions, groups, size, eps);                                                    \
     }
+    if (!vec || size > 256 * 4 * 4) GGN_GO(256, 0)
+    else if (size <= 64 * 4) GGN_GO(64, 1)
+    else if (size <= 128 * 4) GGN_GO(128, 1)
+    else if (size <= 256 * 4) GGN_GO(256, 1)
+    else if (size <= 256 * 8) GGN_GO(256, 2)
+    else GGN_GO(256, 4)
 #undef GGN_GO
     return gb_check_launch("gb_gate_group_norm");
 }

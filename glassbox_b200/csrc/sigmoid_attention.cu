@@ -43,7 +43,7 @@ __global__ void __launch_bounds__(512) qk_norm_rope_write_kernel(
     const int off = (int)(slot % page_size);
     const int pairs = D / 2;          // (an odd last channel is handled apart)
     const float temp = temp_every > 0.f ? 1.0f + temp_coef * logf(floorf(__fdiv_rn((float)(pos + 1), temp_every)) + 1.0f) : 1.0f;
-    for (int head = warp; head < H + G; head += warps) {
+    for (int head = blockIdx.y * warps + warp; head < H + G; head += warps * gridDim.y) {
         const bool is_q = head < H;
         if (!is_q && !store) continue;
         const float* x = src + (size_t)head * D;     // q heads, then k heads: contiguous in the stacked row
@@ -76,7 +76,7 @@ __global__ void __launch_bounds__(512) qk_norm_rope_write_kernel(
         }
         if ((D & 1) && lane == 0) dst[D - 1] = gb_from_float<T>(x[D - 1] * r * (gain ? gain[D - 1] : 1.f));
     }
-    if (store || values_out != nullptr) {
+    if (blockIdx.y == gridDim.y - 1 && (store || values_out != nullptr)) {      // (the row's last block has the fewest heads)
         const float* v = src + (size_t)(H + G) * D;
         const float lam = values_in != nullptr ? *value_mix : 0.f;
         for (int idx = threadIdx.x; idx < G * V; idx += blockDim.x) {
@@ -101,13 +101,15 @@ GB_EXPORT int gb_qk_norm_rope_write(const float* qkv, long long ld, const float*
     GB_REQUIRE(rot >= 0 && rot % 2 == 0 && rot <= D, "gb_qk_norm_rope_write: %d rotated channels of %d", rot, D);
     GB_REQUIRE(rot == 0 || inv_freq != nullptr, "gb_qk_norm_rope_write: a rotation needs its frequencies");
     if (n == 0) return 0;
-    const dim3 block(32 * (H + G < 4 ? 4 : (H + G > 16 ? 16 : H + G)));      // a warp per head, up to 16 at a time
+    // a warp per head: up to sixteen in a block over many rows, up to eight where few rows leave multiprocessors idle
+    const int most = n > 296 ? 16 : 8, warps = H + G < 4 ? 4 : (H + G > most ? most : H + G);
+    const dim3 block(32 * warps), grid(n, n > 296 ? 1 : gb_ceil_div(H + G, warps));
     if (dtype == GB_F32)
-        gb_launch(GB_PDL_ELEMENTWISE, qk_norm_rope_write_kernel<float>, dim3(n), block, 0, stream, qkv, ld, q_gain, k_gain, inv_freq,
+        gb_launch(GB_PDL_ELEMENTWISE, qk_norm_rope_write_kernel<float>, grid, block, 0, stream, qkv, ld, q_gain, k_gain, inv_freq,
                   positions, slots, (float*)q_out, (float*)kcache, (float*)vcache, n, H, G, D, V, rot, eps, page_size, num_slots,
                   write_kv, status, values_out, values_in, ld_values, value_mix, unit_norm, temp_coef, temp_every);
     else if (dtype == GB_BF16)
-        gb_launch(GB_PDL_ELEMENTWISE, qk_norm_rope_write_kernel<__nv_bfloat16>, dim3(n), block, 0, stream, qkv, ld, q_gain, k_gain,
+        gb_launch(GB_PDL_ELEMENTWISE, qk_norm_rope_write_kernel<__nv_bfloat16>, grid, block, 0, stream, qkv, ld, q_gain, k_gain,
                   inv_freq, positions, slots, (__nv_bfloat16*)q_out, (__nv_bfloat16*)kcache, (__nv_bfloat16*)vcache, n, H, G, D, V,
                   rot, eps, page_size, num_slots, write_kv, status, values_out, values_in, ld_values, value_mix, unit_norm, temp_coef, temp_every);
     else

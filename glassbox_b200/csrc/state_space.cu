@@ -222,23 +222,46 @@ struct SdVec<1> { typedef float type; };
 template <>
 struct SdVec<4> { typedef float4 type; };
 
-template <int VEC>
-__global__ void __launch_bounds__(SD_THREADS) ssd_decode_kernel(SsdDecodeArgs p) {
+// One channel's convolution at a single new token: `own` is the token's input, the ring holds the ones before.
+template <int TAPS>
+__device__ __forceinline__ float sd_conv(const SsdDecodeArgs& p, const float* ring, int ch, int pos, int C, float own) {
+    const int taps = TAPS > 0 ? TAPS : p.taps;
+    float acc = p.conv_b[ch];
+    if constexpr (TAPS > 0) {
+        float w[TAPS], v[TAPS];           // every load before the first use
+#pragma unroll
+        for (int j = 0; j < TAPS; ++j) {
+            w[j] = p.conv_w[(size_t)ch * TAPS + j];
+            const int q = pos - (TAPS - 1) + j;
+            v[j] = j == TAPS - 1 ? own : q >= 0 ? ring[(size_t)(q % TAPS) * C + ch] : 0.f;
+        }
+#pragma unroll
+        for (int j = 0; j < TAPS; ++j) acc = fmaf(w[j], v[j], acc);
+    } else {
+        for (int j = 0; j < taps; ++j) {
+            const int q = pos - (taps - 1) + j;
+            if (q >= 0) acc = fmaf(p.conv_w[(size_t)ch * taps + j], j == taps - 1 ? own : ring[(size_t)(q % taps) * C + ch], acc);
+        }
+    }
+    return rc_silu(acc);
+}
+
+template <int VEC, int TAPS>
+__global__ void __launch_bounds__(SD_THREADS, 3) ssd_decode_kernel(SsdDecodeArgs p) {
     typedef typename SdVec<VEC>::type vec_t;
     extern __shared__ __align__(16) float sd_smem[];
     float* Bs = sd_smem, *Cs = Bs + p.N, *xs = Cs + p.N, *part = xs + ((p.cols + 3) & ~3) + ((4 - (2 * p.N) % 4) & 3);
     gb_pdl_launch_dependents();
     gb_pdl_wait();
     const int seq = blockIdx.x, head = blockIdx.y, c0 = blockIdx.z * p.cols, nc = min(p.cols, p.V - c0);
-    const int pos = p.seq_start_pos[seq];
+    const int pos = p.seq_start_pos[seq], slot = p.seq_slots[seq];
+    const size_t row = (size_t)p.seq_first_row[seq];
     if (pos < 0) return;
-    const int slot = p.seq_slots[seq];
     if (slot < 0 || slot >= p.num_slots) {
         if (threadIdx.x == 0) atomicOr(p.status, GB_STATUS_BAD_SLOT);
         return;
     }
-    const size_t row = (size_t)p.seq_first_row[seq];
-    const int N = p.N, V = p.V, tid = threadIdx.x;
+    const int N = p.N, V = p.V, tid = threadIdx.x, taps = TAPS > 0 ? TAPS : p.taps;
     const int inner = p.heads * V, per = p.heads / p.groups, g = head / per, C = inner + 2 * p.groups * N;
     float* slot_state = p.state + (size_t)slot * p.state_stride;
     const int nvec = nc / VEC, par = SD_THREADS / nvec;         // (VEC divides nc: the launch sees to it)
@@ -251,22 +274,29 @@ __global__ void __launch_bounds__(SD_THREADS) ssd_decode_kernel(SsdDecodeArgs p)
         const int r = my_r + u * par;
         if (active && r < N) first[u] = *reinterpret_cast<const vec_t*>(S + (size_t)r * V);
     }
+    const float dt_raw = p.dt_raw[row * p.ld_dt + head] + p.dt_bias[head], rate = p.a_log[head], skip = p.skip[head];
     // the token's B, C and this block's x: the convolution over the ring's last inputs and the token's own
     float* ring = slot_state + p.conv_off;
     const bool keeps_bc = head % per == 0 && blockIdx.z == 0;   // one block per group stores the shared channels' inputs
-    for (int i = tid; i < 2 * N + nc; i += SD_THREADS) {
-        const int ch = i < N ? inner + g * N + i : i < 2 * N ? inner + p.groups * N + g * N + (i - N) : head * V + c0 + (i - 2 * N);
-        const float own = p.xbc[row * p.ldx + ch];
-        float acc = fmaf(p.conv_w[(size_t)ch * p.taps + p.taps - 1], own, p.conv_b[ch]);
-        for (int j = 0; j < p.taps - 1; ++j) {
-            const int q = pos - (p.taps - 1) + j;
-            if (q >= 0) acc = fmaf(p.conv_w[(size_t)ch * p.taps + j], ring[(size_t)(q % p.taps) * C + ch], acc);
+    const int channels = 2 * N + nc;
+    auto channel = [&](int i) {
+        return i < N ? inner + g * N + i : i < 2 * N ? inner + p.groups * N + g * N + (i - N) : head * V + c0 + (i - 2 * N);
+    };
+    for (int i0 = tid; i0 < channels; i0 += 2 * SD_THREADS) {   // two channels of a thread at a time
+        const int i1 = i0 + SD_THREADS;
+        const int ch0 = channel(i0), ch1 = i1 < channels ? channel(i1) : ch0;
+        const float own0 = p.xbc[row * p.ldx + ch0], own1 = p.xbc[row * p.ldx + ch1];
+        const float a0 = sd_conv<TAPS>(p, ring, ch0, pos, C, own0), a1 = i1 < channels ? sd_conv<TAPS>(p, ring, ch1, pos, C, own1) : 0.f;
+        // (B, C and x lie one behind the other)
+        Bs[i0] = a0;
+        if (i1 < channels) Bs[i1] = a1;
+        if (p.write_state) {
+            if (i0 >= 2 * N || keeps_bc) ring[(size_t)(pos % taps) * C + ch0] = own0;
+            if (i1 < channels && (i1 >= 2 * N || keeps_bc)) ring[(size_t)(pos % taps) * C + ch1] = own1;
         }
-        if (p.write_state && (i >= 2 * N || keeps_bc)) ring[(size_t)(pos % p.taps) * C + ch] = own;
-        (i < N ? Bs + i : i < 2 * N ? Cs + (i - N) : xs + (i - 2 * N))[0] = rc_silu(acc);
     }
-    const float dt = gb_softplus(p.dt_raw[row * p.ld_dt + head] + p.dt_bias[head]);
-    const float decay = expf(-expf(p.a_log[head]) * dt);
+    const float dt = gb_softplus(dt_raw);
+    const float decay = expf(-expf(rate) * dt);
     __syncthreads();
     float x[VEC], acc[VEC];
 #pragma unroll
@@ -305,8 +335,9 @@ __global__ void __launch_bounds__(SD_THREADS) ssd_decode_kernel(SsdDecodeArgs p)
     const int rows = min(par, N);
     for (int c = tid; c < nc; c += SD_THREADS) {
         float o = 0.f;
+#pragma unroll 8
         for (int r = 0; r < rows; ++r) o += part[r * nc + c];
-        p.y[row * inner + (size_t)head * V + c0 + c] = fmaf(p.skip[head], xs[c], o);
+        p.y[row * inner + (size_t)head * V + c0 + c] = fmaf(skip, xs[c], o);
     }
 }
 
@@ -331,8 +362,9 @@ GB_EXPORT int gb_ssd_decode(const float* xbc, long long ldx, const float* dt_raw
                        seq_start_pos, seq_slots, heads, groups, N, V, taps, num_slots, write_state, cols, status};
     const dim3 grid(S, heads, gb_ceil_div(V, cols));
     const size_t smem = ((size_t)2 * N + cols + 8 + SD_THREADS * (vec ? 4 : 1)) * sizeof(float);
-    if (vec) gb_launch(GB_PDL_ATTENTION, ssd_decode_kernel<4>, grid, dim3(SD_THREADS), smem, stream, p);
-    else gb_launch(GB_PDL_ATTENTION, ssd_decode_kernel<1>, grid, dim3(SD_THREADS), smem, stream, p);
+    if (vec && taps == 4) gb_launch(GB_PDL_ATTENTION, ssd_decode_kernel<4, 4>, grid, dim3(SD_THREADS), smem, stream, p);
+    else if (vec) gb_launch(GB_PDL_ATTENTION, ssd_decode_kernel<4, 0>, grid, dim3(SD_THREADS), smem, stream, p);
+    else gb_launch(GB_PDL_ATTENTION, ssd_decode_kernel<1, 0>, grid, dim3(SD_THREADS), smem, stream, p);
     return gb_check_launch("gb_ssd_decode");
 }
 
@@ -340,16 +372,20 @@ GB_EXPORT int gb_ssd_decode(const float* xbc, long long ldx, const float* dt_raw
 // Prompt portions in bfloat16. With c_i the running sum of the log decays inside a chunk of SC_L tokens (inclusive), S_0 the
 // state in front of the chunk and M_ij = (C_i . B_j) exp(c_i - c_j) dt_j for j <= i:
 //     y_i = exp(c_i) C_i S_0 + sum_j M_ij x_j + skip x_i,      S_end = exp(c_last) S_0 + sum_j exp(c_last - c_j) dt_j B_j x_j^T
-//   ssd_chunk_state   per (chunk, head): the chunk's own sum, from a zero state, and exp(c_last)
-//   ssd_chain         per element of S: through the request's chunks in order; a chunk's own sum is replaced by the state in
-//                     front of it, the request's slot receives the last state (float32)
+//   ssd_chunk_state   per (chunk, head): the chunk's own sum, from a zero state; dt_j and c_j
+//   ssd_chain         per element of S: through the request's chunks in order, in float32; a chunk's own sum is replaced by the
+//                     state in front of it, the request's slot receives the last state
 //   ssd_chunk_out     per (chunk, head): the read-outs
 // Logarithms of decays, their sums, exponentials and step sizes are float32. x, B and C are bfloat16 (the convolution's output);
 // what they are multiplied with (the weights of the chunk's sum, S_0, M) is float32 and enters the products as a sum of two
-// bfloat16 numbers, so that about 16 bits of it count.
+// bfloat16 numbers, so that about 16 bits of it count. S_0 is handed over in that form already, one 32-bit word per element
+// (the rounded value below, what the rounding left above it); as columns of a product the two halves of a word are neighbours,
+// so the two sums that belong to one element end up in one thread. The words of eight neighbouring channels lie in the order
+// 0 2 4 6 1 3 5 7: of two 8-column tiles the first then gives a thread an even channel and the second the odd one behind it,
+// which are the two channels that the thread holds of M x.
 // Chunk c of request s has the number seq_first_row[s] / SC_L + s + c: unique, and below n / SC_L + S.
 // ----------------------------------------------------------------------------------------------
-constexpr int SC_L = 64, SC_THREADS = 128;
+constexpr int SC_L = 64, SC_THREADS = 128, SC_OUT_THREADS = 256;
 
 struct SsdChunkArgs {
     const __nv_bfloat16* xbc;   // [n, ldx]: x | B | C after the convolution
@@ -363,7 +399,7 @@ struct SsdChunkArgs {
     long long state_stride;
     float* y;                   // [n, heads * V]
     float* chunk_state;         // [chunks, heads, N, V]
-    float* chunk_decay;         // [chunks, heads]
+    float* chunk_steps;         // [chunks, heads, 2, SC_L]: dt_j, c_j
     const int* seq_first_row;
     const int* seq_start_pos;
     const int* seq_slots;
@@ -430,20 +466,54 @@ __device__ __forceinline__ void ssd_split(float a, float b, unsigned& hi, unsign
     lo = *reinterpret_cast<const unsigned*>(&l);
 }
 
+__device__ __forceinline__ void ssd_cp16(void* smem, const void* gmem, bool valid) {
+    const unsigned a = (unsigned)__cvta_generic_to_shared(smem);
+    const int bytes = valid ? 16 : 0;        // 0: the 16 bytes are filled with zeros, nothing is read
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(a), "l"(gmem), "r"(bytes));
+}
+__device__ __forceinline__ void ssd_cp_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int LEFT>
+__device__ __forceinline__ void ssd_cp_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(LEFT) : "memory"); }
+
+__device__ __forceinline__ int ssd_word_at(int channel) { return (channel & ~7) + (channel & 1) * 4 + ((channel & 7) >> 1); }
+__device__ __forceinline__ unsigned ssd_word(float v) {
+    const __nv_bfloat16 h = __float2bfloat16_rn(v), l = __float2bfloat16_rn(v - __bfloat162float(h));
+    return (unsigned)__bfloat16_as_ushort(h) | ((unsigned)__bfloat16_as_ushort(l) << 16);
+}
+
+// A block's threads over the elements of a table of `width` columns: element threadIdx.x, then every blockDim.x-th (no division
+// inside the loop).
+struct SsdCells {
+    int r, c, dr, dc, width;
+    __device__ __forceinline__ explicit SsdCells(int w) : width(w) {
+        r = threadIdx.x / w;
+        c = threadIdx.x - r * w;
+        dr = blockDim.x / w;
+        dc = blockDim.x - dr * w;
+    }
+    __device__ __forceinline__ void next() {
+        r += dr;
+        c += dc;
+        if (c >= width) {
+            c -= width;
+            ++r;
+        }
+    }
+};
+
 // SC_L rows x `width` columns (of which `cols` exist, the rest and the rows behind the chunk's end are zero) into shared memory
 __device__ __forceinline__ void ssd_stage(__nv_bfloat16* dst, int ld, const __nv_bfloat16* src, long long lds, int rows, int cols, int width,
                                           bool vec) {
     const int pieces = width / 8;
     if (vec) {                   // (cols is then a multiple of 8 as well)
-        for (int i = threadIdx.x; i < SC_L * pieces; i += SC_THREADS) {
-            const int r = i / pieces, c = (i % pieces) * 8;
-            uint4 v = make_uint4(0u, 0u, 0u, 0u);
-            if (r < rows && c < cols) v = *reinterpret_cast<const uint4*>(src + (size_t)r * lds + c);
-            *reinterpret_cast<uint4*>(dst + r * ld + c) = v;
+        for (SsdCells at(pieces); at.r < SC_L; at.next()) {
+            const int r = at.r, c = at.c * 8;
+            const bool in = r < rows && c < cols;
+            ssd_cp16(dst + r * ld + c, in ? src + (size_t)r * lds + c : src, in);
         }
     } else {
-        for (int i = threadIdx.x; i < SC_L * width; i += SC_THREADS) {
-            const int r = i / width, c = i % width;
+        for (SsdCells at(width); at.r < SC_L; at.next()) {
+            const int r = at.r, c = at.c;
             dst[r * ld + c] = r < rows && c < cols ? src[(size_t)r * lds + c] : __float2bfloat16_rn(0.f);
         }
     }
@@ -461,34 +531,37 @@ __global__ void __launch_bounds__(SC_THREADS) ssd_chunk_state_kernel(SsdChunkArg
     __nv_bfloat16* Bs = reinterpret_cast<__nv_bfloat16*>(ssd_smem);      // [L][ldb]
     __nv_bfloat16* Xh = Bs + SC_L * ldb, *Xl = Xh + SC_L * ldv;           // [L][ldv]: exp(c_last - c_j) dt_j x_j in two parts
     const __nv_bfloat16* base = p.xbc + (size_t)c.row0 * p.ldx;
+    const __nv_bfloat16* xsrc = base + head * V;
+    if (p.vec) ssd_stage(Xh, ldv, xsrc, p.ldx, c.len, V, VW, true);
+    ssd_cp_commit();
     ssd_stage(Bs, ldb, base + inner + g * N, p.ldx, c.len, N, NW, p.vec);
+    ssd_cp_commit();
     ssd_steps(p, c, head, dt_s, cum_s, &half);
     const float last = cum_s[SC_L - 1];
-    const __nv_bfloat16* xsrc = base + head * V;
+    float* steps = p.chunk_steps + ((size_t)c.number * p.heads + head) * 2 * SC_L;
+    steps[threadIdx.x] = threadIdx.x < SC_L ? dt_s[threadIdx.x] : cum_s[threadIdx.x - SC_L];
+    ssd_cp_wait<1>();                        // (a thread reads back the pieces that it asked for itself)
     if (p.vec) {
-        const int pieces = VW / 8;
-        for (int i = threadIdx.x; i < SC_L * pieces; i += SC_THREADS) {
-            const int r = i / pieces, v = (i % pieces) * 8;
-            uint4 h = make_uint4(0u, 0u, 0u, 0u), l = h;
-            if (r < c.len && v < V) {
-                const uint4 raw = *reinterpret_cast<const uint4*>(xsrc + (size_t)r * p.ldx + v);
-                const float w = expf(last - cum_s[r]) * dt_s[r];
-                const __nv_bfloat162* q = reinterpret_cast<const __nv_bfloat162*>(&raw);
-                float2 f = __bfloat1622float2(q[0]);
-                ssd_split(f.x * w, f.y * w, h.x, l.x);
-                f = __bfloat1622float2(q[1]);
-                ssd_split(f.x * w, f.y * w, h.y, l.y);
-                f = __bfloat1622float2(q[2]);
-                ssd_split(f.x * w, f.y * w, h.z, l.z);
-                f = __bfloat1622float2(q[3]);
-                ssd_split(f.x * w, f.y * w, h.w, l.w);
-            }
+        for (SsdCells at(VW / 8); at.r < SC_L; at.next()) {
+            const int r = at.r, v = at.c * 8;
+            uint4 h, l;
+            const uint4 raw = *reinterpret_cast<const uint4*>(Xh + r * ldv + v);
+            const float w = expf(last - cum_s[r]) * dt_s[r];
+            const __nv_bfloat162* q = reinterpret_cast<const __nv_bfloat162*>(&raw);
+            float2 f = __bfloat1622float2(q[0]);
+            ssd_split(f.x * w, f.y * w, h.x, l.x);
+            f = __bfloat1622float2(q[1]);
+            ssd_split(f.x * w, f.y * w, h.y, l.y);
+            f = __bfloat1622float2(q[2]);
+            ssd_split(f.x * w, f.y * w, h.z, l.z);
+            f = __bfloat1622float2(q[3]);
+            ssd_split(f.x * w, f.y * w, h.w, l.w);
             *reinterpret_cast<uint4*>(Xh + r * ldv + v) = h;
             *reinterpret_cast<uint4*>(Xl + r * ldv + v) = l;
         }
     } else {
-        for (int i = threadIdx.x; i < SC_L * VW / 2; i += SC_THREADS) {
-            const int r = i / (VW / 2), v = (i % (VW / 2)) * 2;
+        for (SsdCells at(VW / 2); at.r < SC_L; at.next()) {
+            const int r = at.r, v = at.c * 2;
             const float w = expf(last - cum_s[r]) * dt_s[r];
             float a = 0.f, b = 0.f;
             if (r < c.len && v < V) a = __bfloat162float(xsrc[(size_t)r * p.ldx + v]) * w;
@@ -499,7 +572,7 @@ __global__ void __launch_bounds__(SC_THREADS) ssd_chunk_state_kernel(SsdChunkArg
             *reinterpret_cast<unsigned*>(Xl + r * ldv + v) = l;
         }
     }
-    if (threadIdx.x == 0) p.chunk_decay[(size_t)c.number * p.heads + head] = expf(last);
+    ssd_cp_wait<0>();
     __syncthreads();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int mt = NW / 16, vt = VW / 16;
@@ -567,13 +640,21 @@ __global__ void __launch_bounds__(256) ssd_chain_kernel(SsdChunkArgs p) {
         for (int u = 0; u < U; ++u) {
             const size_t at = (size_t)(lo + min(c0 + u, chunks - 1)) * p.heads + head;
             own[u] = *reinterpret_cast<const vec_t*>(p.chunk_state + at * numbers + e);
-            f[u] = p.chunk_decay[at];
+            f[u] = expf(p.chunk_steps[(at * 2 + 1) * SC_L + SC_L - 1]);
         }
+        __syncwarp();             // a thread's words go where its neighbour's sums were: both have read theirs
 #pragma unroll
         for (int u = 0; u < U; ++u) {
             if (c0 + u >= chunks) break;
             const size_t at = (size_t)(lo + c0 + u) * p.heads + head;
-            *reinterpret_cast<vec_t*>(p.chunk_state + at * numbers + e) = s;       // the state in front of this chunk
+            unsigned* words = reinterpret_cast<unsigned*>(p.chunk_state) + at * numbers;       // the state in front of this chunk
+            if constexpr (VEC == 4) {
+                unsigned* eight = words + (e & ~7) + ((e >> 2) & 1) * 2;
+                *reinterpret_cast<uint2*>(eight) = make_uint2(ssd_word(sf[0]), ssd_word(sf[2]));
+                *reinterpret_cast<uint2*>(eight + 4) = make_uint2(ssd_word(sf[1]), ssd_word(sf[3]));
+            } else {
+                words[e] = ssd_word(sf[0]);                      // (in order: whoever reads it puts the words in theirs)
+            }
             const float* of = reinterpret_cast<const float*>(&own[u]);
 #pragma unroll
             for (int i = 0; i < VEC; ++i) sf[i] = fmaf(f[u], sf[i], of[i]);
@@ -582,99 +663,107 @@ __global__ void __launch_bounds__(256) ssd_chain_kernel(SsdChunkArgs p) {
     if (p.write_state) *reinterpret_cast<vec_t*>(mine) = s;
 }
 
-__global__ void __launch_bounds__(SC_THREADS) ssd_chunk_out_kernel(SsdChunkArgs p) {
+// Eight warps: a warp has 16 of the chunk's tokens and every second tile of 16 value channels (the two warps of the same
+// tokens each form their C B^T).
+__global__ void __launch_bounds__(SC_OUT_THREADS) ssd_chunk_out_kernel(SsdChunkArgs p) {
     extern __shared__ __align__(16) unsigned char ssd_smem[];
-    __shared__ float dt_s[SC_L], cum_s[SC_L], half;
+    __shared__ __align__(16) float steps[2 * SC_L];
     gb_pdl_launch_dependents();
     gb_pdl_wait();
     SsdChunk c;
     if (!ssd_find_chunk(p, c)) return;
     const int head = blockIdx.y, g = head / (p.heads / p.groups), N = p.N, V = p.V, inner = p.heads * V;
-    const int NW = (N + 15) & ~15, VW = (V + 15) & ~15, ldb = NW + 8, ldv = VW + 8;
+    const int NW = (N + 15) & ~15, VW = (V + 15) & ~15, ldb = NW + 8, ldv = VW + 8, lds = 2 * VW + 8;
     __nv_bfloat16* Cs = reinterpret_cast<__nv_bfloat16*>(ssd_smem);      // [L][ldb]
     __nv_bfloat16* Bs = Cs + SC_L * ldb;                                  // [L][ldb]
     __nv_bfloat16* Xs = Bs + SC_L * ldb;                                  // [L][ldv]
-    __nv_bfloat16* Sh = Xs + SC_L * ldv, *Sl = Sh + NW * ldv;             // [NW][ldv]: S_0 in two parts
+    __nv_bfloat16* Ss = Xs + SC_L * ldv;                                  // [NW][lds]: the words of S_0
     const __nv_bfloat16* base = p.xbc + (size_t)c.row0 * p.ldx;
+    const size_t number = (size_t)c.number * p.heads + head;
     ssd_stage(Cs, ldb, base + inner + p.groups * N + g * N, p.ldx, c.len, N, NW, p.vec);
     ssd_stage(Bs, ldb, base + inner + g * N, p.ldx, c.len, N, NW, p.vec);
+    if (threadIdx.x < SC_L / 2) ssd_cp16(steps + threadIdx.x * 4, p.chunk_steps + number * 2 * SC_L + threadIdx.x * 4, true);
+    ssd_cp_commit();
     ssd_stage(Xs, ldv, base + head * V, p.ldx, c.len, V, VW, p.vec);
-    const float* S0 = p.chunk_state + ((size_t)c.number * p.heads + head) * N * V;
+    const unsigned* S0 = reinterpret_cast<const unsigned*>(p.chunk_state) + number * N * V;
     if (p.vec) {
-        for (int i = threadIdx.x; i < NW * (VW / 4); i += SC_THREADS) {
-            const int r = i / (VW / 4), v = (i % (VW / 4)) * 4;
-            float4 f = make_float4(0.f, 0.f, 0.f, 0.f);
-            if (r < N && v < V) f = *reinterpret_cast<const float4*>(S0 + (size_t)r * V + v);
-            uint2 h, l;
-            ssd_split(f.x, f.y, h.x, l.x);
-            ssd_split(f.z, f.w, h.y, l.y);
-            *reinterpret_cast<uint2*>(Sh + r * ldv + v) = h;
-            *reinterpret_cast<uint2*>(Sl + r * ldv + v) = l;
+        for (SsdCells at(VW / 4); at.r < NW; at.next()) {
+            const int r = at.r, v = at.c * 4;
+            const bool in = r < N && v < V;
+            ssd_cp16(Ss + r * lds + 2 * v, in ? S0 + (size_t)r * V + v : S0, in);
         }
     } else {
-        for (int i = threadIdx.x; i < NW * (VW / 2); i += SC_THREADS) {
-            const int r = i / (VW / 2), v = (i % (VW / 2)) * 2;
-            const float a = r < N && v < V ? S0[(size_t)r * V + v] : 0.f, b = r < N && v + 1 < V ? S0[(size_t)r * V + v + 1] : 0.f;
-            unsigned h, l;
-            ssd_split(a, b, h, l);
-            *reinterpret_cast<unsigned*>(Sh + r * ldv + v) = h;
-            *reinterpret_cast<unsigned*>(Sl + r * ldv + v) = l;
+        for (SsdCells at(VW); at.r < NW; at.next()) {
+            const int r = at.r, v = at.c;
+            reinterpret_cast<unsigned*>(Ss + r * lds)[ssd_word_at(v)] = r < N && v < V ? S0[(size_t)r * V + v] : 0u;
         }
     }
-    ssd_steps(p, c, head, dt_s, cum_s, &half);        // (its barriers also cover the staging)
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    ssd_cp_commit();
+    ssd_cp_wait<1>();
+    __syncthreads();
+    const int warp = (threadIdx.x >> 5) & 3, v0 = threadIdx.x >> 7, lane = threadIdx.x & 31;
     const int i0 = warp * 16;                          // this warp's 16 tokens
-    if (i0 >= c.len) return;
     const int kn = NW / 16;
+    const bool busy = i0 < c.len;
     const __nv_bfloat16* crow = Cs + (i0 + (lane & 15)) * ldb + (lane >> 4) * 8;
-    // C_i . B_j for the tokens up to this warp's last
-    float s[SC_L / 8][4];
-#pragma unroll
-    for (int j = 0; j < SC_L / 8; ++j) s[j][0] = s[j][1] = s[j][2] = s[j][3] = 0.f;
-    for (int k = 0; k < kn; ++k) {
-        unsigned a[4];
-        ssd_ldm(a, crow + k * 16);
-#pragma unroll
-        for (int j2 = 0; j2 < SC_L / 16; ++j2) {
-            if (j2 > warp) break;
-            unsigned b[4];
-            ssd_ldm(b, Bs + (j2 * 16 + (lane & 7) + ((lane >> 4) << 3)) * ldb + k * 16 + ((lane >> 3) & 1) * 8);
-            ssd_mma(s[2 * j2], a, b[0], b[1]);
-            ssd_mma(s[2 * j2 + 1], a, b[2], b[3]);
-        }
-    }
-    // M in two parts, as the A operand of M x
+    const float* dt_s = steps, *cum_s = steps + SC_L;
     const int ia = i0 + (lane >> 2), ib = ia + 8;
     const float ca = cum_s[ia], cb = cum_s[ib];
     unsigned mh[SC_L / 16][4], ml[SC_L / 16][4];
+    if (busy) {
+        // C_i . B_j for the tokens up to this warp's last
+        float s[SC_L / 8][4];
 #pragma unroll
-    for (int j = 0; j < SC_L / 8; ++j) {
-        if ((j >> 1) > warp) break;
-        const int t0 = j * 8 + (lane & 3) * 2, t1 = t0 + 1;
-        const float d0 = dt_s[t0], d1 = dt_s[t1], c0 = cum_s[t0], c1 = cum_s[t1];
-        const float w0 = t0 <= ia ? s[j][0] * (expf(ca - c0) * d0) : 0.f, w1 = t1 <= ia ? s[j][1] * (expf(ca - c1) * d1) : 0.f;
-        const float w2 = t0 <= ib ? s[j][2] * (expf(cb - c0) * d0) : 0.f, w3 = t1 <= ib ? s[j][3] * (expf(cb - c1) * d1) : 0.f;
-        ssd_split(w0, w1, mh[j >> 1][(j & 1) * 2], ml[j >> 1][(j & 1) * 2]);
-        ssd_split(w2, w3, mh[j >> 1][(j & 1) * 2 + 1], ml[j >> 1][(j & 1) * 2 + 1]);
-    }
-    const float fa = expf(ca), fb = expf(cb), skip = p.skip[head];
-    for (int v = 0; v < VW / 16; ++v) {
-        float acc[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
-        for (int k = 0; k < kn; ++k) {                 // C S_0
-            unsigned a[4], h[4], l[4];
+        for (int j = 0; j < SC_L / 8; ++j) s[j][0] = s[j][1] = s[j][2] = s[j][3] = 0.f;
+        for (int k = 0; k < kn; ++k) {
+            unsigned a[4];
             ssd_ldm(a, crow + k * 16);
-            const int at = (k * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * ldv + v * 16 + (lane >> 4) * 8;
-            ssd_ldm_t(h, Sh + at);
-            ssd_ldm_t(l, Sl + at);
-            ssd_mma(acc[0], a, h[0], h[1]);
-            ssd_mma(acc[1], a, h[2], h[3]);
-            ssd_mma(acc[0], a, l[0], l[1]);
-            ssd_mma(acc[1], a, l[2], l[3]);
+#pragma unroll
+            for (int j2 = 0; j2 < SC_L / 16; ++j2) {
+                if (j2 > warp) break;
+                unsigned b[4];
+                ssd_ldm(b, Bs + (j2 * 16 + (lane & 7) + ((lane >> 4) << 3)) * ldb + k * 16 + ((lane >> 3) & 1) * 8);
+                ssd_mma(s[2 * j2], a, b[0], b[1]);
+                ssd_mma(s[2 * j2 + 1], a, b[2], b[3]);
+            }
         }
+        // M in two parts, as the A operand of M x
+#pragma unroll
+        for (int j = 0; j < SC_L / 8; ++j) {
+            if ((j >> 1) > warp) break;
+            const int t0 = j * 8 + (lane & 3) * 2, t1 = t0 + 1;
+            const float d0 = dt_s[t0], d1 = dt_s[t1], c0 = cum_s[t0], c1 = cum_s[t1];
+            const float w0 = t0 <= ia ? s[j][0] * (__expf(ca - c0) * d0) : 0.f, w1 = t1 <= ia ? s[j][1] * (__expf(ca - c1) * d1) : 0.f;
+            const float w2 = t0 <= ib ? s[j][2] * (__expf(cb - c0) * d0) : 0.f, w3 = t1 <= ib ? s[j][3] * (__expf(cb - c1) * d1) : 0.f;
+            ssd_split(w0, w1, mh[j >> 1][(j & 1) * 2], ml[j >> 1][(j & 1) * 2]);
+            ssd_split(w2, w3, mh[j >> 1][(j & 1) * 2 + 1], ml[j >> 1][(j & 1) * 2 + 1]);
+        }
+    }
+    ssd_cp_wait<0>();
+    __syncthreads();
+    if (!busy) return;
+    const float fa = __expf(ca), fb = __expf(cb), skip = p.skip[head];
+    for (int v = v0; v < VW / 16; v += 2) {
+        float w[4][4];                                 // C S_0: four tiles of words, each an 8-column half of 16 channels
+#pragma unroll
+        for (int j = 0; j < 4; ++j) w[j][0] = w[j][1] = w[j][2] = w[j][3] = 0.f;
+#pragma unroll 4
+        for (int k = 0; k < kn; ++k) {
+            unsigned a[4], b0[4], b1[4];
+            ssd_ldm(a, crow + k * 16);
+            const __nv_bfloat16* srow = Ss + (k * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * lds + v * 32 + (lane >> 4) * 8;
+            ssd_ldm_t(b0, srow);
+            ssd_ldm_t(b1, srow + 16);
+            ssd_mma(w[0], a, b0[0], b0[1]);
+            ssd_mma(w[1], a, b0[2], b0[3]);
+            ssd_mma(w[2], a, b1[0], b1[1]);
+            ssd_mma(w[3], a, b1[2], b1[3]);
+        }
+        float acc[2][4];
 #pragma unroll
         for (int j = 0; j < 2; ++j) {
-            acc[j][0] *= fa; acc[j][1] *= fa;
-            acc[j][2] *= fb; acc[j][3] *= fb;
+            acc[j][0] = fa * (w[2 * j][0] + w[2 * j][1]); acc[j][1] = fa * (w[2 * j + 1][0] + w[2 * j + 1][1]);
+            acc[j][2] = fb * (w[2 * j][2] + w[2 * j][3]); acc[j][3] = fb * (w[2 * j + 1][2] + w[2 * j + 1][3]);
         }
 #pragma unroll
         for (int k = 0; k < SC_L / 16; ++k) {          // + M x
@@ -692,8 +781,8 @@ __global__ void __launch_bounds__(SC_THREADS) ssd_chunk_out_kernel(SsdChunkArgs 
             for (int hf = 0; hf < 2; ++hf) {
                 const int i = hf ? ib : ia, col = v * 16 + j * 8 + (lane & 3) * 2;
                 if (i >= c.len) continue;
-                const float y0 = fmaf(skip, __bfloat162float(Xs[i * ldv + col]), acc[j][hf * 2]);
-                const float y1 = fmaf(skip, __bfloat162float(Xs[i * ldv + col + 1]), acc[j][hf * 2 + 1]);
+                const __nv_bfloat162 x = *reinterpret_cast<const __nv_bfloat162*>(Xs + i * ldv + col);
+                const float y0 = fmaf(skip, __low2float(x), acc[j][hf * 2]), y1 = fmaf(skip, __high2float(x), acc[j][hf * 2 + 1]);
                 float* o = p.y + (size_t)(c.row0 + i) * inner + (size_t)head * V + col;
                 if (col + 1 < V && (V & 1) == 0) *reinterpret_cast<float2*>(o) = make_float2(y0, y1);
                 else {
@@ -706,30 +795,31 @@ __global__ void __launch_bounds__(SC_THREADS) ssd_chunk_out_kernel(SsdChunkArgs 
 
 static size_t ssd_out_smem(int N, int V) {
     const int NW = (N + 15) & ~15, VW = (V + 15) & ~15;
-    return ((size_t)2 * SC_L * (NW + 8) + (size_t)SC_L * (VW + 8) + (size_t)2 * NW * (VW + 8)) * 2;
+    return ((size_t)2 * SC_L * (NW + 8) + (size_t)SC_L * (VW + 8) + (size_t)NW * (2 * VW + 8)) * 2;
 }
 
 GB_EXPORT int gb_ssd_chunk_rows() { return SC_L; }
 // 1 if the chunked form takes these sizes
 GB_EXPORT int gb_ssd_chunks_supported(int N, int V) { return N > 0 && V > 0 && N <= 256 && ssd_out_smem(N, V) <= 200 * 1024 ? 1 : 0; }
 
-// chunk_state: float32 [chunks, heads * N * V], chunk_decay: float32 [chunks, heads], chunks at least n / SC_L + S.
+// chunk_state: float32 [chunks, heads * N * V], chunk_steps: float32 [chunks, heads * 2 * SC_L], chunks at least n / SC_L + S.
 GB_EXPORT int gb_ssd_chunks(const void* xbc, long long ldx, const float* dt_raw, long long ld_dt, const float* dt_bias, const float* a_log,
                             const float* skip, float* state, long long state_stride, float* y, const int* seq_first_row,
                             const int* seq_start_pos, const int* seq_slots, int S, int n, int max_rows_per_seq, int heads, int groups, int N,
-                            int V, int num_slots, int write_state, int chunks, float* chunk_state, float* chunk_decay, int* status,
+                            int V, int num_slots, int write_state, int chunks, float* chunk_state, float* chunk_steps, int* status,
                             cudaStream_t stream) {
     GB_REQUIRE(S >= 0 && n >= 0 && heads > 0 && groups > 0 && heads % groups == 0, "gb_ssd_chunks: heads %d must be a multiple of groups %d",
                heads, groups);
     GB_REQUIRE(gb_ssd_chunks_supported(N, V), "gb_ssd_chunks: state size %d and value size %d are not built", N, V);
-    GB_REQUIRE(chunks >= n / SC_L + S && chunk_state && chunk_decay && max_rows_per_seq > 0, "gb_ssd_chunks: %d chunks are too few for %d rows of %d requests",
+    GB_REQUIRE(chunks >= n / SC_L + S && chunk_state && chunk_steps && max_rows_per_seq > 0, "gb_ssd_chunks: %d chunks are too few for %d rows of %d requests",
                chunks, n, S);
     if (S == 0 || n == 0) return 0;
     const int tiles = gb_ceil_div(max_rows_per_seq, SC_L);
     const int NW = (N + 15) & ~15, VW = (V + 15) & ~15;
     const int vec = N % 8 == 0 && V % 8 == 0 && ldx % 8 == 0 && (heads * V) % 8 == 0 && ((uintptr_t)xbc & 15) == 0 &&
-                    ((uintptr_t)chunk_state & 15) == 0;
-    SsdChunkArgs p = {(const __nv_bfloat16*)xbc, ldx, dt_raw, ld_dt, dt_bias, a_log, skip, state, state_stride, y, chunk_state, chunk_decay,
+                    (((uintptr_t)chunk_state | (uintptr_t)chunk_steps | (uintptr_t)state) & 15) == 0 && state_stride % 4 == 0;
+    GB_REQUIRE(((uintptr_t)chunk_steps & 15) == 0, "gb_ssd_chunks: the steps' buffer must be 16-byte aligned");
+    SsdChunkArgs p = {(const __nv_bfloat16*)xbc, ldx, dt_raw, ld_dt, dt_bias, a_log, skip, state, state_stride, y, chunk_state, chunk_steps,
                       seq_first_row, seq_start_pos, seq_slots, S, tiles, heads, groups, N, V, num_slots, write_state, vec, status};
     const size_t smem_state = ((size_t)SC_L * (NW + 8) + (size_t)2 * SC_L * (VW + 8)) * 2, smem_out = ssd_out_smem(N, V);
     cudaFuncSetAttribute(ssd_chunk_state_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem_state);
@@ -737,11 +827,10 @@ GB_EXPORT int gb_ssd_chunks(const void* xbc, long long ldx, const float* dt_raw,
     gb_launch(GB_PDL_ATTENTION, ssd_chunk_state_kernel, dim3(S * tiles, heads), dim3(SC_THREADS), smem_state, stream, p);
     int rc = gb_check_launch("gb_ssd_chunks (state)");
     if (rc) return rc;
-    const bool v4 = (N * V) % 4 == 0 && state_stride % 4 == 0 && (((uintptr_t)state | (uintptr_t)chunk_state) & 15) == 0;
-    if (v4) gb_launch(GB_PDL_ATTENTION, ssd_chain_kernel<4>, dim3(S, heads, gb_ceil_div((long long)N * V, 1024)), dim3(256), 0, stream, p);
+    if (vec) gb_launch(GB_PDL_ATTENTION, ssd_chain_kernel<4>, dim3(S, heads, gb_ceil_div((long long)N * V, 1024)), dim3(256), 0, stream, p);
     else gb_launch(GB_PDL_ATTENTION, ssd_chain_kernel<1>, dim3(S, heads, gb_ceil_div((long long)N * V, 256)), dim3(256), 0, stream, p);
     rc = gb_check_launch("gb_ssd_chunks (chain)");
     if (rc) return rc;
-    gb_launch(GB_PDL_ATTENTION, ssd_chunk_out_kernel, dim3(S * tiles, heads), dim3(SC_THREADS), smem_out, stream, p);
+    gb_launch(GB_PDL_ATTENTION, ssd_chunk_out_kernel, dim3(S * tiles, heads), dim3(SC_OUT_THREADS), smem_out, stream, p);
     return gb_check_launch("gb_ssd_chunks (out)");
 }

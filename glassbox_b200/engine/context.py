@@ -118,7 +118,8 @@ class StepContext:
         self.token_slots = None           # int32 [rows]: state slot of the rows whose token the device supplies itself, else -1
         self.want_slots = None            # int32 [wanted rows]: state slot of the rows that are sampled from their own state, else -1
         self.weight_order: Optional[WeightOrder] = None
-        self.side_stream = None           # a second CUDA stream for work beside the main chain (prefetch)
+        self.side_stream = None           # a second CUDA stream for work beside the main chain (prefetch, one of two mixers)
+        self.scratch_prefix = ""          # set while a part runs on the second stream: its buffers must be its own
         self.program = None               # a kernels.Program: decode steps of few rows run as one persistent kernel
         # An RMSNorm may be split between the product that completes the residual rows and the product that reads
         # the normalised rows (parts/linear.py). Whoever wires the parts says which norm comes next:
@@ -144,10 +145,10 @@ class StepContext:
         self.normed_pair = None
 
     def scratch(self, name: str, shape, dtype: Optional[torch.dtype] = None, grow: bool = False) -> torch.Tensor:
-        return (self._grow if grow else self._scratch).get(name, shape, dtype, grow)
+        return (self._grow if grow else self._scratch).get(self.scratch_prefix + name, shape, dtype, grow)
 
     def zeros_once(self, name: str, count: int, dtype: torch.dtype) -> torch.Tensor:
-        return self._scratch.zeros_once(name, count, dtype)
+        return self._scratch.zeros_once(self.scratch_prefix + name, count, dtype)
 
     @property
     def max_rows(self) -> int:

@@ -1259,27 +1259,32 @@ def ssd_chunks_supported(dtype: torch.dtype, n_state: int, vdim: int) -> bool:
     return dtype == torch.bfloat16 and bool(lib().gb_ssd_chunks_supported(n_state, vdim))
 
 
+def ssd_chunk_rows() -> int:
+    """Tokens of a chunk."""
+    return lib().gb_ssd_chunk_rows()
+
+
 def ssd_chunks_needed(n: int, num_seqs: int) -> int:
     """How many chunks ``ssd_chunks`` may need for a step of ``n`` rows in ``num_seqs`` sequences."""
-    return n // lib().gb_ssd_chunk_rows() + num_seqs
+    return n // ssd_chunk_rows() + num_seqs
 
 
 def ssd_chunks(xbc: torch.Tensor, dt_raw: torch.Tensor, dt_bias: torch.Tensor, a_log: torch.Tensor, skip: torch.Tensor,
                state: torch.Tensor, y: torch.Tensor, seq_first_row: torch.Tensor, seq_start_pos: torch.Tensor, seq_slots: torch.Tensor,
                max_rows_per_seq: int, heads: int, groups: int, n_state: int, vdim: int, write_state: bool, status: torch.Tensor,
-               chunk_state: torch.Tensor, chunk_decay: torch.Tensor) -> None:
+               chunk_state: torch.Tensor, chunk_steps: torch.Tensor) -> None:
     """``ssd_walk`` in chunks that run side by side on the tensor cores; ``xbc`` bfloat16 after its convolution. The chunks' own
     sums are chained afterwards (float32), then every chunk's read-outs are formed. ``chunk_state`` float32 [chunks, heads *
-    n_state * vdim] and ``chunk_decay`` float32 [chunks, heads] are scratch, chunks = ``ssd_chunks_needed``."""
-    _cuda(xbc, dt_raw, dt_bias, a_log, skip, state, y, seq_first_row, seq_start_pos, seq_slots, status, chunk_state, chunk_decay)
+    n_state * vdim] and ``chunk_steps`` float32 [chunks, heads * 2 * chunk rows] are scratch, chunks = ``ssd_chunks_needed``."""
+    _cuda(xbc, dt_raw, dt_bias, a_log, skip, state, y, seq_first_row, seq_start_pos, seq_slots, status, chunk_state, chunk_steps)
     _ssd_check(xbc, dt_raw, dt_bias, a_log, skip, state, y, heads, groups, n_state, vdim)
     n, S, chunks = xbc.shape[0], seq_start_pos.shape[0], chunk_state.shape[0]
-    assert xbc.dtype == torch.bfloat16 and chunk_state.dtype == chunk_decay.dtype == torch.float32
-    assert chunk_state.shape == (chunks, heads * n_state * vdim) and chunk_state.is_contiguous() and chunk_decay.is_contiguous()
-    assert chunk_decay.numel() >= chunks * heads and chunks >= ssd_chunks_needed(n, S)
+    assert xbc.dtype == torch.bfloat16 and chunk_state.dtype == chunk_steps.dtype == torch.float32
+    assert chunk_state.shape == (chunks, heads * n_state * vdim) and chunk_state.is_contiguous() and chunk_steps.is_contiguous()
+    assert chunk_steps.numel() >= chunks * heads * 2 * ssd_chunk_rows() and chunks >= ssd_chunks_needed(n, S)
     _call("gb_ssd_chunks", _ptr(xbc), xbc.stride(0), _ptr(dt_raw), dt_raw.stride(0), _ptr(dt_bias), _ptr(a_log), _ptr(skip), _ptr(state),
           state.stride(0), _ptr(y), _ptr(seq_first_row), _ptr(seq_start_pos), _ptr(seq_slots), S, n, max(int(max_rows_per_seq), 1), heads,
-          groups, n_state, vdim, state.shape[0], 1 if write_state else 0, chunks, _ptr(chunk_state), _ptr(chunk_decay), _ptr(status),
+          groups, n_state, vdim, state.shape[0], 1 if write_state else 0, chunks, _ptr(chunk_state), _ptr(chunk_steps), _ptr(status),
           _stream())
     global launch_count
     launch_count += 2

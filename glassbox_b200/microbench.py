@@ -30,6 +30,9 @@ over operands that rotate through more memory than L2 holds.
     python -m glassbox_b200.microbench babotar                           Babotar's kernels, each beside its like kernel: talking-heads
                                                                          attention, lightning attention and the delta rule with one decay
                                                                          per head, the input convolution, the GELU unit in the products
+    python -m glassbox_b200.microbench felovik                           Felovik's kernels, each beside its like kernel: attention with a
+                                                                         gate per channel, the state-space mixer, the norm after the sum,
+                                                                         the router and the SwiGLU experts
 
 Prints one line per case: microseconds and GB/s or TFLOP/s of the algorithmic bytes or flops. With ``--once`` after
 the case's name every kernel is launched exactly once and nothing is timed: the form in which a profiler captures one
@@ -885,7 +888,177 @@ def bench_layer_gemms(rows) -> None:
     kernels.check_status(st)
 
 
-CASES = ("gemm_stream", "gemm_tc", "attention_decode", "attention_splits", "attention_prefill", "float32", "small", "decode_program", "layer_gemms", "latent_attention", "delta_rule", "lonorax", "tagenex", "babotar")
+def bench_felovik() -> None:
+    """Each kernel of the Felovik path beside the like kernel of the closest path, at the sizes of the width-1024 and width-2048
+    models that ``bench.py --workload felovik`` runs."""
+    status = torch.zeros(1, dtype=torch.int32, device=DEV)
+    ps, hd, t_len, ctx = 16, 64, 2048, 4096
+    for d, H, G in ((1024, 16, 4), (2048, 32, 8)):
+        per = t_len // ps
+        kc = torch.randn(per + 2, G, ps, hd, device=DEV).bfloat16()
+        vc = torch.randn_like(kc)
+        tables = torch.arange(per, dtype=torch.int32, device=DEV).view(1, per).contiguous()
+        first = torch.tensor([0, t_len], dtype=torch.int32, device=DEV)
+        start = torch.zeros(1, dtype=torch.int32, device=DEV)
+        pos = torch.arange(t_len, dtype=torch.int32, device=DEV)
+        q = torch.randn(t_len, H * hd, device=DEV).bfloat16()
+        o = torch.empty_like(q)
+        gate, head_gate, sink = torch.randn(t_len, H * hd, device=DEV), torch.randn(t_len, H, device=DEV), torch.zeros(H, device=DEV)
+        r1, r2 = torch.full((H,), 0.5, device=DEV), torch.full((H,), 0.3, device=DEV)
+        fl = 2.0 * (t_len * (t_len + 1) // 2) * H * 2 * hd
+        for name, terms in (("a gate per channel", (None, None, None, gate)), ("   distance bias, sink and a gate per head", (r1, r2, sink, head_gate)),
+                            ("   grouped-query", None)):
+            t = graph_time(lambda: kernels.attention_prefill_tc(q, o, kc, vc, tables, first, start, t_len, H, G, hd, ps, hd ** -0.5, None, status,
+                                                                sink_terms=terms), reps=4)
+            print(f"{name}: prompt attention (tcgen05) heads {H}/{G} x {hd}, {t_len} tokens: {t:7.1f} us {fl / t / 1e6:6.1f} TFLOP/s", flush=True)
+        for m in (1, 8, 64):
+            per = ctx // ps
+            kd = torch.randn(m * per + 4, G, ps, hd, device=DEV).bfloat16()
+            vd = torch.randn_like(kd)
+            tb = torch.arange(m * per, dtype=torch.int32, device=DEV).view(m, per).contiguous()
+            row_seq = torch.arange(m, dtype=torch.int32, device=DEV)
+            pd = torch.full((m,), ctx - 1, dtype=torch.int32, device=DEV)
+            qd, od = torch.randn(m, H * hd, device=DEV).bfloat16(), torch.empty(m, H * hd, device=DEV).bfloat16()
+            nbytes = m * ctx * G * hd * 2 * 2
+            sp, block_keys, warps = kernels.decode_mma_plan(m, G, hd, ctx)
+            pa = torch.empty(m * H * warps * sp * hd, device=DEV)
+            pm = torch.empty(m * H * warps * sp * 2, device=DEV)
+            cn = torch.zeros(m * G, dtype=torch.int32, device=DEV)
+            for name, terms in (("a gate per channel", (None, None, None, gate[:m])), ("   grouped-query", None)):
+                t = graph_time(lambda: kernels.attention_decode_mma(qd, od, kd, vd, tb, row_seq, pd, H, G, hd, ps, hd ** -0.5, None, sp, pa, pm, cn,
+                                                                    status, block_keys, warps, sink_terms=terms))
+                print(f"{name}: decode attention heads {H}/{G} x {hd} batch {m:3d} context {ctx}: {t:7.1f} us {nbytes / t / 1e3:6.0f} GB/s", flush=True)
+        cols = (H + 2 * G) * hd
+        for n in (t_len, 8):
+            proj, qo, p = torch.randn(n, cols, device=DEV), torch.empty(n, H * hd, device=DEV).bfloat16(), pos[:n]
+            t = graph_time(lambda: kernels.qk_norm_rope_write(proj, None, None, None, p, p, qo, kc, vc, H, G, hd, hd, 0, 1e-6, ps, True, status,
+                                                              unit_norm=True, q_temp=(0.1, 1024)))
+            g = torch.ones(hd, device=DEV)
+            t2 = graph_time(lambda: kernels.qk_norm_rope_write(proj, g, g, None, p, p, qo, kc, vc, H, G, hd, hd, 0, 1e-6, ps, True, status))
+            print(f"unit norm + temperature + cache write heads {H}/{G}, {n:4d} rows: {t:6.1f} us {n * cols * 6 / t / 1e3:6.0f} GB/s; "
+                  f"norm with gains + cache write {t2:6.1f} us", flush=True)
+        # the joins: a stored branch, a routed feed-forward in its parts, two normed branches, beside the branch norm of Tagenex
+        for n in (t_len, 8):
+            x, y, z, w = (torch.randn(n, d, device=DEV) for _ in range(4))
+            w, h, pos_n = w[0].contiguous(), torch.empty(n, d, device=DEV).bfloat16(), pos[:n]
+            pair, weight = torch.randn(n, 4 * d, device=DEV), torch.rand(n, 4, device=DEV)
+            rows = (("stored", y, 14), ("weighted sum of 4", kernels.WeightedRows(pair, weight), 26),
+                    ("two normed", kernels.NormedPair(y, z, w, w, 0.5, 0.5, 1e-6), 18))
+            for name, branch, b in rows:
+                t = graph_time(lambda: kernels.post_norm(x, w, 2.0, 1e-6, branch, positions=pos_n, copy=h))
+                print(f"norm after the sum ({name}) {d}, {n:4d} rows: {t:6.1f} us {n * d * b / t / 1e3:6.0f} GB/s", flush=True)
+            t = graph_time(lambda: kernels.rmsnorm_add(y, w, x, 1e-6, copy=h))
+            print(f"   branch norm into the residual {d}, {n:4d} rows: {t:6.1f} us {n * d * 14 / t / 1e3:6.0f} GB/s", flush=True)
+        # the state-space mixer: inner width 2 d, heads of 64 channels, state 128
+        SH, SG, N, V, taps = 2 * d // 64, 2 * d // 1024, 128, 64, 4
+        inner, C = SH * V, SH * V + 2 * SG * N
+        wc, bc = torch.randn(C, taps, device=DEV), torch.randn(C, device=DEV)
+        dtb, al, sk = torch.full((SH,), -2.0, device=DEV), torch.zeros(SH, device=DEV), torch.ones(SH, device=DEV)
+        numbers = SH * N * V
+        for n, S in ((2048, 1), (1, 1), (8, 8), (64, 64)):
+            per = n // S
+            proj = torch.randn(n, inner + C + SH, device=DEV)
+            xbc, dt = proj[:, inner:inner + C], proj[:, inner + C:]
+            first = torch.arange(0, n + 1, per, dtype=torch.int32, device=DEV)
+            start = torch.full((S,), 100, dtype=torch.int32, device=DEV)
+            slots = torch.arange(S, dtype=torch.int32, device=DEV)
+            row_seq = (torch.arange(n, device=DEV) // per).int()
+            states = [torch.zeros(S, numbers + taps * C, device=DEV) for _ in range(max(1, min(8, int(2 * L2_BYTES / (S * numbers * 4)))))]
+            y = torch.empty(n, inner, device=DEV)
+            turn = [0]
+            if per == 1:
+                def fn():
+                    turn[0] += 1
+                    kernels.ssd_decode(xbc, dt, wc, bc, dtb, al, sk, states[turn[0] % len(states)], numbers, y, first, start, slots, SH, SG, N, V,
+                                       True, status)
+                t = graph_time(fn)
+                nb = 2.0 * S * numbers * 4
+                print(f"state space single tokens heads {SH} x {N} x {V}, {S:2d} requests: {t:7.1f} us {nb / t / 1e3:6.0f} GB/s", flush=True)
+                DH = numbers // (128 * 128)
+                qkv, beta, a = torch.randn(n, 3 * DH * 128, device=DEV), torch.randn(n, DH, device=DEV), torch.randn(n, DH, device=DEV)
+                gt, att, w1 = torch.randn(n, DH * 128, device=DEV), torch.empty(n, DH * 128, device=DEV).bfloat16(), torch.ones(128, device=DEV)
+
+                def like():
+                    turn[0] += 1
+                    kernels.channel_delta_decode(qkv, beta, a, dtb[:DH].contiguous(), al[:DH].contiguous(), states[turn[0] % len(states)], gt, w1, 1e-6,
+                                                 att, first, start, slots, DH, DH, 128, 128, True, status, decay_per_head=True, gate_silu=True)
+                t = graph_time(like)
+                print(f"   delta rule (one decay per head) of as many state numbers, {DH} x 128 x 128: {t:7.1f} us {nb / t / 1e3:6.0f} GB/s", flush=True)
+            else:
+                act = torch.empty(n, C, device=DEV).bfloat16()
+                t = graph_time(lambda: kernels.ring_conv(xbc, wc, bc, act, states[0], numbers, row_seq, pos, first, start, slots, True, status))
+                print(f"convolution over a ring {n} x {C}: {t:7.1f} us {n * C * 6 / t / 1e3:6.0f} GB/s", flush=True)
+                f32 = torch.empty(n, C, device=DEV)
+                st3 = torch.zeros(1, 3 * C, device=DEV)
+                t = graph_time(lambda: kernels.short_conv(xbc, wc, f32, st3, 0, row_seq, pos, first, start, slots, True, status))
+                print(f"   the delta rule's convolution: {t:7.1f} us {n * C * 8 / t / 1e3:6.0f} GB/s", flush=True)
+                chunks = kernels.ssd_chunks_needed(n, S)
+                own, steps = torch.empty(chunks, numbers, device=DEV), torch.empty(chunks, SH * 2 * kernels.ssd_chunk_rows(), device=DEV)
+                args = (dt, dtb, al, sk, states[0], y, first, start, slots)
+                t = graph_time(lambda: kernels.ssd_chunks(act, *args, per, SH, SG, N, V, True, status, own, steps), reps=4)
+                # C B^T and M x below the diagonal, C S_0, the chunk's own sum: multiply-adds of the chunked form at 64 tokens a chunk
+                fl = 2.0 * n * SH * (64 / 2 * (N + V) + 2 * N * V)
+                nb = n * (C * 2 + SH * 4 + inner * 4)
+                print(f"state space prompt in chunks, heads {SH} x {N} x {V}, {n} tokens: {t:7.1f} us = {t / n:6.4f} us per token, {fl / t / 1e6:6.1f} TFLOP/s, "
+                      f"{nb / t / 1e3:6.0f} GB/s of inputs and outputs", flush=True)
+                t = graph_time(lambda: kernels.ssd_walk(f32, *args, SH, SG, N, V, True, status), reps=2)
+                print(f"   token by token (float32): {t:7.1f} us = {t / n:6.4f} us per token", flush=True)
+                DH = numbers // (128 * 128)
+                qkv, beta, a = torch.randn(n, 3 * DH * 128, device=DEV), torch.randn(n, DH, device=DEV), torch.randn(n, DH, device=DEV)
+                od = torch.empty(n, DH * 128, device=DEV)
+                t = graph_time(lambda: kernels.channel_delta(qkv, beta, a, dtb[:DH].contiguous(), al[:DH].contiguous(), states[0], od, first, start, slots, DH, DH,
+                                                             128, 128, True, status, decay_per_head=True), reps=2)
+                print(f"   delta rule (one decay per head) of as many state numbers, {DH} x 128 x 128: {t:7.1f} us = {t / n:6.4f} us per token", flush=True)
+                if kernels.linear_piece_rows(n, DH, 128, 128):
+                    pieces = kernels.linear_pieces_needed(n, S)
+                    meta = torch.zeros(4 * pieces + 2 * S + 1, dtype=torch.int32, device=DEV)
+                    piece_state, fixed = torch.empty(pieces, DH * 128 * 128, device=DEV), torch.full((DH,), 0.97, device=DEV)
+                    t = graph_time(lambda: kernels.decay_linear_attention_pieces(qkv, fixed, states[0], od, first, start, slots, DH,
+                                                                                 128, 128, True, status, meta, piece_state), reps=2)
+                    print(f"   lightning attention in pieces, {DH} x 128 x 128: {t:7.1f} us = {t / n:6.4f} us per token", flush=True)
+            out = torch.empty(n, inner, device=DEV).bfloat16()
+            w = torch.ones(inner, device=DEV)
+            t = graph_time(lambda: kernels.gate_group_norm(y, proj[:, :inner], w, out, SG, 1e-6))
+            t2 = graph_time(lambda: kernels.gated_head_norm(y, proj[:, :inner], w[:inner // SG].contiguous(), out, SG, 1e-6, gate_silu=True))
+            print(f"gate, then norm in {SG} parts, {n:4d} x {inner}: {t:6.1f} us {n * inner * 10 / t / 1e3:6.0f} GB/s; norm, then gate {t2:6.1f} us", flush=True)
+        # the router: 16 experts in four groups of which two are kept, four per token
+        E, top = 16, 4
+        for n in (t_len, 8):
+            h, wr = (torch.randn(n, d, device=DEV) * 0.5).bfloat16(), torch.randn(E, d, device=DEV) * 0.05
+            choice, weight = torch.empty(n, top, dtype=torch.int32, device=DEV), torch.empty(n, top, device=DEV)
+            p = pos[:n]
+            t = graph_time(lambda: kernels.moe_route(h, wr, None, None, p, top, 4, 2, 1.0, choice, weight, None, softmax=True, group_best=True,
+                                                     renorm_eps=1e-20))
+            t2 = graph_time(lambda: kernels.moe_route(h, wr, None, None, p, top, 1, 1, 1.0, choice, weight, None, softmax_chosen=True))
+            print(f"router, softmax over {E} experts, best groups, {n:4d} rows: {t:6.1f} us; largest logits, softmax over the chosen: {t2:6.1f} us", flush=True)
+            ff = d
+            ups = [(torch.randn(E * 2 * ff, d, device=DEV) * 0.03).bfloat16() for _ in range(3)]
+            downs = [(torch.randn(E * d, ff, device=DEV) * 0.03).bfloat16() for _ in range(3)]
+            pair = torch.empty(n, top * d, device=DEV)
+            turn = [0]
+            fl = 2.0 * n * top * 3 * d * ff
+            for name, unit in (("SwiGLU", kernels.SILU_UNIT), ("   clamped", (7.0, 1.702))):
+                if n > 16:
+                    tabs = torch.zeros(2 * (E + 1) + n * top, dtype=torch.int32, device=DEV)
+                    act = torch.empty(n, top * ff, device=DEV).bfloat16()
+
+                    def fn():
+                        turn[0] += 1
+                        kernels.moe_experts_grouped(h, ups[turn[0] % 3], downs[turn[0] % 3], E, choice, p, tabs, act, pair, unit=unit)
+                else:
+                    act = torch.empty(n, top * ff, device=DEV)
+
+                    def fn():
+                        turn[0] += 1
+                        kernels.moe_expert_halves(h, ups[turn[0] % 3], downs[turn[0] % 3], E, choice, p, act, pair, unit=unit)
+                t = graph_time(fn, reps=6)
+                used = int(choice.unique().numel()) * 3 * d * ff * 2
+                print(f"{name} experts {E} x ({d} -> 2 x {ff} -> {d}), {top} per token, {n:4d} rows: {t:7.1f} us {fl / t / 1e6:6.1f} TFLOP/s "
+                      f"{used / t / 1e3:6.0f} GB/s of chosen weights", flush=True)
+    kernels.check_status(status)
+
+
+CASES = ("gemm_stream", "gemm_tc", "attention_decode", "attention_splits", "attention_prefill", "float32", "small", "decode_program", "layer_gemms", "latent_attention", "delta_rule", "lonorax", "tagenex", "babotar", "felovik")
 
 
 def main(argv) -> int:
@@ -925,6 +1098,8 @@ def main(argv) -> int:
         bench_tagenex()
     elif argv[0] == "babotar":
         bench_babotar()
+    elif argv[0] == "felovik":
+        bench_felovik()
     else:
         bench_attention_prefill()
     return 0

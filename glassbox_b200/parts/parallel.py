@@ -7,6 +7,9 @@ a wiring that norms a branch: ``ctx.overwrite_output``); one small kernel forms 
 into the residual, in float32. A wiring that norms the branch may take a normed pair over in its parts
 (``ctx.accepts_normed_pair`` / ``ctx.normed_pair``) and form the sum on its way over the rows. Where both sides begin with one
 stacked product of their input, the two matrices may be one (``shared_projection``): one product then serves both.
+
+The sides do not depend on one another, so the right one runs on the step's second stream where there is one (a fork and a
+join in the recorded step), with scratch buffers of its own.
 """
 from __future__ import annotations
 
@@ -69,9 +72,9 @@ class ParallelMixer(Mixer):
             proj = ctx.scratch("parallel_proj", (n, ld), torch.float32)[:, :self.in_cols]
             linear(ctx, h, self.params["w_in"], proj)
             inputs = {"left": proj[:, :self.left_cols], "right": proj[:, self.left_cols:]}
-        outs = []
-        for name, part in (("left", self.left), ("right", self.right)):
-            y = ctx.scratch("parallel_" + name, (n, d), torch.float32)
+        outs = [ctx.scratch("parallel_" + name, (n, d), torch.float32) for name in ("left", "right")]
+
+        def run(name, part, y):
             ctx.overwrite_output = bool(part.can_overwrite_output)
             if not ctx.overwrite_output:
                 y.zero_()
@@ -79,7 +82,20 @@ class ParallelMixer(Mixer):
                 part.forward(ctx, inputs[name], y, sub_view(cache, name, part.cache_spec()), writes_cache)
             finally:
                 ctx.overwrite_output = overwrite
-            outs.append(y)
+        side, main = getattr(ctx, "side_stream", None), torch.cuda.current_stream()
+        if side is not None and side != main:
+            side.wait_stream(main)
+            with torch.cuda.stream(side):
+                before, ctx.scratch_prefix = ctx.scratch_prefix, ctx.scratch_prefix + "beside_"
+                try:
+                    run("right", self.right, outs[1])
+                finally:
+                    ctx.scratch_prefix = before
+            run("left", self.left, outs[0])
+            main.wait_stream(side)
+        else:
+            run("left", self.left, outs[0])
+            run("right", self.right, outs[1])
         for name, was in offers.items():
             setattr(ctx, name, was)
         s = self.spec

@@ -110,8 +110,8 @@ class StateSpace(Mixer):
             return
         chunks = kernels.ssd_chunks_needed(n, ctx.seq_start_pos.shape[0] - k)
         own = ctx.scratch("ssd_chunk_state", (chunks, self.H * self.N * self.V), torch.float32, grow=True)
-        decay = ctx.scratch("ssd_chunk_decay", (chunks, self.H), torch.float32, grow=True)
-        kernels.ssd_chunks(*args, ctx.max_rows_per_seq, self.H, self.G, self.N, self.V, writes_cache, ctx.status, own, decay)
+        steps = ctx.scratch("ssd_chunk_steps", (chunks, self.H * 2 * kernels.ssd_chunk_rows()), torch.float32, grow=True)
+        kernels.ssd_chunks(*args, ctx.max_rows_per_seq, self.H, self.G, self.N, self.V, writes_cache, ctx.status, own, steps)
 
 
 register_part("mixer", "state_space", StateSpace, replace=True)

@@ -258,8 +258,9 @@ def _run_ssd(how, steps, rows, dts, p, H, G, N, V, slots, state):
         args = (x, dt, p["dt_bias"], p["a_log"], p["skip"], state, y, *meta)
         if how == "chunks":
             need = kernels.ssd_chunks_needed(n, len(step))
-            own, decay = torch.full((need, H * N * V), float("nan"), device=DEV), torch.full((need, H), float("nan"), device=DEV)
-            kernels.ssd_chunks(*args, max(e[1] for e in step if e), H, G, N, V, True, status, own, decay)
+            own = torch.full((need, H * N * V), float("nan"), device=DEV)
+            steps = torch.full((need, H * 2 * kernels.ssd_chunk_rows()), float("nan"), device=DEV)
+            kernels.ssd_chunks(*args, max(e[1] for e in step if e), H, G, N, V, True, status, own, steps)
         else:
             kernels.ssd_walk(*args, H, G, N, V, True, status)
         assert int(status.item()) == 0
