@@ -430,7 +430,8 @@ def _run_attention(how, steps, rows_in, m, cache, dtype, eps):
 
 
 ATTENTION_CASES = [("rows", "float32", 6, 2, 20, 12), ("rows", "float32", 3, 1, 9, 7), ("decode", "float32", 4, 2, 16, 32), ("decode", "bfloat16", 8, 2, 48, 64),
-                   ("split", "bfloat16", 8, 2, 64, 64), ("split", "bfloat16", 4, 4, 32, 32), ("tiles", "bfloat16", 4, 2, 64, 32),
+                   ("split", "bfloat16", 8, 2, 64, 64), ("split", "bfloat16", 4, 4, 32, 32), ("split", "bfloat16", 4, 1, 16, 16), ("split", "bfloat16", 4, 2, 128, 128),
+                   ("tiles", "bfloat16", 4, 2, 64, 32),
                    ("tiles", "bfloat16", 6, 3, 48, 48), ("tiles", "bfloat16", 2, 1, 80, 80), ("tiles", "bfloat16", 2, 2, 96, 96),
                    ("flash", "bfloat16", 4, 2, 64, 64)]
 
