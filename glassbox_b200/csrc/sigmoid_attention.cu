@@ -18,6 +18,12 @@
 
 constexpr int SA_WARPS = 4;
 
+// two neighbours at once (the address is a multiple of two elements)
+__device__ __forceinline__ void sa_store2(float* at, float a, float c) { *reinterpret_cast<float2*>(at) = make_float2(a, c); }
+__device__ __forceinline__ void sa_store2(__nv_bfloat16* at, float a, float c) {
+    *reinterpret_cast<__nv_bfloat162*>(at) = __floats2bfloat162_rn(a, c);
+}
+
 template <typename T>
 __global__ void __launch_bounds__(512) qk_norm_rope_write_kernel(
     const float* __restrict__ qkv, long long ld, const float* __restrict__ q_gain, const float* __restrict__ k_gain,
@@ -42,6 +48,8 @@ __global__ void __launch_bounds__(512) qk_norm_rope_write_kernel(
     const long long page = slot / page_size;
     const int off = (int)(slot % page_size);
     const int pairs = D / 2;          // (an odd last channel is handled apart)
+    // heads of up to 128 channels whose pairs are aligned: a lane has its two pairs in registers, one trip to memory
+    const bool in_pairs = D % 2 == 0 && D <= 128 && ld % 2 == 0 && ((uintptr_t)qkv & 7) == 0;
     const float temp = temp_every > 0.f ? 1.0f + temp_coef * logf(floorf(__fdiv_rn((float)(pos + 1), temp_every)) + 1.0f) : 1.0f;
     for (int head = blockIdx.y * warps + warp; head < H + G; head += warps * gridDim.y) {
         const bool is_q = head < H;
@@ -49,6 +57,39 @@ __global__ void __launch_bounds__(512) qk_norm_rope_write_kernel(
         const float* x = src + (size_t)head * D;     // q heads, then k heads: contiguous in the stacked row
         const float* gain = is_q ? q_gain : k_gain;      // nullptr: the heads are not normed, or (unit_norm) normed without a gain
         float r = 1.f;
+        if (in_pairs) {
+            T* dst = is_q ? q_out + ((size_t)row * H + head) * D : kcache + ((page * G + (head - H)) * page_size + off) * D;
+            float2 v[2], w[2];
+#pragma unroll
+            for (int u = 0; u < 2; ++u) {
+                const int i = lane + 32 * u;
+                v[u] = i < pairs ? *reinterpret_cast<const float2*>(x + 2 * i) : make_float2(0.f, 0.f);
+                w[u] = make_float2(1.f, 1.f);
+                if (gain != nullptr && i < pairs) w[u] = make_float2(gain[2 * i], gain[2 * i + 1]);
+            }
+            if (gain != nullptr || unit_norm) {
+                float ss = 0.f;
+#pragma unroll
+                for (int u = 0; u < 2; ++u) ss = fmaf(v[u].x, v[u].x, fmaf(v[u].y, v[u].y, ss));
+                r = 1.0f / sqrtf(gb_warp_sum(ss) / (float)D + eps);
+            }
+            if (is_q) r *= temp;
+#pragma unroll
+            for (int u = 0; u < 2; ++u) {
+                const int i = lane + 32 * u;
+                if (i >= pairs) continue;
+                float a = v[u].x * r * w[u].x, c = v[u].y * r * w[u].y;
+                if (2 * i + 1 < rot) {
+                    float sn, cs;
+                    sincosf((float)pos * inv_freq[i], &sn, &cs);
+                    const float ra = a * cs - c * sn, rc = c * cs + a * sn;
+                    a = ra;
+                    c = rc;
+                }
+                sa_store2(dst + 2 * i, a, c);
+            }
+            continue;
+        }
         if (gain != nullptr || unit_norm) {
             float ss = 0.f;
             for (int i = lane; i < D; i += 32) ss = fmaf(x[i], x[i], ss);
@@ -79,6 +120,14 @@ __global__ void __launch_bounds__(512) qk_norm_rope_write_kernel(
     if (blockIdx.y == gridDim.y - 1 && (store || values_out != nullptr)) {      // (the row's last block has the fewest heads)
         const float* v = src + (size_t)(H + G) * D;
         const float lam = values_in != nullptr ? *value_mix : 0.f;
+        if (values_in == nullptr && values_out == nullptr && V % 2 == 0 && ld % 2 == 0 && ((((H + G) * D) & 1) | ((uintptr_t)qkv & 7)) == 0) {
+            for (int idx = threadIdx.x; idx < G * V / 2; idx += blockDim.x) {
+                const int g = 2 * idx / V, i = 2 * idx - g * V;
+                const float2 val = *reinterpret_cast<const float2*>(v + 2 * idx);
+                sa_store2(vcache + ((page * G + g) * page_size + off) * V + i, val.x, val.y);
+            }
+            return;
+        }
         for (int idx = threadIdx.x; idx < G * V; idx += blockDim.x) {
             const int g = idx / V, i = idx % V;
             float val = v[idx];
