@@ -3,9 +3,9 @@
 The device only ever sees block tables and slots; every decision is taken here, on the host, and
 can be tested without a GPU.
 
-Layers whose mixers have the same needs (``PagedKvSpec``: kv heads, head size, window) form a
+Layers whose mixers have the same needs (``PagedKvSpec``: kv heads, head size, window, chunk) form a
 *group* with a page pool and per-request block tables of its own, so a group that keeps only a
-window of keys can give pages back early without touching a group that keeps everything. Within a
+window of keys, or the keys of the current chunk, can give pages back early without touching a group that keeps everything. Within a
 group one page id addresses the same page in every cache layer of the group, as in Glassbox
 where one block id is valid in every layer (crates/glassbox-core/src/kv.rs:17-19, 58-65).
 
@@ -46,11 +46,12 @@ class GroupSpec:
     page_size: int = 16
     window: Optional[int] = None
     name: str = ""
+    chunk: Optional[int] = None
 
 
 _I, _LL, _P = ctypes.c_int, ctypes.c_longlong, ctypes.c_void_p
 _SIGNATURES = {
-    "gbh_cache_new": ([_I, _P, _P, _P, _I, _I, _I], _P),
+    "gbh_cache_new": ([_I, _P, _P, _P, _P, _I, _I, _I], _P),
     "gbh_cache_delete": ([_P], None),
     "gbh_cache_shares_prefixes": ([_P], _I),
     "gbh_cache_add": ([_P, _LL, _P, _I, _P], _I),
@@ -112,7 +113,13 @@ class _GroupView:
     """What the rest of the engine may know about a group."""
 
     def __init__(self, spec: GroupSpec):
-        self.spec, self.page_size, self.window = spec, spec.page_size, spec.window
+        self.spec, self.page_size, self.window, self.chunk = spec, spec.page_size, spec.window, spec.chunk
+
+    @property
+    def reach(self) -> Optional[int]:
+        """The most keys that a query of this group sees (None: every earlier one)."""
+        spans = [s for s in (self.window, self.chunk) if s is not None]
+        return min(spans) if spans else None
 
 
 class CacheManager:
@@ -127,12 +134,13 @@ class CacheManager:
         self.max_requests = max_requests
         pages, sizes = _ints([g.num_pages for g in groups]), _ints([g.page_size for g in groups])
         windows = _ints([-1 if g.window is None else g.window for g in groups])
-        self._h = self._lib.gbh_cache_new(len(groups), pages.ctypes.data, sizes.ctypes.data, windows.ctypes.data,
+        chunks = _ints([0 if g.chunk is None else g.chunk for g in groups])
+        self._h = self._lib.gbh_cache_new(len(groups), pages.ctypes.data, sizes.ctypes.data, windows.ctypes.data, chunks.ctypes.data,
                                           max_requests, int(share_prefixes), int(has_state))
         if not self._h:
             raise ValueError(self._lib.gbh_last_error().decode())
         # Prefix sharing is only sound when what a page holds is a pure function of the token prefix
-        # for every mixer: the library switches it off with windows (pages vanish) or per-request state.
+        # for every mixer: the library switches it off with windows or chunks (pages vanish) or per-request state.
         self.share_prefixes = bool(self._lib.gbh_cache_shares_prefixes(self._h))
         self._ids: Dict[object, int] = {}     # request id -> the 64-bit name the library knows it by
         self._next = 1

@@ -32,7 +32,8 @@ class RopeSpec:
     rotary_dim: int
     max_position: int
     pairing: str = "half"
-    #: None, or a ``RopeRescaleSpec``: the frequencies are stretched for contexts longer than the trained one
+    #: None, a ``RopeRescaleSpec`` or a ``RopeBandRescaleSpec``: the frequencies are stretched for contexts longer than the
+    #: trained one
     rescale: Any = None
     kind: str = "rope"
 
@@ -50,6 +51,17 @@ class RopeRescaleSpec:
     fast: float
     slow: float
     magnitude_slope: float = 0.1
+
+
+@dataclass(frozen=True)
+class RopeBandRescaleSpec:
+    """Stretching of a rotation's frequencies in bands of wavelength l = 2 pi / f: f stays where l < ``original`` / ``high``,
+    becomes f / ``factor`` where l > ``original`` / ``low``, and between the two is (1 - s) f / ``factor`` + s f with
+    s = (``original`` / l - ``low``) / (``high`` - ``low``). Sine and cosine keep their length."""
+    factor: float
+    original: float
+    low: float
+    high: float
 
 
 @dataclass(frozen=True)
@@ -102,7 +114,9 @@ class LatentAttentionSpec:
     maps, and one rotated key part of ``rope_dim`` numbers shared by all heads. A head's query is [nope_dim unrotated |
     rope_dim rotated]. ``sink`` adds a learned logit per head to the softmax denominator. ``kv_source`` None: the layer
     projects and stores its own latent; otherwise it has no such projection and reads the cache of the layer it names
-    (the schedule says which cache layer that is)."""
+    (the schedule says which cache layer that is). ``q_rank``: queries go through a latent of their own, W_uq RMSnorm(W_dq h)
+    (a plain gain, ``latent_eps``). ``output_gate``: the concatenated heads are multiplied by sigmoid(W_g h), a logit per
+    output channel. ``window`` as in ``GqaAttentionSpec``."""
     num_heads: int
     nope_dim: int
     rope_dim: int
@@ -114,6 +128,8 @@ class LatentAttentionSpec:
     sink: bool = True
     kv_source: Optional[int] = None
     window: Optional[int] = None
+    q_rank: Optional[int] = None
+    output_gate: bool = False
     kind: str = "latent_attention"
 
 
@@ -155,9 +171,9 @@ class SigmoidAttentionSpec:
 
 @dataclass(frozen=True)
 class SinkAttentionSpec:
-    """Causal grouped-query softmax attention without a rotation, whose positions enter through a bias on the distance:
+    """Causal grouped-query softmax attention, whose positions may enter through a bias on the distance:
     score(i, j) = q_i . k_j * ``scale`` - r1_h * ln(1 + r2_h * (i - j)) with two learned numbers per query head
-    (``distance_bias``). With ``sink`` the softmax's denominator also holds exp(sink_h), a learned logit per head that has no
+    (``distance_bias``), or through a rotation of queries and keys (``position``, half-split pairs). With ``sink`` the softmax's denominator also holds exp(sink_h), a learned logit per head that has no
     key and no value. Queries and keys have ``head_dim`` channels and are RMS-normed per head (``qk_norm_eps``; None: no
     norm; one gain for all query heads, one for all key heads); values have ``value_dim`` channels. ``value_mix``:
     "none"; "source": this layer's values are kept for the step, for later layers to mix in; "mixed": the values become
@@ -165,8 +181,10 @@ class SinkAttentionSpec:
     they are cached. ``output_gate``: head h's output is multiplied by sigmoid(w_gate_h . x), one number per head and
     token, from the same input as the projections; with ``gate_per`` "channel" the gate has a logit per output channel
     instead (the concatenated heads times sigmoid(W_g x)). ``qk_norm_gain`` False: the query and key norms have no gains.
-    ``q_temp`` = (coef, every): the query at position p is multiplied by 1 + coef * ln(floor((p + 1) / every) + 1).
-    ``window`` as in ``GqaAttentionSpec``."""
+    ``qk_norm_over`` "projection": queries (and keys) are normed over all their heads together, with a gain per projected
+    channel. ``q_temp`` = (coef, every): the query at position p is multiplied by 1 + coef * ln(floor((p + 1) / every) + 1).
+    ``softcap``: scores pass softcap * tanh(score / softcap) (the sink does not). ``window`` as in ``GqaAttentionSpec``;
+    ``chunk``: a query at position p sees the keys of its own run of ``chunk`` positions, floor(p / chunk) * chunk .. p."""
     num_heads: int
     num_kv_heads: int
     head_dim: int
@@ -181,6 +199,10 @@ class SinkAttentionSpec:
     gate_per: str = "head"
     qk_norm_gain: bool = True
     q_temp: Optional[Tuple[float, float]] = None
+    qk_norm_over: str = "head"
+    position: Any = None
+    softcap: Optional[float] = None
+    chunk: Optional[int] = None
     kind: str = "sink_attention"
 
 
@@ -345,6 +367,13 @@ class GeluGluSpec:
 
 
 @dataclass(frozen=True)
+class GeluMlpSpec:
+    """Dense feed-forward without a gate: down(gelu(up(x))) with the exact gelu(z) = z/2 (1 + erf(z / sqrt 2))."""
+    intermediate_size: int
+    kind: str = "gelu_mlp"
+
+
+@dataclass(frozen=True)
 class EmbeddingSpec:
     """Token embedding: the float32 residual row of a token is its row of the table, as it is
     (crates/glassbox-core/src/model.rs:228-231). Another kind (a scaled table, a learned position added to it) is
@@ -373,6 +402,13 @@ class ScaledLmHeadSpec:
     """Output head whose logits carry a constant factor: logits = (hidden states times the head matrix) * ``scale``."""
     scale: float
     kind: str = "scaled_lm_head"
+
+
+@dataclass(frozen=True)
+class CappedLmHeadSpec:
+    """Output head whose logits are capped: logits = softcap * tanh((hidden states times the head matrix) / ``softcap``)."""
+    softcap: float
+    kind: str = "capped_lm_head"
 
 
 @dataclass(frozen=True)

@@ -38,6 +38,7 @@ struct DecodeSinkTerms {
     const float* gate;
     long long ld_gate;
     int gate_channels;
+    float cap;
 };
 
 // The merge runs inside a thread-block cluster in the variant for large batches (16 keys per iteration: small
@@ -63,6 +64,7 @@ static int launch_mma(const void* q, long long q_stride, void* out, long long ou
     a.page_shift = page_shift; a.num_pages = num_pages; a.scale = scale; a.window = window; a.splits = splits;
     a.part_acc = part_acc; a.part_ml = part_ml; a.counters = counters; a.status = status; a.n = n; a.hd = HD; a.block_keys = BK;
     a.r1 = terms.r1; a.r2 = terms.r2; a.sink = terms.sink; a.gate = terms.gate; a.ld_gate = terms.ld_gate; a.gate_channels = terms.gate_channels;
+    a.cap = terms.cap;
     a.late_release = 1;   // (135M decode step at batch 1: 0.646 -> 0.630 ms; no difference at batch 64)
     const int group = nh / nkv;
     const int cluster_bytes = decode_attn_cluster_floats<HD>(group, splits, NW) * (int)sizeof(float);
@@ -169,17 +171,19 @@ GB_EXPORT int gb_attention_decode_mma_pdl(const void* q, long long q_stride, voi
 // gb_attention_decode_mma_pdl for a softmax with a distance bias, a sink and an output gate: the score of a key `dist`
 // tokens back loses r1[head] * ln(1 + r2[head] * dist) (r1 and r2 both or neither), the denominator also holds
 // exp(sink[head]), and the head's output is multiplied by sigmoid(gate[row * ld_gate + head]) (with gate_channels: each channel
-// by a gate of its own, gate[row * ld_gate + head * hd + c]). Each term may be nullptr.
+// by a gate of its own, gate[row * ld_gate + head * hd + c]). Each term may be nullptr. cap > 0: scores are capped as
+// cap * tanh(score / cap) first. window < 0: chunks of -window positions (gb_first_key).
 GB_EXPORT int gb_attention_decode_mma_sink(const void* q, long long q_stride, void* out, long long out_stride,
                                            const void* kcache, const void* vcache, const int* block_tables,
                                            int max_pages, const int* row_seq, const int* positions, int n, int nh,
                                            int nkv, int hd, int page_size, long long num_pages, float scale, int window,
                                            int splits, float* part_acc, float* part_ml, int* counters, int* status,
                                            int pdl, int block_keys, int warps, const float* r1, const float* r2,
-                                           const float* sink, const float* gate, long long ld_gate, int gate_channels, cudaStream_t stream) {
+                                           const float* sink, const float* gate, long long ld_gate, int gate_channels, float cap, cudaStream_t stream) {
     GB_REQUIRE((r1 == nullptr) == (r2 == nullptr), "gb_attention_decode_mma_sink: the distance bias needs r1 and r2");
     GB_REQUIRE(gate == nullptr || ld_gate >= (long long)nh * (gate_channels ? hd : 1), "gb_attention_decode_mma_sink: rows of gate logits are too short");
-    DecodeSinkTerms terms = {r1, r2, sink, gate, ld_gate, gate_channels};
+    GB_REQUIRE(cap >= 0.f, "gb_attention_decode_mma_sink: a negative cap");
+    DecodeSinkTerms terms = {r1, r2, sink, gate, ld_gate, gate_channels, cap};
     return decode_mma_dispatch<true>(q, q_stride, out, out_stride, kcache, vcache, block_tables, max_pages, row_seq, positions, n, nh,
                                      nkv, hd, page_size, num_pages, scale, window, splits, part_acc, part_ml, counters, status, pdl,
                                      block_keys, warps, stream, terms);

@@ -21,7 +21,7 @@ struct DecodeAttnArgs {
     int nh, nkv, page_size, page_shift;
     long long num_pages;
     float scale;
-    int window, splits;
+    int window, splits;     // (window: as gb_first_key's mask)
     float* part_acc;
     float* part_ml;
     int* counters;
@@ -29,7 +29,8 @@ struct DecodeAttnArgs {
     int n;           // rows (used by the persistent kernel to count its virtual blocks)
     int hd, block_keys;
     int late_release;   // let the next kernel in the stream go only after this one's own wait (else at its start)
-    // Read only by the SINK instantiations (each may be nullptr): the score of a key `dist` tokens back loses
+    // Read only by the SINK instantiations (each may be nullptr): the score, capped as cap * tanh(score / cap) where cap > 0,
+    // of a key `dist` tokens back loses
     // r1[head] * ln(1 + r2[head] * dist); the softmax's denominator also holds exp(sink[head]), which has no key and
     // no value; the head's output is multiplied by sigmoid(gate[row * ld_gate + head]) (float32 logits), or, with
     // gate_channels, channel c of it by sigmoid(gate[row * ld_gate + head * HD + c]).
@@ -39,6 +40,7 @@ struct DecodeAttnArgs {
     const float* gate;
     long long ld_gate;
     int gate_channels;
+    float cap;
 };
 
 constexpr float MMA_NEG_BIG = -1.0e30f;
@@ -159,6 +161,7 @@ __device__ __forceinline__ void attention_decode_mma_body(const DecodeAttnArgs& 
                 }
         }
     }
+    const float cap = SINK ? a.cap : 0.f, inv_cap2 = cap > 0.f ? 2.0f / cap : 0.f;
     auto sink_logit = [&](int head) { return (SINK && a.sink != nullptr) ? a.sink[head] : MMA_NEG_BIG; };
     auto channel_gate = [&](int head, int c) {
         return (SINK && a.gate != nullptr && a.gate_channels) ? 1.0f / (1.0f + __expf(-a.gate[(size_t)row * a.ld_gate + head * HD + c])) : 1.0f;
@@ -189,7 +192,7 @@ __device__ __forceinline__ void attention_decode_mma_body(const DecodeAttnArgs& 
     if constexpr (CLUSTER)   // every block of the cluster says that it runs (its shared memory exists); waited for before the first store into another block's
         asm volatile("barrier.cluster.arrive.relaxed.aligned;" ::: "memory");
     const int* table = block_tables + (size_t)row_seq[row] * max_pages;
-    const int first = (window > 0 && pos + 1 > window) ? pos + 1 - window : 0;
+    const int first = gb_first_key(pos, window);
     const int first_aligned = first / BK * BK;   // blocks of keys start at multiples of BK; keys before `first` are masked
     const int total = pos + 1 - first_aligned;
     const int chunk = ((total + splits - 1) / splits + BK - 1) / BK * BK;
@@ -317,6 +320,7 @@ __device__ __forceinline__ void attention_decode_mma_body(const DecodeAttnArgs& 
                 const int key = base + 8 * j + 2 * t + (e & 1);
                 float v = s[j][e] * scale;
                 if constexpr (SINK) {
+                    if (cap > 0.f) v = gb_cap_fast(v, cap, inv_cap2);
                     if (a.r1 != nullptr) v -= sk_b1[e >> 1] * logf(fmaf(sk_b2[e >> 1], (float)max(pos - key, 0), 1.0f));
                 }
                 s[j][e] = (key < k_end && key >= first) ? v : MMA_NEG_BIG;

@@ -26,7 +26,8 @@
 //               warp), when a new maximum exceeds it by more than 2^8 in the exponent: until then P stays
 //               below 256, which bfloat16 and the float32 sums hold without loss, and the final O / l is
 //               the same.
-// A query at position p sees keys max(0, p-window+1) .. p (crates/glassbox-core/src/model.rs:278-317);
+// A query at position p sees keys max(0, p-window+1) .. p (crates/glassbox-core/src/model.rs:278-317), or, window < 0, the
+// keys of its own chunk of -window positions up to p;
 // the mask is applied only in tiles that cross a boundary, and key tiles no row can see are skipped.
 // Pages that are missing (beyond what is reserved, or given back behind a window) can only hold
 // masked keys; page 0 is read in their place, so that P = 0 never meets anything but finite numbers
@@ -109,6 +110,12 @@ __device__ __forceinline__ float at_exp2(float x) {
     return y;
 }
 
+__device__ __forceinline__ float at_rcp(float x) {
+    float y;
+    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+
 // What the SINK instantiation reads beside the common arguments (each may be nullptr): the score of a key `dist` tokens
 // back loses r1[head] * ln(1 + r2[head] * dist); the softmax's denominator also holds exp(sink[head]), which has no key and
 // no value; the head's output is multiplied by sigmoid(gate[row * ld_gate + head]) (float32 logits; with gate_channels a gate
@@ -120,6 +127,7 @@ struct AtSinkTerms {
     const float* gate;
     long long ld_gate;
     int gate_channels;
+    float cap;              // > 0: scores are capped as cap * tanh(score / cap) before the bias
 };
 
 template <int HD, bool SINK = false>
@@ -157,7 +165,7 @@ __global__ void __launch_bounds__(AT_WARPS * 32) attention_prefill_tc_kernel(
     const int kvh = head / (nh / nkv);
     const int q_lo = qt * AT_BM;
     const int pos_lo = start_pos + q_lo, pos_hi = start_pos + min(nrows, q_lo + AT_BM) - 1;
-    const int key_lo = (window > 0 && pos_lo + 1 > window) ? pos_lo + 1 - window : 0;
+    const int key_lo = gb_first_key(pos_lo, window);
     const int kt_begin = key_lo / AT_BN, kt_end = pos_hi / AT_BN;   // inclusive
     const int ntiles = kt_end - kt_begin + 1;
     const int* table = block_tables + (size_t)seq * max_pages;
@@ -325,7 +333,8 @@ __global__ void __launch_bounds__(AT_WARPS * 32) attention_prefill_tc_kernel(
         const int my_tiles = (ntiles - g + 1) >> 1;
         float m_run = AT_NEG_BIG, l_run = 0.f;
         bool ok = true;
-        auto visible = [&](int key) { return key <= pos && (window <= 0 || key > pos - window); };
+        const int first = gb_first_key(pos, window), first_last = gb_first_key(pos_lo + AT_BM - 1, window);
+        auto visible = [&](int key) { return key <= pos && key >= first; };
         // SINK: the scores are brought into the base-2 domain and lose their bias before the maximum is taken, so what
         // follows scales them by one. The bias depends on the distance alone: the 32 rows of this warp and the 128 keys of a
         // tile are 159 distances apart, whose biases the warp writes into a table of its own per tile (five logarithms a
@@ -335,7 +344,12 @@ __global__ void __launch_bounds__(AT_WARPS * 32) attention_prefill_tc_kernel(
         float* tb = reinterpret_cast<float*>(at_smem + G::BIAS_OFF) + (warp - 2) * G::BIAS_WARP;
         float b1 = 0.f, b2 = 0.f;
         bool biased = false;
+        float cap2 = 0.f, cap_in = 0.f;       // cap and 2 scale / cap, both in the base-2 domain
         if constexpr (SINK) {
+            if (terms.cap > 0.f) {
+                cap2 = terms.cap * 1.4426950408889634f;
+                cap_in = 2.0f * sl2 / terms.cap;
+            }
             biased = terms.r1 != nullptr;
             if (biased) {
                 b1 = terms.r1[head];
@@ -352,20 +366,29 @@ __global__ void __launch_bounds__(AT_WARPS * 32) attention_prefill_tc_kernel(
             __syncwarp();
             if (lane == 0) mbar_arrive(&sh.s_free[g]);   // the buffer may take the group's next S
             if constexpr (SINK) {
+                if (cap2 > 0.f) {
+                    // cap tanh(s / cap) = cap - 2 cap / (1 + exp(2 s / cap))
+#pragma unroll
+                    for (int k = 0; k < AT_BN; ++k) {
+                        const float e = at_exp2(__uint_as_float(sv[k]) * cap_in);
+                        sv[k] = __float_as_uint(fmaf(-2.0f * cap2, at_rcp(1.0f + e), cap2));
+                    }
+                }
+                const float sl = cap2 > 0.f ? 1.0f : sl2;      // what is left to scale
                 if (biased) {
                     const int base = pos_lo + q * 32 - key0 - 127;
                     __syncwarp();                      // (the table of the tile before has been read)
                     for (int i = lane; i < G::BIAS_WARP; i += 32) tb[i] = b1 * __log2f(fmaf(b2, (float)max(base + i, 0), 1.0f));
                     __syncwarp();
 #pragma unroll
-                    for (int k = 0; k < AT_BN; ++k) sv[k] = __float_as_uint(fmaf(__uint_as_float(sv[k]), sl2, -tb[lane + 127 - k]));
-                } else {
+                    for (int k = 0; k < AT_BN; ++k) sv[k] = __float_as_uint(fmaf(__uint_as_float(sv[k]), sl, -tb[lane + 127 - k]));
+                } else if (cap2 <= 0.f) {
 #pragma unroll
                     for (int k = 0; k < AT_BN; ++k) sv[k] = __float_as_uint(__uint_as_float(sv[k]) * sl2);
                 }
             }
             // the mask matters only where the tile crosses the diagonal, the window's edge or the last key
-            const bool need_mask = key0 + AT_BN - 1 > pos_lo || (window > 0 && key0 < pos_lo + AT_BM - window);
+            const bool need_mask = key0 + AT_BN - 1 > pos_lo || key0 < first_last;
             if (need_mask) {
 #pragma unroll
                 for (int k = 0; k < AT_BN; ++k)
@@ -580,16 +603,17 @@ GB_EXPORT int gb_attention_prefill_tc(const void* q, long long q_stride, int n_r
 // gb_attention_prefill_tc for a softmax with a distance bias, a sink and an output gate: the score of a key `dist` tokens
 // back loses r1[head] * ln(1 + r2[head] * dist) (r1 and r2 both or neither), the denominator also holds exp(sink[head]),
 // and the head's output is multiplied by sigmoid(gate[row * ld_gate + head]) (with gate_channels: each channel by a gate of
-// its own). Each term may be nullptr.
+// its own). Each term may be nullptr. cap > 0: scores are capped as cap * tanh(score / cap) first.
 GB_EXPORT int gb_attention_prefill_tc_sink(const void* q, long long q_stride, int n_rows, void* out, long long out_stride,
                                            const void* kcache, const void* vcache, const int* block_tables, int max_pages,
                                            const int* seq_first_row, const int* seq_start_pos, int num_seqs,
                                            int max_rows_per_seq, int nh, int nkv, int hd, int page_size, long long num_pages,
                                            float scale, int window, int* status, const float* r1, const float* r2,
-                                           const float* sink, const float* gate, long long ld_gate, int gate_channels, cudaStream_t stream) {
+                                           const float* sink, const float* gate, long long ld_gate, int gate_channels, float cap, cudaStream_t stream) {
+    GB_REQUIRE(cap >= 0.f, "gb_attention_prefill_tc_sink: a negative cap");
     GB_REQUIRE((r1 == nullptr) == (r2 == nullptr), "gb_attention_prefill_tc_sink: the distance bias needs r1 and r2");
     GB_REQUIRE(gate == nullptr || ld_gate >= (long long)nh * (gate_channels ? hd : 1), "gb_attention_prefill_tc_sink: rows of gate logits are too short");
-    const AtSinkTerms terms = {r1, r2, sink, gate, ld_gate, gate_channels};
+    const AtSinkTerms terms = {r1, r2, sink, gate, ld_gate, gate_channels, cap};
     return prefill_tc_launch<true>(q, q_stride, n_rows, out, out_stride, kcache, vcache, block_tables, max_pages, seq_first_row,
                                    seq_start_pos, num_seqs, max_rows_per_seq, nh, nkv, hd, page_size, num_pages, scale, window,
                                    status, stream, terms);

@@ -60,6 +60,22 @@ __device__ __forceinline__ float gb_gelu_tanh_fast(float z) {
     return __fdividef(z, 1.0f + __expf(-1.5957691216057308f * (z + 0.044715f * z * z * z)));
 }
 
+// GELU itself: z times the cumulative normal distribution, z / 2 (1 + erf(z / sqrt 2)).
+__device__ __forceinline__ float gb_gelu(float z) { return 0.5f * z * (1.0f + erff(z * 0.7071067811865476f)); }
+
+// cap * tanh(s / cap) through tanh(y) = 1 - 2 / (1 + exp(2 y)) with the hardware's exponential and division: an absolute
+// error of a few 1e-7 * cap, for scores on their way into an exponential. inv2 = 2 / cap.
+__device__ __forceinline__ float gb_cap_fast(float s, float cap, float inv2) {
+    return fmaf(-2.0f * cap, __fdividef(1.0f, 1.0f + __expf(s * inv2)), cap);
+}
+
+// The first key that a query at position `pos` sees. mask > 0: a sliding window of that many keys; mask < 0: chunks of -mask
+// positions counted from position 0, a query sees the keys of its own chunk; 0: every key.
+__device__ __forceinline__ int gb_first_key(int pos, int mask) {
+    if (mask < 0) return pos - pos % -mask;
+    return (mask > 0 && pos + 1 > mask) ? pos + 1 - mask : 0;
+}
+
 // ln(1 + e^z), accurate for any z (also as a factor: no cancellation where e^z is small).
 __device__ __forceinline__ float gb_softplus(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
 

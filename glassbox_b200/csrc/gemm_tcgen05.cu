@@ -25,7 +25,7 @@
 constexpr int TC_BM = 128;
 constexpr int TC_BK = 64;        // 64 bfloat16 = 128 bytes = one swizzle row
 
-enum { TC_STORE_BF16 = 0, TC_STORE_F32 = 1, TC_ADD_F32 = 2, TC_ROPE_QKV = 3, TC_RELU2_BF16 = 4 };   // 4: store bfloat16(max(c, 0)^2)
+enum { TC_STORE_BF16 = 0, TC_STORE_F32 = 1, TC_ADD_F32 = 2, TC_ROPE_QKV = 3, TC_RELU2_BF16 = 4, TC_GELU_BF16 = 5 };   // 4: store bfloat16(max(c, 0)^2), 5: bfloat16(gelu(c))
 
 // What the epilogue of a stacked QKV product needs to rotate the heads and write the cache: the
 // (cos, sin) table [max_pos, hd/2], each row's position (negative: a padding row) and cache slot
@@ -372,7 +372,11 @@ __global__ void __launch_bounds__(192) gemm_tcgen05_kernel(const __grid_constant
                         r[j] = __float_as_uint(g * g);
                     }
                 }
-                if (GATED || mode == TC_STORE_BF16 || mode == TC_RELU2_BF16) {
+                if (!GATED && mode == TC_GELU_BF16) {      // gelu, from the float32 sums
+#pragma unroll
+                    for (int j = 0; j < 32; ++j) r[j] = __float_as_uint(gb_gelu(__uint_as_float(r[j])));
+                }
+                if (GATED || mode == TC_STORE_BF16 || mode == TC_RELU2_BF16 || mode == TC_GELU_BF16) {
                     // a thread's 32 columns are 64 contiguous bytes: store them directly, 16 bytes at a time
                     __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(C) + (size_t)row * ldc + col0;
                     if (row < M) {
@@ -569,7 +573,7 @@ static int pick_bn(int M, int N, int K, int epilogue, int narrowest = 64) {
 // that a producer of a split RMSNorm writes.
 GB_EXPORT int gb_gemm_tcgen05_column_tiles(int M, int N, int K) { return gb_ceil_div(N, pick_bn(M, N, K, TC_EPI_ADD)); }
 
-// mode: 0 store bfloat16, 1 store float32, 2 add into float32.
+// mode: 0 store bfloat16, 1 store float32, 2 add into float32, 4 store bfloat16(max(c, 0)^2), 5 store bfloat16(gelu(c)).
 // Split RMSNorm (see TcNorm): with mode 2 and norm_gain != nullptr the launch also writes pre[M, N] =
 // bfloat16(c * norm_gain) and ss_out[M, gb_gemm_tcgen05_column_tiles(M, N, K)]; with ss_in != nullptr the rows of
 // the product are scaled by 1 / sqrt(sum_p ss_in[row, p] / K + eps) before they are stored or added.
@@ -579,7 +583,7 @@ GB_EXPORT int gb_gemm_tcgen05(const void* a, const void* w, void* c, int mode, i
     GB_REQUIRE(gb_gemm_tcgen05_supported(a, w, M, N, K, lda, ldw),
                "gb_gemm_tcgen05: operands must be 16-byte aligned with row strides that are multiples of 8 (M=%d N=%d K=%d)",
                M, N, K);
-    GB_REQUIRE(((mode >= 0 && mode <= 2) || mode == TC_RELU2_BF16) && ldc >= N && status != nullptr,
+    GB_REQUIRE(((mode >= 0 && mode <= 2) || mode == TC_RELU2_BF16 || mode == TC_GELU_BF16) && ldc >= N && status != nullptr,
                "gb_gemm_tcgen05: bad mode, ldc or status");
     GB_REQUIRE(norm_gain == nullptr || (mode == TC_ADD_F32 && pre != nullptr && ss_out != nullptr && ldp >= N &&
                                         (uintptr_t)norm_gain % 16 == 0),

@@ -3,7 +3,8 @@
 //
 // This is the shape of the up-projections of latent attention once they are moved to the query and to the weighted sum
 // of latents: K and N are a head's sizes (tens to a few hundred), so a head's product is far too small for a launch of
-// its own. One block = 64 rows x one head x up to 128 output columns; a and w[h] are staged once in shared memory
+// its own. Optionally every output is multiplied by sigmoid(gate[row, h, column]), a logit per output (float32 or bfloat16).
+// One block = 64 rows x one head x up to 128 output columns; a and w[h] are staged once in shared memory
 // (rows padded by 16 bytes so that ldmatrix meets no bank twice), each of the four warps takes 16 rows.
 #include "common.cuh"
 
@@ -24,7 +25,8 @@ __device__ __forceinline__ void hl_ldmatrix_x4(uint32_t (&r)[4], uint32_t addr) 
 
 __global__ void __launch_bounds__(128) head_linear_kernel(const __nv_bfloat16* __restrict__ a, long long lda, long long a_head,
                                                           const __nv_bfloat16* __restrict__ w, __nv_bfloat16* __restrict__ out,
-                                                          long long ldc, long long c_head, int n, int N, int K) {
+                                                          long long ldc, long long c_head, int n, int N, int K,
+                                                          const void* __restrict__ gate, long long ld_gate, int gate_f32) {
     extern __shared__ __align__(128) unsigned char hl_smem[];
     gb_pdl_launch_dependents();
     const int KS = K + 8;                                    // padded row, elements
@@ -79,16 +81,22 @@ __global__ void __launch_bounds__(128) head_linear_kernel(const __nv_bfloat16* _
     }
     const int row_a = m0 + warp * 16 + g, row_b = row_a + 8;
     __nv_bfloat16* oh = out + (size_t)head * c_head + n0;
+    auto opened = [&](int row, int col, float v) {       // v behind its gate
+        if (gate == nullptr) return v;
+        const size_t at = (size_t)row * ld_gate + (size_t)head * N + n0 + col;
+        const float z = gate_f32 ? reinterpret_cast<const float*>(gate)[at] : __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(gate)[at]);
+        return __fdividef(v, 1.0f + __expf(-z));
+    };
 #pragma unroll
     for (int nt = 0; nt < HL_BN / 8; ++nt) {
         const int col = nt * 8 + 2 * t;
         if (col < cols) {      // (N is even: a pair never straddles the edge)
             if (row_a < n) {
-                __nv_bfloat162 v = __floats2bfloat162_rn(acc[nt][0], acc[nt][1]);
+                __nv_bfloat162 v = __floats2bfloat162_rn(opened(row_a, col, acc[nt][0]), opened(row_a, col + 1, acc[nt][1]));
                 *reinterpret_cast<__nv_bfloat162*>(oh + (size_t)row_a * ldc + col) = v;
             }
             if (row_b < n) {
-                __nv_bfloat162 v = __floats2bfloat162_rn(acc[nt][2], acc[nt][3]);
+                __nv_bfloat162 v = __floats2bfloat162_rn(opened(row_b, col, acc[nt][2]), opened(row_b, col + 1, acc[nt][3]));
                 *reinterpret_cast<__nv_bfloat162*>(oh + (size_t)row_b * ldc + col) = v;
             }
         }
@@ -102,7 +110,9 @@ GB_EXPORT int gb_head_linear_supported(const void* a, long long lda, long long a
 }
 
 GB_EXPORT int gb_head_linear(const void* a, long long lda, long long a_head, const void* w, void* out, long long ldc,
-                             long long c_head, int n, int heads, int N, int K, cudaStream_t stream) {
+                             long long c_head, int n, int heads, int N, int K, const void* gate, long long ld_gate, int gate_f32,
+                             cudaStream_t stream) {
+    GB_REQUIRE(gate == nullptr || ld_gate >= (long long)heads * N, "gb_head_linear: rows of gate logits are too short");
     GB_REQUIRE(gb_head_linear_supported(a, lda, a_head, w, out, ldc, c_head, N, K),
                "gb_head_linear: K=%d must be a multiple of 16 up to %d, N=%d even, operands aligned", K, HL_MAX_K, N);
     GB_REQUIRE(n >= 0 && heads > 0 && heads <= 65535, "gb_head_linear: bad sizes");
@@ -115,7 +125,7 @@ GB_EXPORT int gb_head_linear(const void* a, long long lda, long long a_head, con
     }
     dim3 grid(gb_ceil_div(n, HL_BM), heads, gb_ceil_div(N, HL_BN));
     cudaError_t e = gb_launch(GB_PDL_GEMM, head_linear_kernel, grid, dim3(128), smem, stream, (const __nv_bfloat16*)a, lda, a_head,
-                              (const __nv_bfloat16*)w, (__nv_bfloat16*)out, ldc, c_head, n, N, K);
+                              (const __nv_bfloat16*)w, (__nv_bfloat16*)out, ldc, c_head, n, N, K, gate, ld_gate, gate_f32);
     if (e != cudaSuccess) {
         gb_set_error("gb_head_linear: launch failed: %s", cudaGetErrorString(e));
         return 2;

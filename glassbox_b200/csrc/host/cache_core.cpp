@@ -8,7 +8,7 @@
 // hashed pages kept for reuse until space is needed, oldest evicted first (kv.rs:96-110).
 //
 // Beyond the reference: several *groups* of layers, each with a page pool and block tables of its
-// own (a group with a window gives pages back as soon as the window has passed them), all-or-nothing
+// own (a group with a window or chunks gives pages back as soon as no later token can see them), all-or-nothing
 // reservation across the groups, and one fixed-size *state slot* per live request.
 //
 // The interface is a C ABI over an opaque handle, loaded with ctypes; requests are named by 64-bit
@@ -55,7 +55,8 @@ uint64_t chain_hash(uint64_t prev, const int32_t* tokens, int n) {
 }
 
 struct Group {
-    int num_pages, page_size, window;   // window < 0: keep every token
+    int num_pages, page_size, window;   // window < 0: no window
+    int chunk;                          // chunk <= 0: no chunks (neither: keep every token)
     bool share;
     std::vector<int> refs;
     std::vector<int> free;              // a stack; page 0 pops first
@@ -96,10 +97,14 @@ struct Group {
         ++refs[p];
     }
 
+    bool forgets() const { return window >= 0 || chunk > 0; }
+
     // index of the first page that a query at position >= length can still see
     int first_live_page(int length) const {
-        if (window < 0) return 0;
-        return std::max(0, length - window + 1) / page_size;
+        int first = 0;
+        if (window >= 0) first = std::max(0, length - window + 1);
+        if (chunk > 0) first = std::max(first, length / chunk * chunk);
+        return first / page_size;
     }
 
     // (new pages, copy-on-write needed) to write positions length .. length+n-1
@@ -140,9 +145,11 @@ GBH_EXPORT const char* gbh_last_error() { return g_error; }
 
 GBH_EXPORT uint64_t gbh_chain_hash(uint64_t prev, const int32_t* tokens, int n) { return chain_hash(prev, tokens, n); }
 
-// window[g] < 0: the group keeps every token. Prefix sharing is only sound when what a page holds is a pure
-// function of the token prefix for every mixer: it is switched off when a group has a window or a request has state.
-GBH_EXPORT void* gbh_cache_new(int n_groups, const int* num_pages, const int* page_size, const int* window,
+// window[g] >= 0: the group keeps the last window[g] tokens; chunk[g] > 0: it keeps the tokens of the run of chunk[g] positions
+// (counted from position 0) that the next token belongs to; neither: it keeps every token. Prefix sharing is only sound when
+// what a page holds is a pure function of the token prefix for every mixer: it is switched off when a group forgets tokens or a
+// request has state.
+GBH_EXPORT void* gbh_cache_new(int n_groups, const int* num_pages, const int* page_size, const int* window, const int* chunk,
                                int max_requests, int share_prefixes, int has_state) {
     for (int g = 0; g < n_groups; ++g)
         if (num_pages[g] <= 0 || page_size[g] <= 0) {
@@ -151,7 +158,7 @@ GBH_EXPORT void* gbh_cache_new(int n_groups, const int* num_pages, const int* pa
         }
     Cache* c = new Cache();
     bool sound = share_prefixes && !has_state;
-    for (int g = 0; g < n_groups; ++g) sound = sound && window[g] < 0;
+    for (int g = 0; g < n_groups; ++g) sound = sound && window[g] < 0 && chunk[g] <= 0;
     c->share = sound;
     c->max_requests = max_requests;
     c->groups.resize(n_groups);
@@ -160,6 +167,7 @@ GBH_EXPORT void* gbh_cache_new(int n_groups, const int* num_pages, const int* pa
         gr.num_pages = num_pages[g];
         gr.page_size = page_size[g];
         gr.window = window[g];
+        gr.chunk = chunk[g];
         gr.share = sound;
         gr.refs.assign(gr.num_pages, 0);
         gr.hashed.assign(gr.num_pages, 0);
@@ -270,7 +278,7 @@ GBH_EXPORT int gbh_cache_reserve(void* h, int64_t rid, int n, int* copies, int* 
 }
 
 // Mark n more positions as written; hash pages that became full (kv.rs:205-233); give back pages that a
-// window has passed.
+// window has passed or that lie in a chunk before the next token's.
 GBH_EXPORT int gbh_cache_commit(void* h, int64_t rid, const int32_t* tokens, int n) {
     Cache* c = static_cast<Cache*>(h);
     Request* req = find(c, rid);
@@ -306,7 +314,7 @@ GBH_EXPORT int gbh_cache_commit(void* h, int64_t rid, const int32_t* tokens, int
                 }
             }
         }
-        if (g.window >= 0) {
+        if (g.forgets()) {
             const int live = std::min(g.first_live_page(req->length), (int)table.size());
             for (int bi = 0; bi < live; ++bi)
                 if (table[bi] >= 0) {
@@ -329,7 +337,7 @@ GBH_EXPORT int gbh_cache_commit_many(void* h, int n, const int64_t* rids, const 
     return OK;
 }
 
-// Forget everything after the first `length` tokens (kv.rs:237-257). Not available once a window has
+// Forget everything after the first `length` tokens (kv.rs:237-257). Not available once a window or a chunk has
 // given pages back behind `length`.
 GBH_EXPORT int gbh_cache_truncate(void* h, int64_t rid, int length) {
     Cache* c = static_cast<Cache*>(h);
@@ -337,11 +345,11 @@ GBH_EXPORT int gbh_cache_truncate(void* h, int64_t rid, int length) {
     if (!req) return fail(UNKNOWN_REQUEST, "unknown request");
     if (length > req->length || length < 0) return fail(BAD_VALUE, "cannot truncate to more than is written");
     for (Group& g : c->groups)
-        if (g.window >= 0) {
+        if (g.forgets()) {
             const std::vector<int>& table = g.tables[rid];
             for (size_t i = (size_t)g.first_live_page(length); i < table.size(); ++i)
                 if (table[i] < 0)
-                    return fail(BAD_VALUE, "a windowed group has already released pages that the shorter request would need");
+                    return fail(BAD_VALUE, "a group with a window or chunks has already released pages that the shorter request would need");
         }
     req->length = length;
     if ((int)req->tokens.size() > length) req->tokens.resize(length);

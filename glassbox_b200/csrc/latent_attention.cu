@@ -14,11 +14,14 @@
 //   gb_latent_attention_rows  one warp per (row, head), float32 online softmax; any sizes; the float32 path's kernel
 //                             and the reference beside the tensor-core one
 //
-// Rotation: dimension 2i is paired with 2i+1 over the first `rot_dims` numbers of the rotated part; the pair (u, v) at
-// position p becomes (u cos a - v sin a, v cos a + u sin a), a = float(p) * inv_freq[i], all in float32.
+// Rotation, over the first `rot_dims` numbers of the rotated part: dimension 2i is paired with 2i+1, or (half_pairs) dimension
+// i with i + rot_dims/2; the pair (u, v) at position p becomes (u cos a - v sin a, v cos a + u sin a), a = float(p) *
+// inv_freq[i], sine and cosine times `magnitude`, all in float32.
 #include "common.cuh"
 
 #include <float.h>
+
+constexpr int LAT_MAX_PAIRS = 512;   // rotated pairs at most
 
 // proj: [n, ldp]; the queries are columns 0 .. H*(dq+r)-1, head by head [dq unrotated | r rotated]; for a layer that
 // writes the cache the c + r columns from `kv_col` on are the raw latent and the raw shared key part.
@@ -29,37 +32,37 @@ __global__ void __launch_bounds__(128) latent_kv_write_kernel(
     const T* __restrict__ proj, long long ldp, int kv_col, T* __restrict__ qabs, T* __restrict__ cache,
     const float* __restrict__ latent_gain, const float* __restrict__ inv_freq, const int* __restrict__ positions,
     const int* __restrict__ slots, int n, int H, int dq, int r, int c, int rot_dims, long long num_slots, float eps,
-    int write_kv, int* __restrict__ status) {
+    int write_kv, int half_pairs, float magnitude, int* __restrict__ status) {
     gb_pdl_launch_dependents();
     gb_pdl_wait();
     const int row = blockIdx.x;
     if (row >= n) return;
     const int pos = positions[row];
     if (pos < 0) return;    // a padding row
-    const float fpos = (float)pos;
     const T* prow = proj + (size_t)row * ldp;
-    const int half = rot_dims / 2;
-    // queries: rotated parts, pair by pair
+    const int half = rot_dims / 2, per = half + (r - rot_dims);      // pairs, then numbers that pass unchanged
+    __shared__ float2 cs[LAT_MAX_PAIRS];
+    for (int i = threadIdx.x; i < half; i += blockDim.x) {
+        float sn, c0;
+        sincosf((float)pos * inv_freq[i], &sn, &c0);
+        cs[i] = make_float2(c0 * magnitude, sn * magnitude);
+    }
+    __syncthreads();
+    auto turn = [&](const T* src, T* dst, int k) {       // item k of a rotated part
+        if (k >= half) {
+            dst[rot_dims + k - half] = src[rot_dims + k - half];
+            return;
+        }
+        const int a = half_pairs ? k : 2 * k, b = half_pairs ? k + half : 2 * k + 1;
+        const float u = gb_to_float(src[a]), v = gb_to_float(src[b]);
+        dst[a] = gb_from_float<T>(u * cs[k].x - v * cs[k].y);
+        dst[b] = gb_from_float<T>(v * cs[k].x + u * cs[k].y);
+    };
+    // queries: rotated parts
     T* qrow = qabs + (size_t)row * H * (c + r);
-    for (int idx = threadIdx.x; idx < H * (r / 2 + (r & 1)); idx += blockDim.x) {
-        const int per = r / 2 + (r & 1);
-        const int h = idx / per, i = idx % per;
-        const T* src = prow + (size_t)h * (dq + r) + dq;
-        T* dst = qrow + (size_t)h * (c + r) + c;
-        if (2 * i + 1 >= r) {   // an odd last number passes unchanged
-            dst[2 * i] = src[2 * i];
-            continue;
-        }
-        const float u = gb_to_float(src[2 * i]), v = gb_to_float(src[2 * i + 1]);
-        if (i < half) {
-            float sn, cs;
-            sincosf(fpos * inv_freq[i], &sn, &cs);
-            dst[2 * i] = gb_from_float<T>(u * cs - v * sn);
-            dst[2 * i + 1] = gb_from_float<T>(v * cs + u * sn);
-        } else {
-            dst[2 * i] = src[2 * i];
-            dst[2 * i + 1] = src[2 * i + 1];
-        }
+    for (int idx = threadIdx.x; idx < H * per; idx += blockDim.x) {
+        const int h = idx / per;
+        turn(prow + (size_t)h * (dq + r) + dq, qrow + (size_t)h * (c + r) + c, idx - h * per);
     }
     if (!write_kv) return;
     const long long slot = slots[row];
@@ -83,40 +86,25 @@ __global__ void __launch_bounds__(128) latent_kv_write_kernel(
     __syncthreads();
     const float s = total;
     for (int j = threadIdx.x; j < c; j += blockDim.x) dst[j] = gb_from_float<T>(latent_gain[j] * (gb_to_float(kv[j]) * s));
-    for (int i = threadIdx.x; i < r / 2 + (r & 1); i += blockDim.x) {
-        if (2 * i + 1 >= r) {
-            dst[c + 2 * i] = kv[c + 2 * i];
-            continue;
-        }
-        const float u = gb_to_float(kv[c + 2 * i]), v = gb_to_float(kv[c + 2 * i + 1]);
-        if (i < half) {
-            float sn, cs;
-            sincosf(fpos * inv_freq[i], &sn, &cs);
-            dst[c + 2 * i] = gb_from_float<T>(u * cs - v * sn);
-            dst[c + 2 * i + 1] = gb_from_float<T>(v * cs + u * sn);
-        } else {
-            dst[c + 2 * i] = kv[c + 2 * i];
-            dst[c + 2 * i + 1] = kv[c + 2 * i + 1];
-        }
-    }
+    for (int k = threadIdx.x; k < per; k += blockDim.x) turn(kv + c, dst + c, k);
 }
 
 GB_EXPORT int gb_latent_kv_write(const void* proj, long long ldp, int kv_col, void* qabs, void* cache, int dtype,
                                  const float* latent_gain, const float* inv_freq, const int* positions, const int* slots,
                                  int n, int H, int dq, int r, int c, int rot_dims, long long num_slots, float eps,
-                                 int write_kv, int* status, cudaStream_t stream) {
+                                 int write_kv, int half_pairs, float magnitude, int* status, cudaStream_t stream) {
     GB_REQUIRE(n >= 0 && H > 0 && dq >= 0 && r >= 0 && c > 0, "gb_latent_kv_write: bad sizes");
-    GB_REQUIRE(rot_dims >= 0 && rot_dims <= r && rot_dims % 2 == 0, "gb_latent_kv_write: %d rotated numbers do not fit a part of %d",
+    GB_REQUIRE(rot_dims >= 0 && rot_dims <= r && rot_dims % 2 == 0 && rot_dims / 2 <= LAT_MAX_PAIRS, "gb_latent_kv_write: %d rotated numbers do not fit a part of %d",
                rot_dims, r);
     if (n == 0) return 0;
     if (dtype == GB_F32)
         gb_launch(GB_PDL_ELEMENTWISE, latent_kv_write_kernel<float>, dim3(n), dim3(128), 0, stream, (const float*)proj, ldp, kv_col,
                   (float*)qabs, (float*)cache, latent_gain, inv_freq, positions, slots, n, H, dq, r, c, rot_dims, num_slots, eps,
-                  write_kv, status);
+                  write_kv, half_pairs, magnitude, status);
     else if (dtype == GB_BF16)
         gb_launch(GB_PDL_ELEMENTWISE, latent_kv_write_kernel<__nv_bfloat16>, dim3(n), dim3(128), 0, stream,
                   (const __nv_bfloat16*)proj, ldp, kv_col, (__nv_bfloat16*)qabs, (__nv_bfloat16*)cache, latent_gain, inv_freq,
-                  positions, slots, n, H, dq, r, c, rot_dims, num_slots, eps, write_kv, status);
+                  positions, slots, n, H, dq, r, c, rot_dims, num_slots, eps, write_kv, half_pairs, magnitude, status);
     else
         GB_REQUIRE(false, "gb_latent_kv_write: unsupported dtype %d", dtype);
     return gb_check_launch("gb_latent_kv_write");

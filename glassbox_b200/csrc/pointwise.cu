@@ -6,7 +6,10 @@
 //   add_bias      y[r, :] += bias
 //   clamped_glu   act[r, f] = g * sigmoid(slope * g) * (u + 1), g = min(gate + b, limit), u = clamp(up + b, -limit, limit)
 //   relu2         out = max(in, 0)^2
+//   gelu          out = gelu(in), the exact form
 //   scale         t *= s
+//   tanh_cap      t <- cap * tanh(t / cap)
+//   gate_rows     y[r, :] *= sigmoid(gate[r, :])
 //   gated_head_norm  out[r, h, :] = w * o[r, h, :] / sqrt(mean_v(o[r, h, :]^2) + eps) * sigmoid(gate[r, h, :])  (or * silu(gate))
 //   gelu_glu      act[r, f] = gelu_tanh(gate[r, f]) * up[r, f]
 //   scaled_sum    out (+)= a * x + b * y
@@ -242,6 +245,72 @@ __global__ void scale_kernel(float* __restrict__ t, long long total, float s) {
     gb_pdl_wait();
     long long idx = (long long)blockIdx.x * blockDim.x + threadIdx.x;
     for (; idx < total; idx += (long long)gridDim.x * blockDim.x) t[idx] *= s;
+}
+
+__global__ void tanh_cap_kernel(float* __restrict__ t, long long total, float cap, float inv_cap) {
+    gb_pdl_launch_dependents();
+    gb_pdl_wait();
+    const long long stride = (long long)gridDim.x * blockDim.x;
+    const long long quads = ((uintptr_t)t & 15) == 0 ? total / 4 : 0;
+    for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < quads; i += stride) {
+        float4 v = reinterpret_cast<float4*>(t)[i];
+        v.x = cap * tanhf(v.x * inv_cap); v.y = cap * tanhf(v.y * inv_cap);
+        v.z = cap * tanhf(v.z * inv_cap); v.w = cap * tanhf(v.w * inv_cap);
+        reinterpret_cast<float4*>(t)[i] = v;
+    }
+    for (long long i = 4 * quads + (long long)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += stride) t[i] = cap * tanhf(t[i] * inv_cap);
+}
+
+GB_EXPORT int gb_tanh_cap(float* t, long long total, float cap, cudaStream_t stream) {
+    GB_REQUIRE(total >= 0 && cap > 0.f, "gb_tanh_cap: bad size or cap");
+    if (total == 0) return 0;
+    const long long blocks = (total / 4 + 255) / 256 + 1;
+    gb_launch(GB_PDL_ELEMENTWISE, tanh_cap_kernel, dim3((unsigned)(blocks < 148 * 8 ? blocks : 148 * 8)), dim3(256), 0, stream, t, total, cap, 1.0f / cap);
+    return gb_check_launch("gb_tanh_cap");
+}
+
+template <typename T>
+__global__ void gelu_kernel(const float* __restrict__ in, T* __restrict__ out, long long total) {
+    gb_pdl_launch_dependents();
+    gb_pdl_wait();
+    const long long stride = (long long)gridDim.x * blockDim.x;
+    for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += stride) out[i] = gb_from_float<T>(gb_gelu(in[i]));
+}
+
+GB_EXPORT int gb_gelu(const float* in, void* out, int dtype, long long total, cudaStream_t stream) {
+    GB_REQUIRE(total >= 0 && (dtype == GB_F32 || dtype == GB_BF16), "gb_gelu: bad size or dtype");
+    if (total == 0) return 0;
+    const long long blocks = (total + 255) / 256;
+    const dim3 grid((unsigned)(blocks < 148 * 8 ? blocks : 148 * 8));
+    if (dtype == GB_F32) gb_launch(GB_PDL_ELEMENTWISE, gelu_kernel<float>, grid, dim3(256), 0, stream, in, (float*)out, total);
+    else gb_launch(GB_PDL_ELEMENTWISE, gelu_kernel<__nv_bfloat16>, grid, dim3(256), 0, stream, in, (__nv_bfloat16*)out, total);
+    return gb_check_launch("gb_gelu");
+}
+
+template <typename T, typename TG>
+__global__ void gate_rows_kernel(T* __restrict__ y, const TG* __restrict__ gate, long long ld_gate, int n, int width) {
+    gb_pdl_launch_dependents();
+    gb_pdl_wait();
+    const long long total = (long long)n * width, stride = (long long)gridDim.x * blockDim.x;
+    for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += stride) {
+        const long long r = i / width;
+        y[i] = gb_from_float<T>(gb_to_float(y[i]) / (1.0f + expf(-gb_to_float(gate[r * ld_gate + (i - r * width)]))));
+    }
+}
+
+GB_EXPORT int gb_gate_rows(void* y, int dtype, const void* gate, int gate_dtype, long long ld_gate, int n, int width, cudaStream_t stream) {
+    GB_REQUIRE(n >= 0 && width > 0 && ld_gate >= width, "gb_gate_rows: bad sizes");
+    GB_REQUIRE((dtype == GB_F32 || dtype == GB_BF16) && (gate_dtype == GB_F32 || gate_dtype == GB_BF16), "gb_gate_rows: unsupported dtype");
+    if (n == 0) return 0;
+    const long long blocks = ((long long)n * width + 255) / 256;
+    const dim3 grid((unsigned)(blocks < 148 * 8 ? blocks : 148 * 8));
+#define GR_CASE(T, TG) gb_launch(GB_PDL_ELEMENTWISE, gate_rows_kernel<T, TG>, grid, dim3(256), 0, stream, (T*)y, (const TG*)gate, ld_gate, n, width)
+    if (dtype == GB_F32 && gate_dtype == GB_F32) GR_CASE(float, float);
+    else if (dtype == GB_F32) GR_CASE(float, __nv_bfloat16);
+    else if (gate_dtype == GB_F32) GR_CASE(__nv_bfloat16, float);
+    else GR_CASE(__nv_bfloat16, __nv_bfloat16);
+#undef GR_CASE
+    return gb_check_launch("gb_gate_rows");
 }
 
 GB_EXPORT int gb_scale(float* t, long long total, float s, cudaStream_t stream) {

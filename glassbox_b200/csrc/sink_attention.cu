@@ -1,12 +1,14 @@
 // Softmax attention over the paged cache whose positions enter as a bias on the distance, with a sink in the denominator
 // and a gate on the output. For a row at position p of its request and a key at position j <= p:
-//     s_j = q . k_j * scale - r1[head] * ln(1 + r2[head] * (p - j))                 (r1 == nullptr: no bias)
+//     s_j = q . k_j * scale;  s_j <- cap * tanh(s_j / cap)                           (cap 0: no cap)
+//     s_j <- s_j - r1[head] * ln(1 + r2[head] * (p - j))                             (r1 == nullptr: no bias)
 //     w_j = exp(s_j - m) / (sum_j' exp(s_j' - m) + exp(sink[head] - m))             (sink == nullptr: a plain softmax)
 //     out = sum_j w_j v_j * sigmoid(gate[row, head])                                (gate == nullptr: no gate)
 // With gate_channels the gate has a logit per output channel: out[c] *= sigmoid(gate[row, head * V + c]).
-// The sink has no key and no value: it only takes its share of the weights. The row sees keys max(0, p - window + 1) .. p
-// (window 0: all of them). Query heads share key/value heads in groups; the key size (dim) and the value size (vdim) may
-// differ. Distances, logarithms, scores, weights, sums and the gate are float32. gate holds logits, float32 [n, ld_gate].
+// The sink has no key and no value: it only takes its share of the weights; it is not capped. The row sees keys
+// gb_first_key(p, mask) .. p: all of them, a sliding window (mask > 0) or its own chunk of positions (mask < 0). Query heads
+// share key/value heads in groups; the key size (dim) and the value size (vdim) may differ. Distances, logarithms, scores,
+// weights, sums and the gate are float32. gate holds logits, float32 [n, ld_gate].
 //
 //   sink_attention_rows    one warp per (row, head), any row (prompt portion or single token), both dtypes: 32 keys at a
 //                          time from the first visible one, a lane per key for the scores, a lane per channel for the sum,
@@ -28,7 +30,7 @@ __global__ void __launch_bounds__(SK_WARPS * 32) sink_attention_rows_kernel(
     const T* __restrict__ q, T* __restrict__ out, const T* __restrict__ kcache, const T* __restrict__ vcache,
     const int* __restrict__ block_tables, int max_pages, const int* __restrict__ row_seq, const int* __restrict__ positions,
     const float* __restrict__ r1, const float* __restrict__ r2, const float* __restrict__ sink, const float* __restrict__ gate,
-    long long ld_gate, int n, int H, int G, int D, int V, int page_size, long long num_pages, float scale, int window,
+    long long ld_gate, int n, int H, int G, int D, int V, int page_size, long long num_pages, float scale, float cap, int mask,
     int gate_channels, int* __restrict__ status) {
     __shared__ float qs[SK_WARPS][SA_MAX_DIM];
     gb_pdl_launch_dependents();
@@ -49,7 +51,8 @@ __global__ void __launch_bounds__(SK_WARPS * 32) sink_attention_rows_kernel(
     for (int i = lane; i < D; i += 32) qs[warp][i] = gb_to_float(qrow[i]);
     __syncwarp();
     const float b1 = r1 ? r1[head] : 0.f, b2 = r1 ? r2[head] : 0.f;
-    const int first = (window > 0 && pos + 1 > window) ? pos + 1 - window : 0;
+    const int first = gb_first_key(pos, mask);
+    const float inv_cap = cap > 0.f ? 1.0f / cap : 0.f;
     // the sink starts the running maximum and the denominator: exp(sink - m) with m = sink
     float m = sink ? sink[head] : -INFINITY, l = sink ? 1.f : 0.f;
     float acc[SA_MAX_DIM / 32];
@@ -66,6 +69,7 @@ __global__ void __launch_bounds__(SK_WARPS * 32) sink_attention_rows_kernel(
             } else {
                 at = (page * G + g) * page_size + key % page_size;
                 s = sa_dot<T>(qs[warp], kcache + at * D, D) * scale;
+                if (cap > 0.f) s = cap * tanhf(s * inv_cap);
                 if (r1) s -= sk_distance_bias(b1, b2, pos - key);
             }
         }
@@ -104,14 +108,14 @@ __global__ void __launch_bounds__(SK_WARPS * 32) sink_attention_rows_kernel(
 #define SK_COMMON_CHECKS(name)                                                                                                          \
     GB_REQUIRE(n >= 0 && H > 0 && G > 0 && H % G == 0, name ": heads %d must be a multiple of kv heads %d", H, G);                      \
     GB_REQUIRE(D > 0 && D <= SA_MAX_DIM && V > 0 && V <= SA_MAX_DIM, name ": head sizes %d / %d are outside 1..%d", D, V, SA_MAX_DIM);  \
-    GB_REQUIRE(page_size > 0 && max_pages > 0 && window >= 0, name ": bad page geometry or window");                                    \
+    GB_REQUIRE(page_size > 0 && max_pages > 0 && cap >= 0.f, name ": bad page geometry or cap");                                        \
     GB_REQUIRE((r1 == nullptr) == (r2 == nullptr), name ": the distance bias needs both of its numbers per head");                      \
     GB_REQUIRE(gate == nullptr || ld_gate >= (long long)H * (gate_channels ? V : 1), name ": rows of gate logits are too short");
 
 GB_EXPORT int gb_sink_attention_rows(const void* q, void* out, int dtype, const void* kcache, const void* vcache, const int* block_tables,
                                      int max_pages, const int* row_seq, const int* positions, const float* r1, const float* r2,
                                      const float* sink, const float* gate, long long ld_gate, int n, int H, int G, int D, int V,
-                                     int page_size, long long num_pages, float scale, int window, int gate_channels, int* status,
+                                     int page_size, long long num_pages, float scale, float cap, int mask, int gate_channels, int* status,
                                      cudaStream_t stream) {
     SK_COMMON_CHECKS("gb_sink_attention_rows")
     if (n == 0) return 0;
@@ -119,11 +123,11 @@ GB_EXPORT int gb_sink_attention_rows(const void* q, void* out, int dtype, const 
     if (dtype == GB_F32)
         gb_launch(GB_PDL_ATTENTION, sink_attention_rows_kernel<float>, dim3(blocks), dim3(SK_WARPS * 32), 0, stream, (const float*)q,
                   (float*)out, (const float*)kcache, (const float*)vcache, block_tables, max_pages, row_seq, positions, r1, r2, sink, gate,
-                  ld_gate, n, H, G, D, V, page_size, num_pages, scale, window, gate_channels, status);
+                  ld_gate, n, H, G, D, V, page_size, num_pages, scale, cap, mask, gate_channels, status);
     else if (dtype == GB_BF16)
         gb_launch(GB_PDL_ATTENTION, sink_attention_rows_kernel<__nv_bfloat16>, dim3(blocks), dim3(SK_WARPS * 32), 0, stream,
                   (const __nv_bfloat16*)q, (__nv_bfloat16*)out, (const __nv_bfloat16*)kcache, (const __nv_bfloat16*)vcache, block_tables,
-                  max_pages, row_seq, positions, r1, r2, sink, gate, ld_gate, n, H, G, D, V, page_size, num_pages, scale, window, gate_channels,
+                  max_pages, row_seq, positions, r1, r2, sink, gate, ld_gate, n, H, G, D, V, page_size, num_pages, scale, cap, mask, gate_channels,
                   status);
     else
         GB_REQUIRE(false, "gb_sink_attention_rows: unsupported dtype %d", dtype);
@@ -138,7 +142,7 @@ GB_EXPORT int gb_sink_attention_rows(const void* q, void* out, int dtype, const 
 // whole and dotted with the R queries, the distance bias taken off. Every warp keeps a running maximum and a denominator
 // per head of its own; a lane sums its 16-byte piece of channels over its keys. At the end the lanes that hold the same
 // channels add up (shuffles), then the warps meet in shared memory, where their maxima, the sink's logit and the gate join
-// (fixed order). The order of a row's sums depends on its position and the window alone. A value row must be 64, 128, 256
+// (fixed order). The order of a row's sums depends on its position and the mask alone. A value row must be 64, 128, 256
 // or 512 bytes.
 // ----------------------------------------------------------------------------------------------
 constexpr int SKD_WARPS = 8;
@@ -148,7 +152,7 @@ __global__ void __launch_bounds__(SKD_WARPS * 32) sink_attention_decode_kernel(
     const T* __restrict__ q, T* __restrict__ out, const T* __restrict__ kcache, const T* __restrict__ vcache,
     const int* __restrict__ block_tables, int max_pages, const int* __restrict__ row_seq, const int* __restrict__ positions,
     const float* __restrict__ r1, const float* __restrict__ r2, const float* __restrict__ sink, const float* __restrict__ gate,
-    long long ld_gate, int n, int H, int G, int D, int V, int page_size, long long num_pages, float scale, int window,
+    long long ld_gate, int n, int H, int G, int D, int V, int page_size, long long num_pages, float scale, float cap, int mask,
     int gate_channels, int* __restrict__ status) {
     constexpr int PN = SadPiece<T>::N;          // channels in a 16-byte piece
     constexpr int KPI = 32 / LPK;               // keys that one warp-wide load fetches
@@ -179,7 +183,8 @@ __global__ void __launch_bounds__(SKD_WARPS * 32) sink_attention_decode_kernel(
         m[r] = -INFINITY;
         l[r] = 0.f;
     }
-    const int first = (window > 0 && pos + 1 > window) ? pos + 1 - window : 0;
+    const int first = gb_first_key(pos, mask);
+    const float inv_cap = cap > 0.f ? 1.0f / cap : 0.f;
     const int chunks = (pos - first) / 32 + 1;
     const int sub = lane / LPK, piece = lane % LPK;     // this lane holds piece `piece` of the keys sub, sub + KPI, ...
     float acc[R][PN];
@@ -209,6 +214,7 @@ __global__ void __launch_bounds__(SKD_WARPS * 32) sink_attention_decode_kernel(
 #pragma unroll
             for (int r = 0; r < R; ++r) {
                 s[r] *= scale;
+                if (cap > 0.f) s[r] = cap * tanhf(s[r] * inv_cap);
                 if (r1) s[r] -= sk_distance_bias(b1[r], b2[r], pos - key);
             }
         }
@@ -284,7 +290,7 @@ GB_EXPORT int gb_sink_attention_decode_supported(int value_row_bytes) {
 template <typename T>
 static int skd_launch(const void* q, void* out, const void* kcache, const void* vcache, const int* block_tables, int max_pages,
                       const int* row_seq, const int* positions, const float* r1, const float* r2, const float* sink, const float* gate,
-                      long long ld_gate, int n, int H, int G, int D, int V, int page_size, long long num_pages, float scale, int window,
+                      long long ld_gate, int n, int H, int G, int D, int V, int page_size, long long num_pages, float scale, float cap, int mask,
                       int gate_channels, int* status, cudaStream_t stream) {
     const int lpk = V * (int)sizeof(T) / 16;
     // With enough (row, key/value head) pairs to fill the GPU, the query heads of a group go four at a time through one
@@ -295,7 +301,7 @@ static int skd_launch(const void* q, void* out, const void* kcache, const void* 
     if (lpk == L && (together ? 4 : 1) == RR)                                                                                            \
         gb_launch(GB_PDL_ATTENTION, sink_attention_decode_kernel<T, L, RR>, dim3(n, H / RR), dim3(SKD_WARPS * 32), 0, stream,            \
                   (const T*)q, (T*)out, (const T*)kcache, (const T*)vcache, block_tables, max_pages, row_seq, positions, r1, r2, sink,   \
-                  gate, ld_gate, n, H, G, D, V, page_size, num_pages, scale, window, gate_channels, status);
+                  gate, ld_gate, n, H, G, D, V, page_size, num_pages, scale, cap, mask, gate_channels, status);
     SKD_CASE(4, 1) SKD_CASE(8, 1) SKD_CASE(16, 1) SKD_CASE(32, 1) SKD_CASE(4, 4) SKD_CASE(8, 4) SKD_CASE(16, 4)
 #undef SKD_CASE
     return gb_check_launch("gb_sink_attention_decode");
@@ -304,7 +310,7 @@ static int skd_launch(const void* q, void* out, const void* kcache, const void* 
 GB_EXPORT int gb_sink_attention_decode(const void* q, void* out, int dtype, const void* kcache, const void* vcache,
                                        const int* block_tables, int max_pages, const int* row_seq, const int* positions, const float* r1,
                                        const float* r2, const float* sink, const float* gate, long long ld_gate, int n, int H, int G,
-                                       int D, int V, int page_size, long long num_pages, float scale, int window, int gate_channels, int* status,
+                                       int D, int V, int page_size, long long num_pages, float scale, float cap, int mask, int gate_channels, int* status,
                                        cudaStream_t stream) {
     SK_COMMON_CHECKS("gb_sink_attention_decode")
     GB_REQUIRE(dtype == GB_F32 || dtype == GB_BF16, "gb_sink_attention_decode: unsupported dtype %d", dtype);
@@ -314,17 +320,17 @@ GB_EXPORT int gb_sink_attention_decode(const void* q, void* out, int dtype, cons
     if (n == 0) return 0;
     if (dtype == GB_F32)
         return skd_launch<float>(q, out, kcache, vcache, block_tables, max_pages, row_seq, positions, r1, r2, sink, gate, ld_gate, n, H, G,
-                                 D, V, page_size, num_pages, scale, window, gate_channels, status, stream);
+                                 D, V, page_size, num_pages, scale, cap, mask, gate_channels, status, stream);
     return skd_launch<__nv_bfloat16>(q, out, kcache, vcache, block_tables, max_pages, row_seq, positions, r1, r2, sink, gate, ld_gate, n,
-                                     H, G, D, V, page_size, num_pages, scale, window, gate_channels, status, stream);
+                                     H, G, D, V, page_size, num_pages, scale, cap, mask, gate_channels, status, stream);
 }
 
 // ----------------------------------------------------------------------------------------------
 // Prompt portions in bfloat16 on the tensor cores. A block is 64 consecutive rows of one request x one head; its 4 warps
-// own 16 rows each. The keys any of the 64 rows can see, first_position - window + 1 .. last_position, pass in tiles of 64
+// own 16 rows each. The keys any of the 64 rows can see, gb_first_key(first position) .. last position, pass in tiles of 64
 // through shared memory (cp.async, two buffers, each key's row found through the block table): S = Q K^T with mma.sync
-// m16n8k16; in float32 and in the base-2 domain t = S * (scale * log2 e) - r1 * log2(1 + r2 * distance), the window and the
-// causal edge per element, a running maximum per row that starts at the sink's logit, weights 2^(t - m) rounded to
+// m16n8k16; in float32 and in the base-2 domain t = S * (scale * log2 e) (capped, if there is a cap) - r1 * log2(1 + r2 *
+// distance), the mask's first key and the causal edge per element, a running maximum per row that starts at the sink's logit, weights 2^(t - m) rounded to
 // bfloat16 as the A operand of O += P V (float32 sums), O rescaled when the maximum moves. At the end the sink's share
 // joins the denominator and the gate multiplies the row. Head sizes 32, 64 or 128 for keys and for values, and 48, 80 or 96
 // for both.
@@ -338,7 +344,7 @@ __global__ void __launch_bounds__(128) sink_attention_tiles_kernel(
     const __nv_bfloat16* __restrict__ vcache, const int* __restrict__ block_tables, int max_pages, const int* __restrict__ seq_first_row,
     const int* __restrict__ seq_start_pos, const float* __restrict__ r1, const float* __restrict__ r2, const float* __restrict__ sink,
     const float* __restrict__ gate, long long ld_gate, int num_seqs, int tiles_per_seq, int H, int G, int page_size, long long num_pages,
-    float scale, int window, int gate_channels, int* __restrict__ status) {
+    float scale, float cap, int mask, int gate_channels, int* __restrict__ status) {
     constexpr int LDK = D + 8, LDV = V + 8;          // rows padded by 16 bytes: ldmatrix meets no bank twice
     extern __shared__ __align__(16) unsigned char skt_smem[];
     __nv_bfloat16* sq = reinterpret_cast<__nv_bfloat16*>(skt_smem);             // [64][LDK]
@@ -358,7 +364,7 @@ __global__ void __launch_bounds__(128) sink_attention_tiles_kernel(
         if (threadIdx.x == 0) atomicOr(status, GB_STATUS_BAD_POSITION);
         return;
     }
-    const int k_lo = (window > 0 && p_lo + 1 > window) ? p_lo + 1 - window : 0;
+    const int k_lo = gb_first_key(p_lo, mask);
     const int g = head / (H / G);
     const int* table = block_tables + (size_t)seq * max_pages;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -396,6 +402,8 @@ __global__ void __launch_bounds__(128) sink_attention_tiles_kernel(
     const float sink2 = sink ? sink[head] * SK_LOG2E : -INFINITY;                     // the sink's logit in the base-2 domain
     const float scale2 = scale * SK_LOG2E;
     const int my_pos0 = p_lo + warp * 16 + (lane >> 2), my_pos1 = my_pos0 + 8;       // positions of this thread's two rows
+    const int first0 = gb_first_key(my_pos0, mask), first1 = gb_first_key(my_pos1, mask);
+    const float cap2 = cap * SK_LOG2E, inv_cap2 = cap > 0.f ? 2.0f / cap : 0.f;
     float mrow[2] = {sink2, sink2}, lrow[2] = {0.f, 0.f};                             // (a thread's share of the denominator)
     // The bias depends on the distance alone, and a tile of 64 rows x 64 keys holds 127 distances: one logarithm per thread
     // and tile instead of one per score. sbias[i] belongs to the distance (p_lo - kb) + i - 63, which is row - key + 63
@@ -420,10 +428,10 @@ __global__ void __launch_bounds__(128) sink_attention_tiles_kernel(
                              : "=r"(qf[kd][0]), "=r"(qf[kd][1]), "=r"(qf[kd][2]), "=r"(qf[kd][3]) : "r"(addr));
             }
         }
-        // a warp whose rows lie wholly before this tile's first key or (with a window) wholly behind its last visible one
+        // a warp whose rows lie wholly before this tile's first key or (with a window or chunks) see none of its keys
         // still walks the barriers, but skips the arithmetic
         const int w_lo = p_lo + warp * 16, w_hi = w_lo + 15;
-        const bool any = kb <= w_hi && (window <= 0 || kb + SKT_BN - 1 > w_lo - window) && warp * 16 < rows;
+        const bool any = kb <= w_hi && kb + SKT_BN > gb_first_key(w_lo, mask) && warp * 16 < rows;
         if (any) {
             float s[SKT_BN / 8][4];
 #pragma unroll
@@ -445,9 +453,9 @@ __global__ void __launch_bounds__(128) sink_attention_tiles_kernel(
                                  : "r"(qf[kd][0]), "r"(qf[kd][1]), "r"(qf[kd][2]), "r"(qf[kd][3]), "r"(b2_), "r"(b3));
                 }
             }
-            // base-2 logits with the distance bias; the causal edge and the window per element, except in tiles that every
+            // base-2 logits with the cap and the distance bias; the causal edge and the first visible key per element, except in tiles that every
             // row of the warp sees whole (most of them); then the rows' maxima (a row lies in the four lanes of a quad)
-            const bool whole = kb + SKT_BN - 1 <= w_lo && (window <= 0 || w_hi - kb < window) && w_hi <= p_hi;
+            const bool whole = kb + SKT_BN - 1 <= w_lo && kb >= gb_first_key(w_hi, mask) && w_hi <= p_hi;
             float mx[2] = {mrow[0], mrow[1]};
 #pragma unroll
             for (int j = 0; j < SKT_BN / 8; ++j) {
@@ -455,10 +463,10 @@ __global__ void __launch_bounds__(128) sink_attention_tiles_kernel(
                 for (int e = 0; e < 4; ++e) {
                     const int key = kb + j * 8 + (lane & 3) * 2 + (e & 1);
                     const int pos = e < 2 ? my_pos0 : my_pos1;
-                    float v = s[j][e] * scale2;
+                    float v = cap > 0.f ? gb_cap_fast(s[j][e] * scale, cap2, inv_cap2) : s[j][e] * scale2;
                     if (r1) v -= my_bias[(e >> 1) * 8 - j * 8 - (e & 1)];
                     if (!whole) {
-                        const bool sees = key <= pos && (window <= 0 || pos - key < window) && pos <= p_hi;
+                        const bool sees = key <= pos && key >= (e < 2 ? first0 : first1) && pos <= p_hi;
                         v = sees ? v : -INFINITY;
                     }
                     s[j][e] = v;
@@ -547,20 +555,20 @@ template <int D, int V>
 static int skt_launch(const void* q, void* out, const void* kcache, const void* vcache, const int* block_tables, int max_pages,
                       const int* seq_first_row, const int* seq_start_pos, const float* r1, const float* r2, const float* sink,
                       const float* gate, long long ld_gate, int num_seqs, int tiles_per_seq, int H, int G, int page_size,
-                      long long num_pages, float scale, int window, int gate_channels, int* status, cudaStream_t stream) {
+                      long long num_pages, float scale, float cap, int mask, int gate_channels, int* status, cudaStream_t stream) {
     const size_t smem = ((size_t)3 * SKT_BM * (D + 8) + (size_t)2 * SKT_BN * (V + 8)) * 2;
     cudaFuncSetAttribute(sink_attention_tiles_kernel<D, V>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     gb_launch(GB_PDL_ATTENTION, sink_attention_tiles_kernel<D, V>, dim3(num_seqs * tiles_per_seq, H), dim3(128), smem, stream,
               (const __nv_bfloat16*)q, (__nv_bfloat16*)out, (const __nv_bfloat16*)kcache, (const __nv_bfloat16*)vcache, block_tables,
               max_pages, seq_first_row, seq_start_pos, r1, r2, sink, gate, ld_gate, num_seqs, tiles_per_seq, H, G, page_size, num_pages,
-              scale, window, gate_channels, status);
+              scale, cap, mask, gate_channels, status);
     return gb_check_launch("gb_sink_attention_tiles");
 }
 
 GB_EXPORT int gb_sink_attention_tiles(const void* q, void* out, const void* kcache, const void* vcache, const int* block_tables,
                                       int max_pages, const int* seq_first_row, const int* seq_start_pos, const float* r1, const float* r2,
                                       const float* sink, const float* gate, long long ld_gate, int num_seqs, int max_rows_per_seq, int H,
-                                      int G, int D, int V, int page_size, long long num_pages, float scale, int window, int gate_channels,
+                                      int G, int D, int V, int page_size, long long num_pages, float scale, float cap, int mask, int gate_channels,
                                       int* status, cudaStream_t stream) {
     const int n = num_seqs;
     SK_COMMON_CHECKS("gb_sink_attention_tiles")
@@ -571,7 +579,7 @@ GB_EXPORT int gb_sink_attention_tiles(const void* q, void* out, const void* kcac
 #define SKT_CASE(DD, VV)                                                                                                              \
     if (D == DD && V == VV)                                                                                                           \
         return skt_launch<DD, VV>(q, out, kcache, vcache, block_tables, max_pages, seq_first_row, seq_start_pos, r1, r2, sink, gate,   \
-                                  ld_gate, num_seqs, tiles, H, G, page_size, num_pages, scale, window, gate_channels, status, stream);
+                                  ld_gate, num_seqs, tiles, H, G, page_size, num_pages, scale, cap, mask, gate_channels, status, stream);
     SKT_CASE(32, 32) SKT_CASE(32, 64) SKT_CASE(32, 128) SKT_CASE(64, 32) SKT_CASE(64, 64) SKT_CASE(64, 128) SKT_CASE(128, 32)
     SKT_CASE(128, 64) SKT_CASE(128, 128) SKT_CASE(48, 48) SKT_CASE(80, 80) SKT_CASE(96, 96)
 #undef SKT_CASE

@@ -81,7 +81,7 @@ class Engine:
         pages_for = group_pages if group_pages is not None else (lambda spec: self.num_pages)
         self.device_cache = DeviceCache(layer_specs, pages_for, self.page_size, self.max_requests, self.dtype, self.device)
         groups = [GroupSpec(num_pages=self.device_cache.group_pages[i], page_size=self.page_size, window=s.window,
-                            name=f"group{i}") for i, s in enumerate(self.device_cache.group_specs)]
+                            name=f"group{i}", chunk=s.chunk) for i, s in enumerate(self.device_cache.group_specs)]
         self.cache = CacheManager(groups, max_requests=self.max_requests, share_prefixes=share_prefixes,
                                   has_state=self.device_cache.has_state)
         self.status = torch.zeros(1, dtype=torch.int32, device=self.device)

@@ -228,7 +228,7 @@ class Scheduler:
         group that keeps a window of keys only ever holds the window and one step's rows of a request."""
         cache = self.backend.cache
         for g, group in enumerate(cache.groups):
-            held = span if group.window is None else min(span, group.window + self.config.token_budget)
+            held = span if group.reach is None else min(span, group.reach + self.config.token_budget)
             if cache.free_pages(g) < cache.pages_needed(held, g) + 1:
                 return False
         return True

@@ -58,7 +58,7 @@ _SIGNATURES = {
     "gb_attention_decode_mma_pdl": [_P, _LL, _P, _LL, _P, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _LL, _F, _I, _I, _P, _P,
                                     _P, _P, _I, _I, _I, _P],
     "gb_attention_decode_mma_sink": [_P, _LL, _P, _LL, _P, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _LL, _F, _I, _I, _P, _P,
-                                     _P, _P, _I, _I, _I, _P, _P, _P, _P, _LL, _I, _P],
+                                     _P, _P, _I, _I, _I, _P, _P, _P, _P, _LL, _I, _F, _P],
     "gb_attention_decode_mma": [_P, _LL, _P, _LL, _P, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _LL, _F, _I, _I, _P, _P, _P,
                                 _P, _P],
     "gb_attention_decode_mma_supported": [_I, _I, _I],
@@ -71,7 +71,7 @@ _SIGNATURES = {
     "gb_gemm_tcgen05_qkv_supported": [_I],
     "gb_attention_prefill_tc": [_P, _LL, _I, _P, _LL, _P, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _I, _LL, _F, _I, _P, _P],
     "gb_attention_prefill_tc_sink": [_P, _LL, _I, _P, _LL, _P, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _I, _LL, _F, _I, _P, _P, _P,
-                                     _P, _P, _LL, _I, _P],
+                                     _P, _P, _LL, _I, _F, _P],
     "gb_attention_prefill_tc_supported": [_I, _I, _I, _I],
     "gb_gemm_tcgen05": [_P, _P, _P, _I, _I, _I, _I, _LL, _LL, _LL, _P, _P, _P, _P, _LL, _P, _P, _I, _F],
     "gb_gemm_tcgen05_column_tiles": [_I, _I, _I],
@@ -94,14 +94,19 @@ _SIGNATURES = {
     "gb_clamped_glu": [_P, _I, _LL, _P, _F, _F, _P, _I, _I, _I, _P],
     "gb_relu2": [_P, _P, _I, _LL, _P],
     "gb_scale": [_P, _LL, _F, _P],
+    "gb_tanh_cap": [_P, _LL, _F, _P],
+    "gb_gelu": [_P, _P, _I, _LL, _P],
+    "gb_gate_rows": [_P, _I, _P, _I, _LL, _I, _I, _P],
     "gb_gated_head_norm": [_P, _P, _LL, _P, _P, _I, _I, _I, _I, _F, _I, _P],
-    "gb_latent_kv_write": [_P, _LL, _I, _P, _P, _I, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _LL, _F, _I, _P, _P],
+    "gb_latent_kv_write": [_P, _LL, _I, _P, _P, _I, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _LL, _F, _I, _I, _F, _P, _P],
+    "gb_latent_inputs": [_P, _LL, _P, _P, _P, _F, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _LL, _F, _I, _P, _P],
+    "gb_projection_norm_rope_write": [_P, _LL, _P, _P, _P, _F, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _F, _I, _LL, _I, _P, _P],
     "gb_latent_attention_rows": [_P, _P, _I, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _LL, _F, _I, _P, _P],
     "gb_latent_attention_mma_supported": [_I, _I, _I],
     "gb_latent_attention_mma": [_P, _P, _P, _P, _P, _P, _I, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _LL, _F, _I, _I, _I,
                                 _P, _P],
     "gb_head_linear_supported": [_P, _LL, _LL, _P, _P, _LL, _LL, _I, _I],
-    "gb_head_linear": [_P, _LL, _LL, _P, _P, _LL, _LL, _I, _I, _I, _I, _P],
+    "gb_head_linear": [_P, _LL, _LL, _P, _P, _LL, _LL, _I, _I, _I, _I, _P, _LL, _I, _P],
     "gb_embed_positions": [_P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _F, _P, _P],
     "gb_residual_conv": [_P, _I, _P, _I, _P, _P, _LL, _LL, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _P, _P],
     "gb_gelu_glu": [_P, _I, _LL, _P, _I, _I, _I, _P],
@@ -124,11 +129,11 @@ _SIGNATURES = {
     "gb_streams_step": [_P, _I, _I, _P, _LL, _P, _P, _I, _P, _LL, _P, _P, _P, _P, _P, _P, _F, _P, _I, _P, _P, _P, _I, _I, _P],
     "gb_qk_norm_rope_write": [_P, _LL, _P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _F, _I, _LL, _I, _P, _P, _P, _LL,
                               _P, _I, _F, _F, _P],
-    "gb_sink_attention_rows": [_P, _P, _I, _P, _P, _P, _I, _P, _P, _P, _P, _P, _P, _LL, _I, _I, _I, _I, _I, _I, _LL, _F, _I, _I, _P, _P],
-    "gb_sink_attention_decode": [_P, _P, _I, _P, _P, _P, _I, _P, _P, _P, _P, _P, _P, _LL, _I, _I, _I, _I, _I, _I, _LL, _F, _I, _I, _P, _P],
+    "gb_sink_attention_rows": [_P, _P, _I, _P, _P, _P, _I, _P, _P, _P, _P, _P, _P, _LL, _I, _I, _I, _I, _I, _I, _LL, _F, _F, _I, _I, _P, _P],
+    "gb_sink_attention_decode": [_P, _P, _I, _P, _P, _P, _I, _P, _P, _P, _P, _P, _P, _LL, _I, _I, _I, _I, _I, _I, _LL, _F, _F, _I, _I, _P, _P],
     "gb_sink_attention_decode_supported": [_I],
     "gb_sink_attention_tiles_supported": [_I, _I],
-    "gb_sink_attention_tiles": [_P, _P, _P, _P, _P, _I, _P, _P, _P, _P, _P, _P, _LL, _I, _I, _I, _I, _I, _I, _I, _LL, _F, _I, _I, _P, _P],
+    "gb_sink_attention_tiles": [_P, _P, _P, _P, _P, _I, _P, _P, _P, _P, _P, _P, _LL, _I, _I, _I, _I, _I, _I, _I, _LL, _F, _F, _I, _I, _P, _P],
     "gb_sigmoid_attention_rows": [_P, _P, _I, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _LL, _F, _I, _P, _P],
     "gb_sigmoid_attention_decode": [_P, _P, _I, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _LL, _F, _I, _P, _P],
     "gb_sigmoid_attention_decode_supported": [_I],
@@ -502,7 +507,7 @@ def _prefetch_args(t: Optional[torch.Tensor]):
 
 
 def gemm_stream(a: torch.Tensor, w: torch.Tensor, c: torch.Tensor, accumulate: bool = False, gated: bool = False,
-                norm=None, prefetch: Optional[torch.Tensor] = None, relu2: bool = False) -> None:
+                norm=None, prefetch: Optional[torch.Tensor] = None, relu2: bool = False, gelu: bool = False) -> None:
     """c[M, N] (+)= a[M, K] @ w[N, K]^T for M <= 64 on the tensor cores, streaming w once. With
     ``gated``, w is [2I, K] (gate rows, then up rows) and c[M, I] = silu(a gate^T) * (a up^T). With
     ``norm`` = (gain, eps), ``a`` is the float32 residual and is RMS-normalised on the way in.
@@ -514,9 +519,9 @@ def gemm_stream(a: torch.Tensor, w: torch.Tensor, c: torch.Tensor, accumulate: b
     if gated:
         assert c.dtype == torch.bfloat16 and not accumulate
         mode = 3
-    elif relu2:                      # c = bfloat16(max(a w^T, 0)^2)
-        assert c.dtype == torch.bfloat16 and not accumulate
-        mode = 5
+    elif relu2 or gelu:              # c = bfloat16(max(a w^T, 0)^2), or bfloat16(gelu(a w^T))
+        assert c.dtype == torch.bfloat16 and not accumulate and not (relu2 and gelu)
+        mode = 5 if relu2 else 7
     elif accumulate:
         assert c.dtype == torch.float32
         mode = 2
@@ -601,7 +606,8 @@ def gemm_tc_column_tiles(rows: int, n: int, k: int) -> int:
 
 
 def gemm_tc(a: torch.Tensor, w: torch.Tensor, c: torch.Tensor, accumulate: bool = False,
-            status: Optional[torch.Tensor] = None, prepare=None, row_scale: Optional[RowScale] = None, relu2: bool = False) -> None:
+            status: Optional[torch.Tensor] = None, prepare=None, row_scale: Optional[RowScale] = None, relu2: bool = False,
+            gelu: bool = False) -> None:
     """c[M, N] (+)= a[M, K] @ w[N, K]^T with TMA + tcgen05.mma + TMEM. ``status`` receives the
     wait-timeout bit if a bounded wait inside the kernel ever gives up.
 
@@ -625,9 +631,9 @@ def gemm_tc(a: torch.Tensor, w: torch.Tensor, c: torch.Tensor, accumulate: bool 
         status = _tc_status.get(a.device)
         if status is None:
             status = _tc_status[a.device] = torch.zeros(1, dtype=torch.int32, device=a.device)
-    if relu2:                        # c = bfloat16(max(a w^T, 0)^2)
-        assert c.dtype == torch.bfloat16 and not accumulate
-        mode = 4
+    if relu2 or gelu:                # c = bfloat16(max(a w^T, 0)^2), or bfloat16(gelu(a w^T))
+        assert c.dtype == torch.bfloat16 and not accumulate and not (relu2 and gelu)
+        mode = 4 if relu2 else 5
     elif accumulate:
         assert c.dtype == torch.float32
         mode = 2
@@ -818,12 +824,14 @@ def attention_decode_mma(q: torch.Tensor, out: torch.Tensor, kcache: torch.Tenso
                          block_tables: torch.Tensor, row_seq: torch.Tensor, positions: torch.Tensor, nh: int, nkv: int,
                          hd: int, page_size: int, scale: float, window: Optional[int], splits: int,
                          part_acc: torch.Tensor, part_ml: torch.Tensor, counters: torch.Tensor,
-                         status: torch.Tensor, block_keys: int = 0, warps: int = 4, sink_terms=None) -> None:
+                         status: torch.Tensor, block_keys: int = 0, warps: int = 4, sink_terms=None,
+                         softcap: Optional[float] = None, chunk: Optional[int] = None) -> None:
     """bfloat16 split-key decode attention on the tensor cores. Scratch: part_acc float32
     [n, nh, warps*splits, hd], part_ml float32 [n, nh, warps*splits, 2], counters int32 [n*nkv], zero on entry
     and left zero. ``warps`` per block: 4, or 8 (head size 64). ``sink_terms`` = (r1, r2, sink, gate), each a float32
     tensor or None as in ``sink_attention_rows``: the softmax then has a distance bias, a sink in its denominator and a
-    sigmoid gate on each head's output (the kernel's instantiation for these terms; never part of a decode program)."""
+    sigmoid gate on each head's output (the kernel's instantiation for these terms; never part of a decode program), and takes
+    ``softcap`` and ``chunk`` as in ``sink_attention_rows``."""
     _cuda(q, out, kcache, vcache, block_tables, row_seq, positions, part_acc, part_ml, counters, status)
     n = q.shape[0]
     assert q.dtype == out.dtype == kcache.dtype == torch.bfloat16 and q.stride(1) == 1 and out.stride(1) == 1
@@ -839,9 +847,10 @@ def attention_decode_mma(q: torch.Tensor, out: torch.Tensor, kcache: torch.Tenso
         terms, by_channel = _sink_args(r1, r2, sink, gate, nh, hd)
         _call("gb_attention_decode_mma_sink", _ptr(q), q.stride(0), _ptr(out), out.stride(0), _ptr(kcache), _ptr(vcache),
               _ptr(block_tables), block_tables.shape[1], _ptr(row_seq), _ptr(positions), n, nh, nkv, hd, page_size,
-              kcache.shape[0], float(scale), int(window or 0), int(splits), _ptr(part_acc), _ptr(part_ml), _ptr(counters),
-              _ptr(status), 1 if USE_PDL else 0, int(block_keys), int(warps), *terms, by_channel, _stream())
+              kcache.shape[0], float(scale), _mask(window, chunk), int(splits), _ptr(part_acc), _ptr(part_ml), _ptr(counters),
+              _ptr(status), 1 if USE_PDL else 0, int(block_keys), int(warps), *terms, by_channel, float(softcap or 0.0), _stream())
         return
+    assert softcap is None and chunk is None
     if prog is not None and prog.takes_rows(n):
         if not prog.takes_attention(hd, block_keys):
             prog.flush()
@@ -872,11 +881,13 @@ def attention_prefill_tc_supported(q: torch.Tensor, out: torch.Tensor, nh: int, 
 def attention_prefill_tc(q: torch.Tensor, out: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor,
                          block_tables: torch.Tensor, seq_first_row: torch.Tensor, seq_start_pos: torch.Tensor,
                          max_rows_per_seq: int, nh: int, nkv: int, hd: int, page_size: int, scale: float,
-                         window: Optional[int], status: torch.Tensor, sink_terms=None) -> None:
+                         window: Optional[int], status: torch.Tensor, sink_terms=None, softcap: Optional[float] = None,
+                         chunk: Optional[int] = None) -> None:
     """bfloat16 flash attention on tcgen05 (TMA loads from the paged cache, S and PV in tensor memory) for
     batches whose requests bring runs of consecutive rows; arguments as ``attention_prefill``. ``sink_terms`` =
     (r1, r2, sink, gate), each a float32 tensor or None as in ``sink_attention_rows``: the kernel's instantiation whose
-    softmax has a distance bias, a sink in its denominator and a sigmoid gate on each head's output."""
+    softmax has a distance bias, a sink in its denominator and a sigmoid gate on each head's output, and which takes
+    ``softcap`` and ``chunk`` as described there."""
     _cuda(q, out, kcache, vcache, block_tables, seq_first_row, seq_start_pos, status)
     assert q.dtype == out.dtype == kcache.dtype == torch.bfloat16 and q.stride(1) == 1 and out.stride(1) == 1
     assert block_tables.dtype == torch.int32 and block_tables.is_contiguous()
@@ -889,9 +900,10 @@ def attention_prefill_tc(q: torch.Tensor, out: torch.Tensor, kcache: torch.Tenso
         terms, by_channel = _sink_args(r1, r2, sink, gate, nh, hd)
         _call("gb_attention_prefill_tc_sink", _ptr(q), q.stride(0), q.shape[0], _ptr(out), out.stride(0), _ptr(kcache),
               _ptr(vcache), _ptr(block_tables), block_tables.shape[1], _ptr(seq_first_row), _ptr(seq_start_pos), S,
-              int(max_rows_per_seq), nh, nkv, hd, page_size, kcache.shape[0], float(scale), int(window or 0), _ptr(status),
-              *terms, by_channel, _stream())
+              int(max_rows_per_seq), nh, nkv, hd, page_size, kcache.shape[0], float(scale), _mask(window, chunk), _ptr(status),
+              *terms, by_channel, float(softcap or 0.0), _stream())
         return
+    assert softcap is None and chunk is None
     _call("gb_attention_prefill_tc", _ptr(q), q.stride(0), q.shape[0], _ptr(out), out.stride(0), _ptr(kcache),
           _ptr(vcache), _ptr(block_tables), block_tables.shape[1], _ptr(seq_first_row), _ptr(seq_start_pos), S,
           int(max_rows_per_seq), nh, nkv, hd, page_size, kcache.shape[0], float(scale), int(window or 0), _ptr(status),
@@ -1016,6 +1028,27 @@ def scale_(t: torch.Tensor, s: float) -> None:
     _call("gb_scale", _ptr(t), t.numel(), float(s), _stream())
 
 
+def tanh_cap_(t: torch.Tensor, cap: float) -> None:
+    """t <- cap * tanh(t / cap) in place (float32)."""
+    _cuda(t)
+    assert t.dtype == torch.float32 and t.is_contiguous()
+    _call("gb_tanh_cap", _ptr(t), t.numel(), float(cap), _stream())
+
+
+def gelu(h: torch.Tensor, out: torch.Tensor) -> None:
+    """out = h / 2 * (1 + erf(h / sqrt 2)), element by element; h float32."""
+    _cuda(h, out)
+    assert h.dtype == torch.float32 and h.shape == out.shape and h.is_contiguous() and out.is_contiguous()
+    _call("gb_gelu", _ptr(h), _ptr(out), _dt(out), h.numel(), _stream())
+
+
+def gate_rows_(y: torch.Tensor, gate: torch.Tensor) -> None:
+    """y *= sigmoid(gate), in place; the gate's rows may be strided."""
+    _cuda(y, gate)
+    assert y.is_contiguous() and gate.shape == y.shape and gate.stride(1) == 1
+    _call("gb_gate_rows", _ptr(y), _dt(y), _ptr(gate), _dt(gate), gate.stride(0), y.shape[0], y.shape[1], _stream())
+
+
 def gated_head_norm(o: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, heads: int, eps: float,
                     gate_silu: bool = False) -> None:
     """out[r, h, :] = weight * o[r, h, :] / sqrt(mean(o[r, h, :]^2) + eps) * sigmoid(gate[r, h, :]); o, gate, weight
@@ -1048,10 +1081,11 @@ def scaled_sum(x: torch.Tensor, y: torch.Tensor, a: float, b: float, out: torch.
 # ------------------------------------------------------------------------------- attention over a latent cache
 def latent_kv_write(proj: torch.Tensor, kv_col: int, qabs: torch.Tensor, cache: torch.Tensor, latent_gain: Optional[torch.Tensor],
                     inv_freq: torch.Tensor, positions: torch.Tensor, slots: torch.Tensor, heads: int, dq: int, r: int, c: int,
-                    rot_dims: int, eps: float, write_kv: bool, status: torch.Tensor) -> None:
+                    rot_dims: int, eps: float, write_kv: bool, status: torch.Tensor, half_pairs: bool = False, magnitude: float = 1.0) -> None:
     """Rotate every head's rotated query part of ``proj`` [n, >= heads * (dq + r)] into ``qabs`` [n, heads, c + r][..., c:];
     with ``write_kv`` also RMS-norm the raw latent (columns kv_col .. kv_col + c), rotate the raw shared key part behind it
-    and store both at each row's slot of ``cache`` [pages, 1, page_size, c + r]."""
+    and store both at each row's slot of ``cache`` [pages, 1, page_size, c + r]. ``half_pairs``: number i turns with number
+    i + rot_dims/2, not neighbour with neighbour; ``magnitude`` multiplies sine and cosine."""
     _cuda(proj, qabs, cache, latent_gain, inv_freq, positions, slots, status)
     n = proj.shape[0]
     assert proj.stride(1) == 1 and qabs.is_contiguous() and cache.is_contiguous() and proj.dtype == qabs.dtype == cache.dtype
@@ -1060,7 +1094,24 @@ def latent_kv_write(proj: torch.Tensor, kv_col: int, qabs: torch.Tensor, cache: 
     num_slots = cache.numel() // (c + r)
     _call("gb_latent_kv_write", _ptr(proj), proj.stride(0), kv_col, _ptr(qabs), _ptr(cache), _dt(proj), _ptr(latent_gain),
           _ptr(inv_freq), _ptr(positions), _ptr(slots), n, heads, dq, r, c, rot_dims, num_slots, float(eps),
-          1 if write_kv else 0, _ptr(status), _stream())
+          1 if write_kv else 0, 1 if half_pairs else 0, float(magnitude), _ptr(status), _stream())
+
+
+def latent_inputs(proj: torch.Tensor, q_gain: torch.Tensor, latent_gain: Optional[torch.Tensor], inv_freq: torch.Tensor, magnitude: float,
+                  positions: torch.Tensor, slots: torch.Tensor, cq: torch.Tensor, cache: torch.Tensor, c: int, r: int, rot_dims: int,
+                  eps: float, write_kv: bool, status: torch.Tensor) -> None:
+    """From the float32 sums of the stacked projection query latent | latent | shared key part: ``cq`` [n, q_rank] = the query
+    latent, RMS-normed with its gain; with ``write_kv`` the latent, RMS-normed, and the key part, rotated (number i with number
+    i + rot_dims/2, sine and cosine times ``magnitude``), go to each row's slot of ``cache`` [pages, 1, page_size, c + r]."""
+    _cuda(proj, q_gain, latent_gain, inv_freq, positions, slots, cq, cache, status)
+    n, qr = cq.shape
+    assert proj.dtype == torch.float32 and proj.stride(1) == 1 and proj.shape[0] == n and proj.shape[1] >= qr + (c + r if write_kv else 0)
+    assert cq.is_contiguous() and cache.is_contiguous() and cq.dtype == cache.dtype and cache.shape[-1] == c + r
+    assert q_gain.dtype == torch.float32 and q_gain.numel() == qr and (latent_gain is None or latent_gain.numel() == c)
+    assert inv_freq.dtype == torch.float32 and inv_freq.numel() >= rot_dims // 2
+    _call("gb_latent_inputs", _ptr(proj), proj.stride(0), _ptr(q_gain), _ptr(latent_gain), _ptr(inv_freq), float(magnitude), _ptr(positions),
+          _ptr(slots), _ptr(cq), _ptr(cache), _dt(cq), n, qr, c, r, rot_dims, cache.numel() // (c + r), float(eps), 1 if write_kv else 0,
+          _ptr(status), _stream())
 
 
 def latent_attention_rows(q: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, block_tables: torch.Tensor,
@@ -1088,14 +1139,17 @@ def head_linear_supported(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, a
                                                w.shape[1], w.shape[2]))
 
 
-def head_linear(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, a_head: int, c_head: int) -> None:
+def head_linear(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, a_head: int, c_head: int, gate: Optional[torch.Tensor] = None) -> None:
     """out[row, h * c_head : h * c_head + N] = a[row, h * a_head : h * a_head + K] @ w[h]^T for every head h of
-    w [heads, N, K], in one launch (bfloat16, float32 sums)."""
-    _cuda(a, w, out)
+    w [heads, N, K], in one launch (bfloat16, float32 sums). ``gate`` [n, heads * N] (float32 or bfloat16 logits, rows may be
+    strided): every output is multiplied by sigmoid(gate[row, h * N + column]) first."""
+    _cuda(a, w, out, gate)
+    assert gate is None or (gate.shape == (a.shape[0], w.shape[0] * w.shape[1]) and gate.stride(1) == 1)
     heads, N, K = w.shape
     n = a.shape[0]
     assert out.shape[0] == n and a.shape[1] >= (heads - 1) * a_head + K and out.shape[1] >= (heads - 1) * c_head + N
-    _call("gb_head_linear", _ptr(a), a.stride(0), a_head, _ptr(w), _ptr(out), out.stride(0), c_head, n, heads, N, K, _stream())
+    _call("gb_head_linear", _ptr(a), a.stride(0), a_head, _ptr(w), _ptr(out), out.stride(0), c_head, n, heads, N, K, _ptr(gate),
+          gate.stride(0) if gate is not None else 0, 1 if gate is not None and gate.dtype == torch.float32 else 0, _stream())
 
 
 def latent_attention_mma_supported(dtype: torch.dtype, c: int, r: int, page_size: int) -> bool:
@@ -1604,6 +1658,27 @@ def qk_norm_rope_write(qkv: torch.Tensor, q_gain: Optional[torch.Tensor], k_gain
           float(q_temp[1]) if q_temp else 0.0, _stream())
 
 
+def projection_norm_rope_write(qkv: torch.Tensor, q_gain: Optional[torch.Tensor], k_gain: Optional[torch.Tensor],
+                               inv_freq: Optional[torch.Tensor], magnitude: float, positions: torch.Tensor, slots: torch.Tensor,
+                               q_out: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor, heads: int, kv_heads: int, dim: int,
+                               vdim: int, rot: int, eps: float, page_size: int, write_kv: bool, status: torch.Tensor) -> None:
+    """From the float32 sums of the stacked projection q | k | v: RMS norm over all query channels at once and over all key
+    channels at once (a gain per channel; None: no norm), rotation of the first ``rot`` channels of every head (channel i with
+    channel i + rot/2, by float32(position) * inv_freq[i], sine and cosine times ``magnitude``), q into ``q_out`` [n, heads * dim],
+    k and v into the paged cache at each row's slot."""
+    _cuda(qkv, q_gain, k_gain, inv_freq, positions, slots, q_out, kcache, vcache, status)
+    n = qkv.shape[0]
+    assert qkv.dtype == torch.float32 and qkv.stride(1) == 1 and qkv.shape[1] == (heads + kv_heads) * dim + kv_heads * vdim
+    assert q_gain is None or (q_gain.dtype == torch.float32 and q_gain.numel() == heads * dim and q_gain.is_contiguous())
+    assert k_gain is None or (k_gain.dtype == torch.float32 and k_gain.numel() == kv_heads * dim and k_gain.is_contiguous())
+    assert q_out.shape == (n, heads * dim) and q_out.is_contiguous() and q_out.dtype == kcache.dtype == vcache.dtype
+    assert kcache.is_contiguous() and vcache.is_contiguous() and kcache.shape[-1] == dim and vcache.shape[-1] == vdim
+    assert rot == 0 or (inv_freq is not None and inv_freq.dtype == torch.float32 and inv_freq.numel() == rot // 2)
+    _call("gb_projection_norm_rope_write", _ptr(qkv), qkv.stride(0), _ptr(q_gain), _ptr(k_gain), _ptr(inv_freq), float(magnitude),
+          _ptr(positions), _ptr(slots), _ptr(q_out), _ptr(kcache), _ptr(vcache), _dt(q_out), n, heads, kv_heads, dim, vdim, rot, float(eps),
+          page_size, kcache.shape[0] * page_size, 1 if write_kv else 0, _ptr(status), _stream())
+
+
 def sigmoid_attention_rows(q: torch.Tensor, out: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor, block_tables: torch.Tensor,
                            row_seq: torch.Tensor, positions: torch.Tensor, head_bias: Optional[torch.Tensor], heads: int, kv_heads: int,
                            dim: int, vdim: int, page_size: int, scale: float, window: Optional[int], status: torch.Tensor) -> None:
@@ -1661,6 +1736,12 @@ def sigmoid_attention_tiles(q: torch.Tensor, out: torch.Tensor, kcache: torch.Te
 
 
 # ------------------------------------------------------- softmax attention with a distance bias, a sink and an output gate
+def _mask(window: Optional[int], chunk: Optional[int]) -> int:
+    """Which keys a query sees, as one number for the launchers: a sliding window (positive), chunks (negative), all (0)."""
+    assert not (window and chunk), "a window and chunks at once"
+    return -int(chunk) if chunk else int(window or 0)
+
+
 def _sink_args(r1, r2, sink, gate, heads, vdim):
     """The four terms for the launchers, and whether the gate has a logit per output channel (heads * vdim columns) instead
     of one per head."""
@@ -1675,12 +1756,13 @@ def _sink_args(r1, r2, sink, gate, heads, vdim):
 def sink_attention_rows(q: torch.Tensor, out: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor, block_tables: torch.Tensor,
                         row_seq: torch.Tensor, positions: torch.Tensor, *, r1: Optional[torch.Tensor], r2: Optional[torch.Tensor],
                         sink: Optional[torch.Tensor], gate: Optional[torch.Tensor], heads: int, kv_heads: int, dim: int, vdim: int,
-                        page_size: int, scale: float, window: Optional[int], status: torch.Tensor) -> None:
+                        page_size: int, scale: float, window: Optional[int], status: torch.Tensor,
+                        softcap: Optional[float] = None, chunk: Optional[int] = None) -> None:
     """out[row, head, :] = sigmoid(gate[row, head]) * sum over the row's visible keys j of w_j v_j, the weights a softmax of
     s_j = q . k_j * scale - r1[head] * ln(1 + r2[head] * distance) whose denominator also holds exp(sink[head]). ``r1``/``r2``,
     ``sink`` (float32 [heads]) and ``gate`` (float32 logits [n, heads], or [n, heads * vdim] for a gate per output channel; rows
-    may be strided) are each optional. One warp per
-    (row, head); any row, both dtypes."""
+    may be strided) are each optional. ``softcap``: q . k * scale passes softcap * tanh(. / softcap) first (the sink does not).
+    ``chunk``: a row sees the keys of its own run of ``chunk`` positions. One warp per (row, head); any row, both dtypes."""
     _cuda(q, out, kcache, vcache, block_tables, row_seq, positions, r1, r2, sink, gate, status)
     n = q.shape[0]
     assert q.shape == (n, heads * dim) and out.shape == (n, heads * vdim) and q.is_contiguous() and out.is_contiguous()
@@ -1688,7 +1770,7 @@ def sink_attention_rows(q: torch.Tensor, out: torch.Tensor, kcache: torch.Tensor
     terms, by_channel = _sink_args(r1, r2, sink, gate, heads, vdim)
     _call("gb_sink_attention_rows", _ptr(q), _ptr(out), _dt(q), _ptr(kcache), _ptr(vcache), _ptr(block_tables), block_tables.shape[1],
           _ptr(row_seq), _ptr(positions), *terms, n, heads, kv_heads, dim, vdim, page_size,
-          kcache.shape[0], float(scale), int(window) if window else 0, by_channel, _ptr(status), _stream())
+          kcache.shape[0], float(scale), float(softcap or 0.0), _mask(window, chunk), by_channel, _ptr(status), _stream())
 
 
 def sink_attention_decode_supported(dtype: torch.dtype, vdim: int) -> bool:
@@ -1698,7 +1780,8 @@ def sink_attention_decode_supported(dtype: torch.dtype, vdim: int) -> bool:
 def sink_attention_decode(q: torch.Tensor, out: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor, block_tables: torch.Tensor,
                           row_seq: torch.Tensor, positions: torch.Tensor, *, r1: Optional[torch.Tensor], r2: Optional[torch.Tensor],
                           sink: Optional[torch.Tensor], gate: Optional[torch.Tensor], heads: int, kv_heads: int, dim: int, vdim: int,
-                          page_size: int, scale: float, window: Optional[int], status: torch.Tensor) -> None:
+                          page_size: int, scale: float, window: Optional[int], status: torch.Tensor,
+                          softcap: Optional[float] = None, chunk: Optional[int] = None) -> None:
     """``sink_attention_rows`` for single decoded tokens: a block of eight warps per (row, head) that share the row's keys,
     each with a running maximum of its own, and meet in a fixed order; a value row must be 64, 128, 256 or 512 bytes
     (``sink_attention_decode_supported``)."""
@@ -1709,7 +1792,7 @@ def sink_attention_decode(q: torch.Tensor, out: torch.Tensor, kcache: torch.Tens
     terms, by_channel = _sink_args(r1, r2, sink, gate, heads, vdim)
     _call("gb_sink_attention_decode", _ptr(q), _ptr(out), _dt(q), _ptr(kcache), _ptr(vcache), _ptr(block_tables),
           block_tables.shape[1], _ptr(row_seq), _ptr(positions), *terms, n, heads, kv_heads, dim, vdim,
-          page_size, kcache.shape[0], float(scale), int(window) if window else 0, by_channel, _ptr(status), _stream())
+          page_size, kcache.shape[0], float(scale), float(softcap or 0.0), _mask(window, chunk), by_channel, _ptr(status), _stream())
 
 
 def sink_attention_tiles_supported(dtype: torch.dtype, dim: int, vdim: int) -> bool:
@@ -1720,7 +1803,8 @@ def sink_attention_tiles(q: torch.Tensor, out: torch.Tensor, kcache: torch.Tenso
                          seq_first_row: torch.Tensor, seq_start_pos: torch.Tensor, max_rows_per_seq: int, *,
                          r1: Optional[torch.Tensor], r2: Optional[torch.Tensor], sink: Optional[torch.Tensor],
                          gate: Optional[torch.Tensor], heads: int, kv_heads: int, dim: int, vdim: int, page_size: int, scale: float,
-                         window: Optional[int], status: torch.Tensor) -> None:
+                         window: Optional[int], status: torch.Tensor, softcap: Optional[float] = None,
+                         chunk: Optional[int] = None) -> None:
     """``sink_attention_rows`` for runs of consecutive rows (prompt portions) in bfloat16 on the tensor cores: a block
     takes 64 rows of one request and one head; ``max_rows_per_seq`` bounds the rows a request brings (it sizes the grid)."""
     _cuda(q, out, kcache, vcache, block_tables, seq_first_row, seq_start_pos, r1, r2, sink, gate, status)
@@ -1732,7 +1816,7 @@ def sink_attention_tiles(q: torch.Tensor, out: torch.Tensor, kcache: torch.Tenso
     _call("gb_sink_attention_tiles", _ptr(q), _ptr(out), _ptr(kcache), _ptr(vcache), _ptr(block_tables), block_tables.shape[1],
           _ptr(seq_first_row), _ptr(seq_start_pos), *terms, seq_start_pos.shape[0],
           max(int(max_rows_per_seq), 1), heads, kv_heads, dim, vdim, page_size, kcache.shape[0], float(scale),
-          int(window) if window else 0, by_channel, _ptr(status), _stream())
+          float(softcap or 0.0), _mask(window, chunk), by_channel, _ptr(status), _stream())
 
 
 # ------------------------------------------------------------------------------------------------ minGRU

@@ -1,2 +1,2 @@
 """Architectures. Importing this package registers them."""
-from . import babotar, felovik, llama, lonorax, tagenex, zurerax  # noqa: F401
+from . import babotar, felovik, llama, lodenex, lonorax, tagenex, zurerax  # noqa: F401

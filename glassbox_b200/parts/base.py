@@ -39,13 +39,15 @@ from ..weights.binding import ParamSpec
 class PagedKvSpec:
     """A mixer that keeps keys and values per token, in pages. Layers with equal specs share a
     cache group (one block table, one page pool). ``window`` None keeps every token; an integer
-    keeps only the last ``window`` tokens, and pages behind the window are given back. ``value_dim`` is the size of the
+    keeps only the last ``window`` tokens, and pages behind the window are given back; ``chunk`` keeps only the tokens of the
+    run of ``chunk`` positions (counted from position 0) that the next token belongs to. ``value_dim`` is the size of the
     second tensor per token and head (None: ``head_dim``; 0: the mixer keeps one tensor per token, the second pool is
     empty)."""
     num_kv_heads: int
     head_dim: int
     window: Optional[int] = None
     value_dim: Optional[int] = None
+    chunk: Optional[int] = None
 
 
 @dataclass(frozen=True)

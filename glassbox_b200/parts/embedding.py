@@ -68,8 +68,17 @@ class ScaledLmHead(LmHead):
             kernels.scale_(logits, self.spec.scale)
 
 
+class CappedLmHead(LmHead):
+    """logits = softcap * tanh((hs H^T) / softcap), from the float32 sums."""
+
+    def forward(self, ctx, hs, logits) -> None:
+        linear(ctx, hs, self.params["weight"], logits)
+        kernels.tanh_cap_(logits, self.spec.softcap)
+
+
 register_part("embedding", "embedding", Embedding, replace=True)
 register_part("embedding", "scaled_embedding", ScaledEmbedding, replace=True)
 register_part("embedding", "positional_embedding", PositionalEmbedding, replace=True)
 register_part("head", "scaled_lm_head", ScaledLmHead, replace=True)
+register_part("head", "capped_lm_head", CappedLmHead, replace=True)
 register_part("head", "lm_head", LmHead, replace=True)

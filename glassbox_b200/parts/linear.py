@@ -126,8 +126,14 @@ def gated_linear(ctx, a, w_gate_up: torch.Tensor, act: torch.Tensor, unit: str =
 
 
 def relu2_linear(ctx, a, w: torch.Tensor, act: torch.Tensor) -> bool:
-    """act = max(a w^T, 0)^2 in one kernel (the activation in the product's epilogue, from the float32 sums) when the
-    operands are bfloat16 and a tensor-core kernel takes them; returns False (and does nothing) otherwise."""
+    """``activated_linear`` with the squared ReLU: act = max(a w^T, 0)^2."""
+    return activated_linear(ctx, a, w, act, "relu2")
+
+
+def activated_linear(ctx, a, w: torch.Tensor, act: torch.Tensor, unit: str) -> bool:
+    """act = f(a w^T) in one kernel (the activation in the product's epilogue, from the float32 sums), f "relu2" or "gelu", when
+    the operands are bfloat16 and a tensor-core kernel takes them; returns False (and does nothing) otherwise."""
+    which = {unit: True}
     if w.dtype != torch.bfloat16 or act.dtype != torch.bfloat16:
         return False
     x, norm, deferred, scale = _resolve(a, w)
@@ -135,12 +141,12 @@ def relu2_linear(ctx, a, w: torch.Tensor, act: torch.Tensor) -> bool:
         x, scale = deferred.tensor(), None
     wide = norm is None and _tile_kernel_wins(x.shape[0], w) and kernels.gemm_tc_supported(x, w, act)
     if not wide and kernels.gemm_stream_supported(x, w) and (norm is not None or x.dtype == torch.bfloat16):
-        kernels.gemm_stream(x, w, act, norm=norm, prefetch=weights_ahead(ctx, w), relu2=True)
+        kernels.gemm_stream(x, w, act, norm=norm, prefetch=weights_ahead(ctx, w), **which)
         return True
     if deferred is not None:
         x = deferred.tensor()
     if x.dtype == torch.bfloat16 and kernels.gemm_tc_supported(x, w, act):
-        kernels.gemm_tc(x, w, act, False, ctx.status, relu2=True)
+        kernels.gemm_tc(x, w, act, False, ctx.status, **which)
         return True
     return False
 

@@ -8,7 +8,7 @@ import torch
 from .. import kernels
 from ..weights.binding import ParamSpec
 from .base import FeedForward, register_part
-from .linear import clamped_glu_linear, gated_linear, linear, relu2_linear
+from .linear import activated_linear, clamped_glu_linear, gated_linear, linear, relu2_linear
 
 
 class SwiGlu(FeedForward):
@@ -86,6 +86,32 @@ class SquaredRelu(FeedForward):
         linear(ctx, act, self.params["w_down"], residual, accumulate=not getattr(ctx, "overwrite_output", False))
 
 
+class GeluMlp(FeedForward):
+    """Dense feed-forward without a gate: residual += gelu(h Wup^T) Wdown^T with the exact GELU, no bias. The activation is formed
+    in float32 from the float32 sums of the first product."""
+    accepts_deferred_input = True
+    launches_through_kernels_only = True
+    can_overwrite_output = True
+
+    def __init__(self, spec, *, hidden_size: int):
+        super().__init__(spec)
+        self.hidden_size = hidden_size
+        self.inter = spec.intermediate_size
+
+    def param_specs(self):
+        d, i = self.hidden_size, self.inter
+        return {"w_up": ParamSpec((i, d)), "w_down": ParamSpec((d, i))}
+
+    def forward(self, ctx, h, residual) -> None:
+        n = h.shape[0]
+        act = ctx.scratch("act", (n, self.inter))
+        if not activated_linear(ctx, h, self.params["w_up"], act, "gelu"):
+            up = ctx.scratch("ffn_up32", (n, self.inter), torch.float32)
+            linear(ctx, h, self.params["w_up"], up)
+            kernels.gelu(up, act)
+        linear(ctx, act, self.params["w_down"], residual, accumulate=not getattr(ctx, "overwrite_output", False))
+
+
 class ClampedGlu(FeedForward):
     """Dense gated feed-forward with clamped branches: g = min(x Wgate^T + b_gate, limit), u = clamp(x Wup^T + b_up, -limit,
     limit), residual += (g * sigmoid(slope * g) * (u + 1)) Wdown^T + b_down. Gate rows then up rows stacked in one matrix
@@ -130,3 +156,4 @@ register_part("ffn", "clamped_glu", ClampedGlu, replace=True)
 register_part("ffn", "swiglu", SwiGlu, replace=True)
 register_part("ffn", "gelu_glu", GeluGlu, replace=True)
 register_part("ffn", "relu2", SquaredRelu, replace=True)
+register_part("ffn", "gelu_mlp", GeluMlp, replace=True)

@@ -13,6 +13,7 @@ import math
 import numpy as np
 import torch
 
+from ..config.specs import RopeBandRescaleSpec
 from .base import Position, register_part
 
 
@@ -21,12 +22,19 @@ def rescaled_frequencies(theta: float, rotary_dim: int, rescale):
     wavelength (``RopeRescaleSpec``): pair i turns f_i = theta^(-2i / rotary_dim) radians per token; with dim(t) = rotary_dim *
     ln(original / (2 pi t)) / (2 ln theta) the pair index that makes t turns within the original context, the pairs below
     lo = max(floor(dim(fast)), 0) keep f_i, those above hi = min(ceil(dim(slow)), rotary_dim - 1) get f_i / factor, the
-    ones between a blend along the ramp clamp((i - lo) / max(hi - lo, 0.001), 0, 1)."""
+    ones between a blend along the ramp clamp((i - lo) / max(hi - lo, 0.001), 0, 1). A ``RopeBandRescaleSpec`` blends along
+    the wavelength itself instead: with t = original f_i / (2 pi) turns within the original context, pairs of more than
+    ``high`` turns keep f_i, those of fewer than ``low`` get f_i / factor, the ones between mix the two in proportion."""
     half = rotary_dim // 2
     i = np.arange(half, dtype=np.float64)
     f = np.power(np.float64(theta), -2.0 * i / np.float64(rotary_dim))
     if rescale is None:
         return f, 1.0
+    if isinstance(rescale, RopeBandRescaleSpec):
+        turns = rescale.original * f / (2.0 * math.pi)
+        span = rescale.high - rescale.low
+        keep = np.clip((turns - rescale.low) / span, 0.0, 1.0) if span else (turns >= rescale.low).astype(np.float64)
+        return (1.0 - keep) * f / rescale.factor + keep * f, 1.0
 
     def pair_of(turns: float) -> float:
         return rotary_dim * math.log(rescale.original / (2.0 * math.pi * turns)) / (2.0 * math.log(theta))
@@ -48,17 +56,16 @@ def rotary_table(theta: float, rotary_dim: int, max_position: int, rescale=None)
     return torch.from_numpy(np.ascontiguousarray(table))
 
 
-def inverse_frequencies(theta: float, rotary_dim: int) -> torch.Tensor:
-    """float32 [rotary_dim/2]: theta^(-2i / rotary_dim), formed in float64 and rounded once."""
-    i = np.arange(rotary_dim // 2, dtype=np.float64)
-    return torch.from_numpy(np.power(np.float64(theta), -2.0 * i / np.float64(rotary_dim)).astype(np.float32))
+def inverse_frequencies(theta: float, rotary_dim: int, rescale=None) -> torch.Tensor:
+    """float32 [rotary_dim/2]: theta^(-2i / rotary_dim), stretched if there is a rescaling, formed in float64 and rounded once."""
+    return torch.from_numpy(rescaled_frequencies(theta, rotary_dim, rescale)[0].astype(np.float32))
 
 
 class Rope(Position):
     """``pairing`` "half": a (cos, sin) table for the kernels that rotate channel i with channel i + rotary_dim/2.
-    ``pairing`` "interleaved" (channel 2i with 2i + 1): no table; the mixers that take it ask for ``inv_freq`` and
-    form the angle float32(position) * inv_freq[i] and its sine and cosine on the device, so no largest position has to
-    be known beforehand."""
+    ``pairing`` "interleaved" (channel 2i with 2i + 1): no table. Mixers that rotate without a table, in either pairing,
+    ask for ``inv_freq`` and ``magnitude`` and form the angle float32(position) * inv_freq[i] and its sine and cosine, times
+    the magnitude, on the device, so no largest position has to be known beforehand."""
     launches_through_kernels_only = True
 
     def __init__(self, spec, **_):
@@ -67,8 +74,8 @@ class Rope(Position):
             raise ValueError(f"rope pairing {spec.pairing!r} is not supported ('half' or 'interleaved')")
         if spec.rotary_dim % 2:
             raise ValueError(f"rotary_dim {spec.rotary_dim} must be even")
-        if getattr(spec, "rescale", None) is not None and spec.pairing != "half":
-            raise ValueError("rescaled frequencies are built into the (cos, sin) table, which only the 'half' pairing uses")
+        self.rescale = getattr(spec, "rescale", None)
+        self.magnitude = float(rescaled_frequencies(spec.theta, spec.rotary_dim, self.rescale)[1])
         self.rotary_dim = spec.rotary_dim
         self.pairing = spec.pairing
         self._tables = {}
@@ -76,7 +83,7 @@ class Rope(Position):
     def inv_freq(self, device):
         key = ("inv_freq", str(device))
         if key not in self._tables:
-            self._tables[key] = inverse_frequencies(self.spec.theta, self.spec.rotary_dim).to(device)
+            self._tables[key] = inverse_frequencies(self.spec.theta, self.spec.rotary_dim, self.rescale).to(device)
         return self._tables[key]
 
     def fused_table(self, device):
@@ -85,7 +92,7 @@ class Rope(Position):
         key = str(device)
         if key not in self._tables:
             self._tables[key] = rotary_table(self.spec.theta, self.spec.rotary_dim, self.spec.max_position,
-                                             getattr(self.spec, "rescale", None)).to(device)
+                                             self.rescale).to(device)
         return self._tables[key]
 
 
