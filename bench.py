@@ -637,6 +637,53 @@ def felovik_workload(args):
     return out
 
 
+# ------------------------------------------------------------------------------------------------ Lodenex beside its neighbours
+#: layer sizes that resemble real models' (random weights): a Lodenex model whose layers are in turn attention within chunks of
+#: 1,024 positions and latent attention within a window of 1,024, all with a dense GELU feed-forward. Beside it Zurerax (the
+#: framework's other model of latent attention, whose feed-forwards are as large), Tagenex (its other model of attention with a
+#: sink and a gate per head) and the Llama decoder, all of the same width, depth and feed-forward width.
+LODENEX_SIZES = {
+    "w1024": dict(attn=dict(heads=16, kv_heads=4, dim=64, vdim=64), latent=dict(heads=16, dim=64, rot_dim=32, vdim=64, kv_rank=128, q_rank=512),
+                  chunk=1024, window=1024),
+    "w2048": dict(attn=dict(heads=32, kv_heads=8, dim=64, vdim=64), latent=dict(heads=32, dim=64, rot_dim=64, vdim=64, kv_rank=128, q_rank=768),
+                  chunk=1024, window=1024),
+}
+
+
+def lodenex_raw(size: dict, own: dict) -> dict:
+    from glassbox_b200.models.lodenex import make_lodenex_raw_config
+    layers = []
+    for i in range(size["layers"]):
+        mlp = {"kind": "dense", "ff": size["ff"]}
+        if i % 2:
+            m = dict(own["latent"])
+            m.update(scale=(m["dim"] + m["rot_dim"]) ** -0.5, mask={"size": own["window"]},
+                     rot={"base": 10000.0, "dims": m["rot_dim"], "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}})
+            layers.append({"type": "latent_attention", "mixer": m, "mlp": mlp})
+        else:
+            m = dict(own["attn"])
+            m.update(scale=m["dim"] ** -0.5, softcap=30.0, mask={"size": own["chunk"]},
+                     rot={"base": 10000.0, "dims": m["dim"], "scaling": {"factor": 8.0, "original": 4096, "low": 1.0, "high": 4.0}})
+            layers.append({"type": "attention", "mixer": m, "mlp": mlp})
+    return make_lodenex_raw_config(vocab=size["vocab"], width=size["width"], layers=layers)
+
+
+def lodenex_workload(args):
+    """Prefill and decode throughput of Lodenex models beside Zurerax, Tagenex and the Llama decoder of equal width, depth and
+    feed-forward width; one JSON line. Decode steps end at the context length; three timed regions per point."""
+    T, ctx, K, W = 2048, args.context, min(args.steps, 128), max(args.warmup, 3)
+    out = {"workload": "lodenex", "dtype": args.dtype, "context": ctx, "prefill_tokens": T, "decode_steps": K, "sizes": {}}
+    for name, size in ZURERAX_SIZES.items():
+        llama = dict(num_hidden_layers=size["layers"], hidden_size=size["width"], intermediate_size=size["ff"],
+                     vocab_size=size["vocab"], rope_theta=10000.0, rms_norm_eps=1e-5, tie_word_embeddings=False,
+                     max_position_embeddings=8192, **size["llama"])
+        arms = (("lodenex", dict(raw=lodenex_raw(size, LODENEX_SIZES[name]))), ("zurerax", dict(raw=zurerax_raw(size))),
+                ("tagenex", dict(raw=tagenex_raw(size, TAGENEX_SIZES[name]))), ("llama", dict(shape=llama)))
+        out["sizes"][name] = {label: measure_arm(f"{label}-{name}", args, T, ctx, K, W, **kw) for label, kw in arms
+                              if not args.only or label in args.only.split(",")}
+    return out
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -651,15 +698,16 @@ def main():
     ap.add_argument("--no-points", action="store_true", help="only the headline region: no other batches, prefill or e2e")
     ap.add_argument("--no-others", action="store_true",
                     help="skip the other model sizes, the serving workload, the 32-bit path and the CPU baseline")
-    ap.add_argument("--workload", default="decode", choices=["decode", "serving", "zurerax", "lonorax", "tagenex", "babotar", "felovik"],
+    ap.add_argument("--workload", default="decode", choices=["decode", "serving", "zurerax", "lonorax", "tagenex", "babotar", "felovik", "lodenex"],
                     help="serving: the mixed workload of the 360M configuration (64 requests, prompts 32-2048, outputs "
                          "32-512, prompt portions of 512, a quarter of the requests sharing a 384-token prefix) through "
                          "the scheduler; prints its own JSON line. zurerax: prefill and decode throughput of Zurerax models "
                          "at two widths beside the Llama decoder of equal size; prints its own JSON line. lonorax: the same for "
                          "Lonorax models beside Zurerax and Llama of equal size; tagenex: the same for Tagenex models beside Llama "
                          "and Lonorax of equal size; babotar: the same for Babotar models beside Zurerax and Llama of equal size; "
-                         "felovik: the same for Felovik models beside Babotar, Tagenex and Llama of equal size")
-    ap.add_argument("--only", default="", help="with --workload lonorax, tagenex, babotar or felovik: the arms to run (felovik,babotar,tagenex,lonorax,zurerax,llama), with commas")
+                         "felovik: the same for Felovik models beside Babotar, Tagenex and Llama of equal size; "
+                         "lodenex: the same for Lodenex models beside Zurerax, Tagenex and Llama of equal size")
+    ap.add_argument("--only", default="", help="with --workload lonorax, tagenex, babotar, felovik or lodenex: the arms to run (lodenex,felovik,babotar,tagenex,lonorax,zurerax,llama), with commas")
     args = ap.parse_args()
 
     if args.impl == "reference":
@@ -689,6 +737,9 @@ def main():
         return 0
     if args.workload == "felovik":
         print(json.dumps(felovik_workload(args)))
+        return 0
+    if args.workload == "lodenex":
+        print(json.dumps(lodenex_workload(args)))
         return 0
     K, W, B, CTX = args.steps, max(args.warmup, 3), args.batch, args.context
     pk = peaks()

@@ -367,11 +367,25 @@ __global__ void __launch_bounds__(AT_WARPS * 32) attention_prefill_tc_kernel(
             if (lane == 0) mbar_arrive(&sh.s_free[g]);   // the buffer may take the group's next S
             if constexpr (SINK) {
                 if (cap2 > 0.f) {
-                    // cap tanh(s / cap) = cap - 2 cap / (1 + exp(2 s / cap))
+                    // cap tanh(s / cap) = cap - 2 cap / (1 + exp(2 s / cap)). Four scores share one reciprocal, of the product of
+                    // their denominators (each at most 1 + 2^30, where the tanh is 1 to the last bit): the exponentials and
+                    // reciprocals go through the pipe that bounds this kernel.
+                    const float2 in2 = make_float2(cap_in, cap_in), one2 = make_float2(1.f, 1.f);
+                    const float2 top2 = make_float2(cap2, cap2), down2 = make_float2(-2.0f * cap2, -2.0f * cap2);
 #pragma unroll
-                    for (int k = 0; k < AT_BN; ++k) {
-                        const float e = at_exp2(__uint_as_float(sv[k]) * cap_in);
-                        sv[k] = __float_as_uint(fmaf(-2.0f * cap2, at_rcp(1.0f + e), cap2));
+                    for (int k = 0; k < AT_BN; k += 4) {
+                        const float2 ya = __fmul2_rn(make_float2(__uint_as_float(sv[k]), __uint_as_float(sv[k + 1])), in2);
+                        const float2 yb = __fmul2_rn(make_float2(__uint_as_float(sv[k + 2]), __uint_as_float(sv[k + 3])), in2);
+                        const float2 ea = __fadd2_rn(make_float2(at_exp2(fminf(ya.x, 30.f)), at_exp2(fminf(ya.y, 30.f))), one2);
+                        const float2 eb = __fadd2_rn(make_float2(at_exp2(fminf(yb.x, 30.f)), at_exp2(fminf(yb.y, 30.f))), one2);
+                        const float2 both = __fmul2_rn(ea, eb);                             // (a0 b0, a1 b1)
+                        const float r = at_rcp(both.x * both.y);
+                        const float2 rb = __fmul2_rn(make_float2(both.y, both.x), make_float2(r, r));      // (1 / a0 b0, 1 / a1 b1)
+                        const float2 sa = __ffma2_rn(__fmul2_rn(eb, rb), down2, top2), sb = __ffma2_rn(__fmul2_rn(ea, rb), down2, top2);
+                        sv[k] = __float_as_uint(sa.x);
+                        sv[k + 1] = __float_as_uint(sa.y);
+                        sv[k + 2] = __float_as_uint(sb.x);
+                        sv[k + 3] = __float_as_uint(sb.y);
                     }
                 }
                 const float sl = cap2 > 0.f ? 1.0f : sl2;      // what is left to scale

@@ -63,10 +63,37 @@ __device__ __forceinline__ float gb_gelu_tanh_fast(float z) {
 // GELU itself: z times the cumulative normal distribution, z / 2 (1 + erf(z / sqrt 2)).
 __device__ __forceinline__ float gb_gelu(float z) { return 0.5f * z * (1.0f + erff(z * 0.7071067811865476f)); }
 
+// The same with erf from the rational approximation 7.1.26 of Abramowitz and Stegun's handbook (an error of 1.5e-7) and the
+// hardware's exponential and division: for epilogues that round the result to bfloat16.
+__device__ __forceinline__ float gb_gelu_fast(float z) {
+    const float x = fabsf(z) * 0.7071067811865476f;
+    const float t = __fdividef(1.0f, fmaf(0.3275911f, x, 1.0f));
+    float p = fmaf(1.061405429f, t, -1.453152027f);
+    p = fmaf(p, t, 1.421413741f);
+    p = fmaf(p, t, -0.284496736f);
+    p = fmaf(p, t, 0.254829592f);
+    const float tail = p * t * __expf(-x * x);           // 1 - erf(x), x >= 0
+    return 0.5f * z * (z < 0.f ? tail : 2.0f - tail);
+}
+
 // cap * tanh(s / cap) through tanh(y) = 1 - 2 / (1 + exp(2 y)) with the hardware's exponential and division: an absolute
 // error of a few 1e-7 * cap, for scores on their way into an exponential. inv2 = 2 / cap.
 __device__ __forceinline__ float gb_cap_fast(float s, float cap, float inv2) {
     return fmaf(-2.0f * cap, __fdividef(1.0f, 1.0f + __expf(s * inv2)), cap);
+}
+
+// The same for four scores in place, which share one division: by the product of their denominators, each kept at or below
+// 1 + e^20 (where the tanh is 1 to the last bit).
+__device__ __forceinline__ void gb_cap_fast4(float (&s)[4], float cap, float inv2) {
+    float e[4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i) e[i] = 1.0f + __expf(fminf(s[i] * inv2, 20.0f));
+    const float a = e[0] * e[1], b = e[2] * e[3], r = __fdividef(1.0f, a * b), ra = r * b, rb = r * a;
+    const float down = -2.0f * cap;
+    s[0] = fmaf(down, e[1] * ra, cap);
+    s[1] = fmaf(down, e[0] * ra, cap);
+    s[2] = fmaf(down, e[3] * rb, cap);
+    s[3] = fmaf(down, e[2] * rb, cap);
 }
 
 // The first key that a query at position `pos` sees. mask > 0: a sliding window of that many keys; mask < 0: chunks of -mask

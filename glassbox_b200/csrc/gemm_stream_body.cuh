@@ -473,7 +473,7 @@ __device__ __forceinline__ void gemm_stream_body(const StreamArgs& a, const int 
             const float g = fmaxf(v[0], 0.f);
             reinterpret_cast<__nv_bfloat16*>(a.C)[(size_t)tok * a.ldc + n] = __float2bfloat16_rn(g * g);
         } else if (a.mode == WS_GELU_BF16) {        // gelu, from the float32 sum
-            reinterpret_cast<__nv_bfloat16*>(a.C)[(size_t)tok * a.ldc + n] = __float2bfloat16_rn(gb_gelu(v[0]));
+            reinterpret_cast<__nv_bfloat16*>(a.C)[(size_t)tok * a.ldc + n] = __float2bfloat16_rn(gb_gelu_fast(v[0]));
         } else if (a.mode == WS_STORE_F32) {
             reinterpret_cast<float*>(a.C)[(size_t)tok * a.ldc + n] = v[0];
         } else {

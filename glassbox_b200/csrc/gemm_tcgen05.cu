@@ -374,7 +374,7 @@ __global__ void __launch_bounds__(192) gemm_tcgen05_kernel(const __grid_constant
                 }
                 if (!GATED && mode == TC_GELU_BF16) {      // gelu, from the float32 sums
 #pragma unroll
-                    for (int j = 0; j < 32; ++j) r[j] = __float_as_uint(gb_gelu(__uint_as_float(r[j])));
+                    for (int j = 0; j < 32; ++j) r[j] = __float_as_uint(gb_gelu_fast(__uint_as_float(r[j])));
                 }
                 if (GATED || mode == TC_STORE_BF16 || mode == TC_RELU2_BF16 || mode == TC_GELU_BF16) {
                     // a thread's 32 columns are 64 contiguous bytes: store them directly, 16 bytes at a time

@@ -4,7 +4,7 @@
 // This is the shape of the up-projections of latent attention once they are moved to the query and to the weighted sum
 // of latents: K and N are a head's sizes (tens to a few hundred), so a head's product is far too small for a launch of
 // its own. Optionally every output is multiplied by sigmoid(gate[row, h, column]), a logit per output (float32 or bfloat16).
-// One block = 64 rows x one head x up to 128 output columns; a and w[h] are staged once in shared memory
+// One block = 64 rows x one head x up to 128 output columns (64 for narrow heads); a and w[h] are staged once in shared memory
 // (rows padded by 16 bytes so that ldmatrix meets no bank twice), each of the four warps takes 16 rows.
 #include "common.cuh"
 
@@ -23,17 +23,28 @@ __device__ __forceinline__ void hl_ldmatrix_x4(uint32_t (&r)[4], uint32_t addr) 
                  : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
 }
 
+enum { HL_GATE_BF16 = 0, HL_GATE_F32 = 1, HL_GATE_F32_PAIRS = 2 };     // PAIRS: two neighbours can be loaded as one
+
+__device__ __forceinline__ float2 hl_pair(const void* gate, int kind, size_t at) {
+    if (kind == HL_GATE_F32_PAIRS) return *reinterpret_cast<const float2*>(reinterpret_cast<const float*>(gate) + at);
+    if (kind == HL_GATE_F32) return make_float2(reinterpret_cast<const float*>(gate)[at], reinterpret_cast<const float*>(gate)[at + 1]);
+    const __nv_bfloat16* b = reinterpret_cast<const __nv_bfloat16*>(gate) + at;
+    return make_float2(__bfloat162float(b[0]), __bfloat162float(b[1]));
+}
+__device__ __forceinline__ float hl_open(float v, float z) { return __fdividef(v, 1.0f + __expf(-z)); }      // v times sigmoid(z)
+
+template <int BN, bool GATED>
 __global__ void __launch_bounds__(128) head_linear_kernel(const __nv_bfloat16* __restrict__ a, long long lda, long long a_head,
                                                           const __nv_bfloat16* __restrict__ w, __nv_bfloat16* __restrict__ out,
                                                           long long ldc, long long c_head, int n, int N, int K,
-                                                          const void* __restrict__ gate, long long ld_gate, int gate_f32) {
+                                                          const void* __restrict__ gate, long long ld_gate, int gate_kind) {
     extern __shared__ __align__(128) unsigned char hl_smem[];
     gb_pdl_launch_dependents();
     const int KS = K + 8;                                    // padded row, elements
     __nv_bfloat16* As = reinterpret_cast<__nv_bfloat16*>(hl_smem);     // [64][KS]
-    __nv_bfloat16* Ws = As + HL_BM * KS;                               // [128][KS]
-    const int head = blockIdx.y, m0 = blockIdx.x * HL_BM, n0 = blockIdx.z * HL_BN;
-    const int cols = min(HL_BN, N - n0);
+    __nv_bfloat16* Ws = As + HL_BM * KS;                               // [BN][KS]
+    const int head = blockIdx.y, m0 = blockIdx.x * HL_BM, n0 = blockIdx.z * BN;
+    const int cols = min(BN, N - n0);
     const int cpr = K / 8;                                   // 16-byte chunks per row
     const __nv_bfloat16* wh = w + ((size_t)head * N + n0) * K;
     for (int c = threadIdx.x; c < cols * cpr; c += 128) {    // the weights do not depend on the kernel before: ask first
@@ -49,28 +60,42 @@ __global__ void __launch_bounds__(128) head_linear_kernel(const __nv_bfloat16* _
         if (m0 + r < n) __pipeline_memcpy_async(d, ah + (size_t)(m0 + r) * lda + ch * 8, 16);
         else *reinterpret_cast<uint4*>(d) = make_uint4(0u, 0u, 0u, 0u);
     }
-    for (int c = threadIdx.x + cols * cpr; c < HL_BN * cpr; c += 128) {      // rows of the weight tile beyond N: zeros
+    for (int c = threadIdx.x + cols * cpr; c < BN * cpr; c += 128) {      // rows of the weight tile beyond N: zeros
         const int r = c / cpr, ch = c % cpr;
         *reinterpret_cast<uint4*>(Ws + r * KS + ch * 8) = make_uint4(0u, 0u, 0u, 0u);
     }
     __pipeline_commit();
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const int g = lane >> 2, t = lane & 3, m = lane >> 3, r8 = lane & 7;
+    const int row_a = m0 + warp * 16 + g, row_b = row_a + 8;
+    // the logits of this thread's outputs, asked for before the product starts
+    float2 gate_a[GATED ? BN / 8 : 1], gate_b[GATED ? BN / 8 : 1];
+    if constexpr (GATED) {
+        const size_t at = (size_t)head * N + n0 + 2 * t;
+#pragma unroll
+        for (int nt = 0; nt < BN / 8; ++nt) {
+            gate_a[nt] = gate_b[nt] = make_float2(0.f, 0.f);
+            if (nt * 8 + 2 * t < cols) {
+                if (row_a < n) gate_a[nt] = hl_pair(gate, gate_kind, (size_t)row_a * ld_gate + at + nt * 8);
+                if (row_b < n) gate_b[nt] = hl_pair(gate, gate_kind, (size_t)row_b * ld_gate + at + nt * 8);
+            }
+        }
+    }
     __pipeline_wait_prior(0);
     __syncthreads();
 
-    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    const int g = lane >> 2, t = lane & 3, m = lane >> 3, r8 = lane & 7;
     const uint32_t a_base = (uint32_t)__cvta_generic_to_shared(As + (size_t)warp * 16 * KS);
     const uint32_t w_base = (uint32_t)__cvta_generic_to_shared(Ws);
-    float acc[HL_BN / 8][4];
+    float acc[BN / 8][4];
 #pragma unroll
-    for (int i = 0; i < HL_BN / 8; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
+    for (int i = 0; i < BN / 8; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
     const int n_pairs = (cols + 15) / 16;
     for (int ks = 0; ks < K / 16; ++ks) {
         uint32_t af[4];
         // A fragment: matrices (rows 0-7, k 0-7), (rows 8-15, k 0-7), (rows 0-7, k 8-15), (rows 8-15, k 8-15)
         hl_ldmatrix_x4(af, a_base + (uint32_t)((((m & 1) * 8 + r8) * KS + ks * 16 + (m >> 1) * 8) * 2));
 #pragma unroll
-        for (int np = 0; np < HL_BN / 16; ++np) {
+        for (int np = 0; np < BN / 16; ++np) {
             if (np < n_pairs) {
                 uint32_t b[4];
                 hl_ldmatrix_x4(b, w_base + (uint32_t)(((np * 16 + (m >> 1) * 8 + r8) * KS + ks * 16 + (m & 1) * 8) * 2));
@@ -79,24 +104,23 @@ __global__ void __launch_bounds__(128) head_linear_kernel(const __nv_bfloat16* _
             }
         }
     }
-    const int row_a = m0 + warp * 16 + g, row_b = row_a + 8;
     __nv_bfloat16* oh = out + (size_t)head * c_head + n0;
-    auto opened = [&](int row, int col, float v) {       // v behind its gate
-        if (gate == nullptr) return v;
-        const size_t at = (size_t)row * ld_gate + (size_t)head * N + n0 + col;
-        const float z = gate_f32 ? reinterpret_cast<const float*>(gate)[at] : __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(gate)[at]);
-        return __fdividef(v, 1.0f + __expf(-z));
-    };
 #pragma unroll
-    for (int nt = 0; nt < HL_BN / 8; ++nt) {
+    for (int nt = 0; nt < BN / 8; ++nt) {
         const int col = nt * 8 + 2 * t;
+        if constexpr (GATED) {
+            acc[nt][0] = hl_open(acc[nt][0], gate_a[nt].x);
+            acc[nt][1] = hl_open(acc[nt][1], gate_a[nt].y);
+            acc[nt][2] = hl_open(acc[nt][2], gate_b[nt].x);
+            acc[nt][3] = hl_open(acc[nt][3], gate_b[nt].y);
+        }
         if (col < cols) {      // (N is even: a pair never straddles the edge)
             if (row_a < n) {
-                __nv_bfloat162 v = __floats2bfloat162_rn(opened(row_a, col, acc[nt][0]), opened(row_a, col + 1, acc[nt][1]));
+                __nv_bfloat162 v = __floats2bfloat162_rn(acc[nt][0], acc[nt][1]);
                 *reinterpret_cast<__nv_bfloat162*>(oh + (size_t)row_a * ldc + col) = v;
             }
             if (row_b < n) {
-                __nv_bfloat162 v = __floats2bfloat162_rn(opened(row_b, col, acc[nt][2]), opened(row_b, col + 1, acc[nt][3]));
+                __nv_bfloat162 v = __floats2bfloat162_rn(acc[nt][2], acc[nt][3]);
                 *reinterpret_cast<__nv_bfloat162*>(oh + (size_t)row_b * ldc + col) = v;
             }
         }
@@ -117,15 +141,23 @@ GB_EXPORT int gb_head_linear(const void* a, long long lda, long long a_head, con
                "gb_head_linear: K=%d must be a multiple of 16 up to %d, N=%d even, operands aligned", K, HL_MAX_K, N);
     GB_REQUIRE(n >= 0 && heads > 0 && heads <= 65535, "gb_head_linear: bad sizes");
     if (n == 0) return 0;
-    const size_t smem = (size_t)(HL_BM + HL_BN) * (K + 8) * sizeof(__nv_bfloat16);
-    static size_t allowed = 48 * 1024;
-    if (smem > allowed) {
-        cudaFuncSetAttribute(head_linear_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-        allowed = smem;
+    const int kind = !gate_f32 ? HL_GATE_BF16 : (N % 2 == 0 && ld_gate % 2 == 0 && (uintptr_t)gate % 8 == 0) ? HL_GATE_F32_PAIRS : HL_GATE_F32;
+    // narrow heads take the narrow tile: half the registers and less shared memory, so more blocks at once
+    const bool narrow = N <= HL_BN / 2;
+    const int bn = narrow ? HL_BN / 2 : HL_BN;
+    const size_t smem = (size_t)(HL_BM + bn) * (K + 8) * sizeof(__nv_bfloat16);
+    void (*kernel)(const __nv_bfloat16*, long long, long long, const __nv_bfloat16*, __nv_bfloat16*, long long, long long, int, int, int, const void*,
+                   long long, int) = narrow ? (gate ? head_linear_kernel<HL_BN / 2, true> : head_linear_kernel<HL_BN / 2, false>)
+                                            : (gate ? head_linear_kernel<HL_BN, true> : head_linear_kernel<HL_BN, false>);
+    static size_t allowed[4] = {48 * 1024, 48 * 1024, 48 * 1024, 48 * 1024};
+    size_t& have = allowed[(narrow ? 2 : 0) + (gate ? 1 : 0)];
+    if (smem > have) {
+        cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        have = smem;
     }
-    dim3 grid(gb_ceil_div(n, HL_BM), heads, gb_ceil_div(N, HL_BN));
-    cudaError_t e = gb_launch(GB_PDL_GEMM, head_linear_kernel, grid, dim3(128), smem, stream, (const __nv_bfloat16*)a, lda, a_head,
-                              (const __nv_bfloat16*)w, (__nv_bfloat16*)out, ldc, c_head, n, N, K, gate, ld_gate, gate_f32);
+    dim3 grid(gb_ceil_div(n, HL_BM), heads, gb_ceil_div(N, bn));
+    cudaError_t e = gb_launch(GB_PDL_GEMM, kernel, grid, dim3(128), smem, stream, (const __nv_bfloat16*)a, lda, a_head, (const __nv_bfloat16*)w,
+                              (__nv_bfloat16*)out, ldc, c_head, n, N, K, gate, ld_gate, kind);
     if (e != cudaSuccess) {
         gb_set_error("gb_head_linear: launch failed: %s", cudaGetErrorString(e));
         return 2;

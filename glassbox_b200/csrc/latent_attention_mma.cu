@@ -19,6 +19,7 @@
 #include <cuda_pipeline.h>
 
 constexpr int LM_BN = 64;                 // keys per staged tile
+constexpr int LM_STAGES = 2;              // staged tiles (a third one in decoding, two tiles' loads in flight, was no faster)
 constexpr float LM_NEG_BIG = -1.0e30f;
 constexpr float LM_LOG2E = 1.4426950408889634f;
 
@@ -66,8 +67,9 @@ __global__ void __launch_bounds__(128) latent_attention_mma_kernel(LatentMmaArgs
     constexpr int KS = W / 16, CT = C / 8, CPR = W / 8;   // k16 steps of the scores, n8 tiles of the output, 16-byte chunks per row
     constexpr int NK = KEYS_OVER_WARPS ? LM_BN / 4 : LM_BN;   // keys of a staged tile that one warp takes
     constexpr int NT = NK / 8;
+    constexpr int ST = LM_STAGES;
     extern __shared__ __align__(128) unsigned char lm_smem[];
-    __nv_bfloat16* Ks = reinterpret_cast<__nv_bfloat16*>(lm_smem);   // [2][LM_BN][WS]
+    __nv_bfloat16* Ks = reinterpret_cast<__nv_bfloat16*>(lm_smem);   // [ST][LM_BN][WS]
     gb_pdl_launch_dependents();
     gb_pdl_wait();
 
@@ -136,27 +138,29 @@ __global__ void __launch_bounds__(128) latent_attention_mma_kernel(LatentMmaArgs
         }
     }
 
-    // Two threads per key of the tile: one page look-up and one address per thread, then half a row of 16-byte pieces.
-    static_assert(CPR % 2 == 0, "a cached row is an even number of 16-byte pieces");
-    auto load_tile = [&](int kt, int buf) {
-        const int kk = threadIdx.x >> 1, half = threadIdx.x & 1;
-        const int key = kt * LM_BN + kk;
-        long long page = -1;
-        if (key <= pos_hi) {
-            page = table[key >> p.page_shift];
-            if (page < 0 || page >= p.num_pages) {
-                if (key >= key_lo) atomicOr(p.status, GB_STATUS_BAD_SLOT);   // (pages behind a window may be gone)
-                page = -1;
-            }
+    // Where the keys of a tile lie is looked up a tile ahead of its loads, one key per thread, and kept in shared memory; the
+    // loads then go piece by piece along the rows, so that neighbouring lanes fetch neighbouring 16-byte pieces (a lane that
+    // walked a row of its own would touch a cache line per lane and instruction).
+    __shared__ long long tile_rows[ST][LM_BN];          // cache row of each key, -1: zeros
+    auto find_row = [&](int kt) -> long long {          // (threads 0 .. LM_BN - 1)
+        const int key = kt * LM_BN + (int)threadIdx.x;
+        if (key > pos_hi) return -1;
+        const long long page = table[key >> p.page_shift];
+        if (page < 0 || page >= p.num_pages) {
+            if (key >= key_lo) atomicOr(p.status, GB_STATUS_BAD_SLOT);   // (pages behind a window may be gone)
+            return -1;
         }
-        __nv_bfloat16* d = Ks + (size_t)buf * LM_BN * WS + kk * WS + half * (CPR / 2) * 8;
-        if (page >= 0) {
-            const __nv_bfloat16* src = p.cache + ((size_t)page * page_size + (key & (page_size - 1))) * W + half * (CPR / 2) * 8;
+        return page * page_size + (key & (page_size - 1));
+    };
+    static_assert(LM_BN * CPR % 128 == 0, "every thread loads as many pieces");
+    auto load_tile = [&](int buf) {
+        __nv_bfloat16* d = Ks + (size_t)buf * LM_BN * WS;
 #pragma unroll
-            for (int j = 0; j < CPR / 2; ++j) __pipeline_memcpy_async(d + j * 8, src + j * 8, 16);
-        } else {
-#pragma unroll
-            for (int j = 0; j < CPR / 2; ++j) *reinterpret_cast<uint4*>(d + j * 8) = make_uint4(0u, 0u, 0u, 0u);
+        for (int i = 0; i < LM_BN * CPR / 128; ++i) {
+            const int idx = i * 128 + (int)threadIdx.x, kk = idx / CPR, ch = idx - kk * CPR;
+            const long long row = tile_rows[buf][kk];
+            if (row >= 0) __pipeline_memcpy_async(d + kk * WS + ch * 8, p.cache + row * W + ch * 8, 16);
+            else *reinterpret_cast<uint4*>(d + kk * WS + ch * 8) = make_uint4(0u, 0u, 0u, 0u);
         }
         __pipeline_commit();
     };
@@ -166,16 +170,26 @@ __global__ void __launch_bounds__(128) latent_attention_mma_kernel(LatentMmaArgs
     for (int i = 0; i < CT; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
     float m_a = LM_NEG_BIG, m_b = LM_NEG_BIG, l_a = 0.f, l_b = 0.f;
 
-    if (kt_begin < kt_end) load_tile(kt_begin, 0);
-    for (int kt = kt_begin; kt < kt_end; ++kt) {
-        const int buf = (kt - kt_begin) & 1;
-        if (kt + 1 < kt_end) {
-            load_tile(kt + 1, buf ^ 1);
-            __pipeline_wait_prior(1);
-        } else {
-            __pipeline_wait_prior(0);
-        }
+    const bool finds = threadIdx.x < LM_BN;
+    if (finds) {
+#pragma unroll
+        for (int j = 0; j < ST; ++j) tile_rows[j][threadIdx.x] = kt_begin + j < kt_end ? find_row(kt_begin + j) : -1;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int j = 0; j < ST - 1; ++j) {
+        if (kt_begin + j < kt_end) load_tile(j);
+        else __pipeline_commit();
+    }
+    int buf = 0, ahead = ST - 1;                         // the buffers of this tile and of the one loaded meanwhile
+    for (int kt = kt_begin; kt < kt_end; ++kt, buf = buf + 1 == ST ? 0 : buf + 1, ahead = ahead + 1 == ST ? 0 : ahead + 1) {
+        long long later = -1;
+        if (finds && kt + ST < kt_end) later = find_row(kt + ST);
+        if (kt + ST - 1 < kt_end) load_tile(ahead);
+        else __pipeline_commit();
+        __pipeline_wait_prior(ST - 1);
         __syncthreads();
+        if (finds) tile_rows[buf][threadIdx.x] = later;      // (read after the barrier at the end of this round)
         const int key0 = kt * LM_BN + (KEYS_OVER_WARPS ? warp * NK : 0);      // this warp's first key of the tile
         if (key0 <= warp_pos_hi) {
             const uint32_t tile = (uint32_t)__cvta_generic_to_shared(Ks + (size_t)buf * LM_BN * WS + (size_t)(key0 - kt * LM_BN) * WS);
@@ -393,7 +407,7 @@ GB_EXPORT int gb_latent_attention_mma_supported(int c, int r, int page_size) {
 template <int C, int R>
 static int launch_latent_mma(const LatentMmaArgs& p, bool decode, int n_or_groups, int head_groups, int S, cudaStream_t stream) {
     constexpr int W = C + R;
-    const size_t stage = (size_t)2 * LM_BN * (W + 8) * sizeof(__nv_bfloat16);
+    const size_t stage = (size_t)LM_STAGES * LM_BN * (W + 8) * sizeof(__nv_bfloat16);
     const size_t merge = (size_t)(4 * 16 * C + 4 * 16 * 2) * sizeof(float);
     const size_t smem = decode && merge > stage ? merge : stage;
     cudaError_t e;

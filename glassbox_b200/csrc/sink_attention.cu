@@ -338,8 +338,9 @@ GB_EXPORT int gb_sink_attention_decode(const void* q, void* out, int dtype, cons
 constexpr int SKT_BM = 64, SKT_BN = 64;
 constexpr float SK_LOG2E = 1.4426950408889634f;
 
-template <int D, int V>
-__global__ void __launch_bounds__(128) sink_attention_tiles_kernel(
+// (three blocks on a multiprocessor where their shared memory allows it: the registers must then fit as well)
+template <int D, int V, bool CAP>
+__global__ void __launch_bounds__(128, D + V <= 192 ? 3 : 2) sink_attention_tiles_kernel(
     const __nv_bfloat16* __restrict__ q, __nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict__ kcache,
     const __nv_bfloat16* __restrict__ vcache, const int* __restrict__ block_tables, int max_pages, const int* __restrict__ seq_first_row,
     const int* __restrict__ seq_start_pos, const float* __restrict__ r1, const float* __restrict__ r2, const float* __restrict__ sink,
@@ -374,26 +375,40 @@ __global__ void __launch_bounds__(128) sink_attention_tiles_kernel(
         const int r = chunk / (D / 8), c = (chunk % (D / 8)) * 8;
         sat_cp16(sq + r * LDK + c, q + ((size_t)(row0 + (r < rows ? r : 0)) * H + head) * D + c, r < rows);
     }
-    auto stage = [&](int buf, int kb) {
-        // two threads per key: one page look-up each, then half of the key's 16-byte pieces (key row, then value row)
-        constexpr int CPK = (D + V) / 8;
-        const int key = tid >> 1, kk = kb + key;
-        long long page = kk <= p_hi ? table[kk / page_size] : -1;
-        if (kk <= p_hi && (page < 0 || page >= num_pages)) {
+    // Where the keys of a tile lie is looked up a tile ahead of its loads, one key per thread, and kept in shared memory; the
+    // loads then go piece by piece along the rows (the key row, then the value row), so that neighbouring lanes fetch
+    // neighbouring 16-byte pieces.
+    __shared__ long long tile_rows[2][SKT_BN];        // cache row of each key, -1: zeros
+    auto find_row = [&](int kb) -> long long {        // (threads 0 .. SKT_BN - 1)
+        const int kk = kb + tid;
+        if (kk > p_hi) return -1;
+        const long long page = table[kk / page_size];
+        if (page < 0 || page >= num_pages) {
             atomicOr(status, GB_STATUS_BAD_SLOT);
-            page = -1;
+            return -1;
         }
-        const long long at = page < 0 ? 0 : (page * G + g) * page_size + kk % page_size;
+        return (page * G + g) * page_size + kk % page_size;
+    };
+    auto stage = [&](int buf) {
+        constexpr int CPK = (D + V) / 8;
+        static_assert(SKT_BN * CPK % 128 == 0, "every thread loads as many pieces");
 #pragma unroll
-        for (int i = 0; i < CPK / 2; ++i) {
-            const int c = ((tid & 1) * (CPK / 2) + i) * 8;
-            if (c < D) sat_cp16(sk + (buf * SKT_BN + key) * LDK + c, kcache + at * D + c, page >= 0);
-            else sat_cp16(sv + (buf * SKT_BN + key) * LDV + (c - D), vcache + at * V + (c - D), page >= 0);
+        for (int i = 0; i < SKT_BN * CPK / 128; ++i) {
+            const int idx = i * 128 + tid, key = idx / CPK, c = (idx - key * CPK) * 8;
+            const long long row = tile_rows[buf][key], at = row < 0 ? 0 : row;
+            if (c < D) sat_cp16(sk + (buf * SKT_BN + key) * LDK + c, kcache + at * D + c, row >= 0);
+            else sat_cp16(sv + (buf * SKT_BN + key) * LDV + (c - D), vcache + at * V + (c - D), row >= 0);
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
     const int n_tiles = (p_hi - k_lo) / SKT_BN + 1;
-    stage(0, k_lo);                                   // (one group holds Q and the first keys)
+    const bool finds = tid < SKT_BN;
+    if (finds) {
+        tile_rows[0][tid] = find_row(k_lo);
+        tile_rows[1][tid] = n_tiles > 1 ? find_row(k_lo + SKT_BN) : -1;
+    }
+    __syncthreads();
+    stage(0);                                         // (one group holds Q and the first keys)
     unsigned qf[D / 16][4];
     float o[V / 8][4];
 #pragma unroll
@@ -403,7 +418,7 @@ __global__ void __launch_bounds__(128) sink_attention_tiles_kernel(
     const float scale2 = scale * SK_LOG2E;
     const int my_pos0 = p_lo + warp * 16 + (lane >> 2), my_pos1 = my_pos0 + 8;       // positions of this thread's two rows
     const int first0 = gb_first_key(my_pos0, mask), first1 = gb_first_key(my_pos1, mask);
-    const float cap2 = cap * SK_LOG2E, inv_cap2 = cap > 0.f ? 2.0f / cap : 0.f;
+    const float cap2 = cap * SK_LOG2E, inv_cap2 = CAP ? 2.0f * scale / cap : 0.f;
     float mrow[2] = {sink2, sink2}, lrow[2] = {0.f, 0.f};                             // (a thread's share of the denominator)
     // The bias depends on the distance alone, and a tile of 64 rows x 64 keys holds 127 distances: one logarithm per thread
     // and tile instead of one per score. sbias[i] belongs to the distance (p_lo - kb) + i - 63, which is row - key + 63
@@ -413,13 +428,16 @@ __global__ void __launch_bounds__(128) sink_attention_tiles_kernel(
     for (int t = 0; t < n_tiles; ++t) {
         const int kb = k_lo + t * SKT_BN, buf = t & 1;
         if (r1) sbias[tid] = b1 * log2f(fmaf(b2, (float)max(p_lo - kb + tid - 63, 0), 1.0f));   // (read after the barrier below)
+        long long later = -1;
+        if (finds && t + 2 < n_tiles) later = find_row(kb + 2 * SKT_BN);
         if (t + 1 < n_tiles) {
-            stage(buf ^ 1, kb + SKT_BN);
+            stage(buf ^ 1);
             asm volatile("cp.async.wait_group 1;" ::: "memory");
         } else {
             asm volatile("cp.async.wait_group 0;" ::: "memory");
         }
         __syncthreads();
+        if (finds) tile_rows[buf][tid] = later;       // (read after the barrier at the end of this round)
         if (t == 0) {
 #pragma unroll
             for (int kd = 0; kd < D / 16; ++kd) {
@@ -459,11 +477,12 @@ __global__ void __launch_bounds__(128) sink_attention_tiles_kernel(
             float mx[2] = {mrow[0], mrow[1]};
 #pragma unroll
             for (int j = 0; j < SKT_BN / 8; ++j) {
+                if constexpr (CAP) gb_cap_fast4(s[j], cap2, inv_cap2);
 #pragma unroll
                 for (int e = 0; e < 4; ++e) {
                     const int key = kb + j * 8 + (lane & 3) * 2 + (e & 1);
                     const int pos = e < 2 ? my_pos0 : my_pos1;
-                    float v = cap > 0.f ? gb_cap_fast(s[j][e] * scale, cap2, inv_cap2) : s[j][e] * scale2;
+                    float v = CAP ? s[j][e] : s[j][e] * scale2;
                     if (r1) v -= my_bias[(e >> 1) * 8 - j * 8 - (e & 1)];
                     if (!whole) {
                         const bool sees = key <= pos && key >= (e < 2 ? first0 : first1) && pos <= p_hi;
@@ -557,8 +576,9 @@ static int skt_launch(const void* q, void* out, const void* kcache, const void* 
                       const float* gate, long long ld_gate, int num_seqs, int tiles_per_seq, int H, int G, int page_size,
                       long long num_pages, float scale, float cap, int mask, int gate_channels, int* status, cudaStream_t stream) {
     const size_t smem = ((size_t)3 * SKT_BM * (D + 8) + (size_t)2 * SKT_BN * (V + 8)) * 2;
-    cudaFuncSetAttribute(sink_attention_tiles_kernel<D, V>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    gb_launch(GB_PDL_ATTENTION, sink_attention_tiles_kernel<D, V>, dim3(num_seqs * tiles_per_seq, H), dim3(128), smem, stream,
+    auto kernel = cap > 0.f ? sink_attention_tiles_kernel<D, V, true> : sink_attention_tiles_kernel<D, V, false>;
+    cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    gb_launch(GB_PDL_ATTENTION, kernel, dim3(num_seqs * tiles_per_seq, H), dim3(128), smem, stream,
               (const __nv_bfloat16*)q, (__nv_bfloat16*)out, (const __nv_bfloat16*)kcache, (const __nv_bfloat16*)vcache, block_tables,
               max_pages, seq_first_row, seq_start_pos, r1, r2, sink, gate, ld_gate, num_seqs, tiles_per_seq, H, G, page_size, num_pages,
               scale, cap, mask, gate_channels, status);

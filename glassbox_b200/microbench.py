@@ -33,6 +33,11 @@ over operands that rotate through more memory than L2 holds.
     python -m glassbox_b200.microbench felovik                           Felovik's kernels, each beside its like kernel: attention with a
                                                                          gate per channel, the state-space mixer, the norm after the sum,
                                                                          the router and the SwiGLU experts
+    python -m glassbox_b200.microbench lodenex                           Lodenex's kernels, each beside its like kernel: capped attention
+                                                                         within chunks beside sink attention with a window; windowed
+                                                                         latent attention, its inputs and its up-projections; the norm
+                                                                         over whole projections with rotation and cache write; GELU in
+                                                                         a product's epilogue; capped logits
 
 Prints one line per case: microseconds and GB/s or TFLOP/s of the algorithmic bytes or flops. With ``--once`` after
 the case's name every kernel is launched exactly once and nothing is timed: the form in which a profiler captures one
@@ -1058,7 +1063,120 @@ def bench_felovik() -> None:
     kernels.check_status(status)
 
 
-CASES = ("gemm_stream", "gemm_tc", "attention_decode", "attention_splits", "attention_prefill", "float32", "small", "decode_program", "layer_gemms", "latent_attention", "delta_rule", "lonorax", "tagenex", "babotar", "felovik")
+def bench_lodenex() -> None:
+    """Each kernel of the Lodenex path beside the like kernel of the closest path, at the sizes of the width-1024 and width-2048
+    models that ``bench.py --workload lodenex`` runs."""
+    status = torch.zeros(1, dtype=torch.int32, device=DEV)
+    ps, hd, t_len, ctx, span, c = 16, 64, 2048, 4096, 1024, 128
+    for d, H, G, r, qr in ((1024, 16, 4, 32, 512), (2048, 32, 8, 64, 768)):
+        per = t_len // ps
+        kc = torch.randn(per + 2, G, ps, hd, device=DEV).bfloat16()
+        vc = torch.randn_like(kc)
+        tables = torch.arange(per, dtype=torch.int32, device=DEV).view(1, per).contiguous()
+        first = torch.tensor([0, t_len], dtype=torch.int32, device=DEV)
+        start = torch.zeros(1, dtype=torch.int32, device=DEV)
+        pos = torch.arange(t_len, dtype=torch.int32, device=DEV)
+        q = torch.randn(t_len, H * hd, device=DEV).bfloat16()
+        o = torch.empty_like(q)
+        gate, sink = torch.randn(t_len, H, device=DEV), torch.zeros(H, device=DEV)
+        r1, r2 = torch.full((H,), 0.5, device=DEV), torch.full((H,), 0.3, device=DEV)
+        in_chunks = 2.0 * (t_len // span) * (span * (span + 1) // 2) * H * 2 * hd
+        in_window = 2.0 * sum(min(p + 1, span) for p in range(t_len)) * H * 2 * hd
+        own = (None, None, sink, gate)
+        rows = (("capped, chunks of 1024, sink and gate", own, dict(softcap=30.0, chunk=span), None, in_chunks),
+                ("   the same without the cap", own, dict(chunk=span), None, in_chunks),
+                ("   distance bias, sink and gate, window 1024", (r1, r2, sink, gate), {}, span, in_window),
+                ("   grouped-query, window 1024", None, {}, span, in_window))
+        for name, terms, kw, window, fl in rows:
+            t = graph_time(lambda: kernels.attention_prefill_tc(q, o, kc, vc, tables, first, start, t_len, H, G, hd, ps, hd ** -0.5, window, status,
+                                                                sink_terms=terms, **kw), reps=6)
+            print(f"{name}: prompt attention (tcgen05) heads {H}/{G} x {hd}, {t_len} tokens: {t:7.1f} us {fl / t / 1e6:6.1f} TFLOP/s", flush=True)
+        for D in (96, 128):
+            kd, qd = torch.randn(per + 2, G, ps, D, device=DEV).bfloat16(), torch.randn(t_len, H * D, device=DEV).bfloat16()
+            vd, od = torch.randn_like(kd), torch.empty_like(qd)
+            for name, kw in (("capped, chunks of 1024", dict(softcap=30.0, chunk=span, window=None)), ("   window 1024", dict(window=span))):
+                t = graph_time(lambda: kernels.sink_attention_tiles(qd, od, kd, vd, tables, first, start, t_len, r1=None, r2=None, sink=sink, gate=gate,
+                                                                    heads=H, kv_heads=G, dim=D, vdim=D, page_size=ps, scale=D ** -0.5,
+                                                                    status=status, **kw), reps=6)
+                fl = (in_window if kw["window"] else in_chunks) / hd * D
+                print(f"{name}: prompt attention (mma.sync tiles) heads {H}/{G} x {D}: {t:7.1f} us {fl / t / 1e6:6.1f} TFLOP/s", flush=True)
+        w = c + r
+        lc = torch.randn(per + 2, 1, ps, w, device=DEV).bfloat16()
+        ql, ol = torch.randn(t_len, H * w, device=DEV).bfloat16(), torch.empty(t_len, H * c, device=DEV).bfloat16()
+        for window in (span, None):
+            keys = sum(min(p + 1, window or t_len) for p in range(t_len))
+            t = graph_time(lambda: kernels.latent_attention_mma(ql, ol, lc, tables, first, start, pos, None, H, c, r, ps, w ** -0.5, window, status,
+                                                                max_rows_per_seq=t_len), reps=6)
+            fl = 2.0 * keys * H * (w + c)
+            print(f"latent attention prompt heads {H} latent {c}+{r}, window {window}: {t:7.1f} us {fl / t / 1e6:6.1f} TFLOP/s", flush=True)
+        for m in (1, 8, 64):
+            per = ctx // ps
+            kd = torch.randn(m * per + 4, G, ps, hd, device=DEV).bfloat16()
+            vd = torch.randn_like(kd)
+            tb = torch.arange(m * per, dtype=torch.int32, device=DEV).view(m, per).contiguous()
+            row_seq = torch.arange(m, dtype=torch.int32, device=DEV)
+            pd = torch.full((m,), ctx - 1, dtype=torch.int32, device=DEV)
+            qd, od = torch.randn(m, H * hd, device=DEV).bfloat16(), torch.empty(m, H * hd, device=DEV).bfloat16()
+            nbytes = m * span * G * hd * 2 * 2
+            sp, block_keys, warps = kernels.decode_mma_plan(m, G, hd, span)
+            pa = torch.empty(m * H * warps * sp * hd, device=DEV)
+            pm = torch.empty(m * H * warps * sp * 2, device=DEV)
+            cn = torch.zeros(m * G, dtype=torch.int32, device=DEV)
+            rows = (("capped, chunks of 1024, sink and gate", (None, None, sink, gate[:m]), dict(softcap=30.0, chunk=span), None),
+                    ("   distance bias, sink and gate, window 1024", (r1, r2, sink, gate[:m]), {}, span),
+                    ("   grouped-query, window 1024", None, {}, span))
+            for name, terms, kw, window in rows:
+                t = graph_time(lambda: kernels.attention_decode_mma(qd, od, kd, vd, tb, row_seq, pd, H, G, hd, ps, hd ** -0.5, window, sp, pa, pm, cn,
+                                                                    status, block_keys, warps, sink_terms=terms, **kw))
+                print(f"{name}: decode attention heads {H}/{G} x {hd} batch {m:3d}: {t:7.1f} us {nbytes / t / 1e3:6.0f} GB/s", flush=True)
+            lc = torch.randn(m * per + 4, 1, ps, w, device=DEV).bfloat16()
+            fr = torch.arange(m + 1, dtype=torch.int32, device=DEV)
+            qd, od = torch.randn(m, H * w, device=DEV).bfloat16(), torch.empty(m, H * c, device=DEV).bfloat16()
+            for window in (span, None):
+                shares = kernels.latent_decode_splits(m, H, window or ctx)
+                po, pl = torch.empty(m, H * shares * c, device=DEV), torch.empty(m, H * shares * 2, device=DEV)
+                t = graph_time(lambda: kernels.latent_attention_mma(qd, od, lc, tb, fr, pd, pd, None, H, c, r, ps, w ** -0.5, window, status,
+                                                                    decode=True, splits=shares, part_o=po, part_ml=pl))
+                print(f"latent attention decode heads {H} latent {c}+{r} batch {m:3d} window {window}: {t:7.1f} us "
+                      f"{m * (window or ctx) * w * 2 / t / 1e3:6.0f} GB/s", flush=True)
+        freqs, qn, kn, hn = (torch.rand(k, device=DEV) for k in (hd // 2, H * hd, G * hd, hd))
+        cols, inner = (H + 2 * G) * hd, H * hd
+        for n in (t_len, 8):
+            p = pos[:n]
+            proj, qo = torch.randn(n, cols, device=DEV), torch.empty(n, H * hd, device=DEV).bfloat16()
+            t = graph_time(lambda: kernels.projection_norm_rope_write(proj, qn, kn, freqs, 1.0, p, p, qo, kc, vc, H, G, hd, hd, hd, 1e-6, ps, True,
+                                                                      status))
+            t2 = graph_time(lambda: kernels.qk_norm_rope_write(proj, hn, hn, freqs, p, p, qo, kc, vc, H, G, hd, hd, hd, 1e-6, ps, True, status))
+            print(f"norm over the projections + rotation + cache write heads {H}/{G}, {n:4d} rows: {t:6.1f} us {n * cols * 6 / t / 1e3:6.0f} GB/s; "
+                  f"norm per head + rotation + cache write {t2:6.1f} us", flush=True)
+            lat, cq = torch.randn(n, qr + w, device=DEV), torch.empty(n, qr, device=DEV).bfloat16()
+            ln, lk = torch.rand(qr, device=DEV), torch.rand(c, device=DEV)
+            lcache = torch.empty(n, 1, ps, w, device=DEV).bfloat16()
+            t = graph_time(lambda: kernels.latent_inputs(lat, ln, lk, freqs, 1.1, p, p, cq, lcache, c, r, r, 1e-6, True, status))
+            print(f"latent inputs (both norms, key rotation, cache write) {qr} + {c} + {r}, {n:4d} rows: {t:6.1f} us "
+                  f"{n * (qr + w) * 6 / t / 1e3:6.0f} GB/s", flush=True)
+            uq, qa = torch.randn(n, H * (hd + r), device=DEV).bfloat16(), torch.empty(n, H * w, device=DEV).bfloat16()
+            t = graph_time(lambda: kernels.latent_kv_write(uq, 0, qa, lcache, None, freqs, p, p, H, hd, r, c, r, 1e-6, False, status,
+                                                           half_pairs=True, magnitude=1.1))
+            print(f"query rotation heads {H} x {r}, {n:4d} rows: {t:6.1f} us {n * H * r * 4 / t / 1e3:6.0f} GB/s", flush=True)
+            wk, wv = torch.randn(H, c, hd, device=DEV).bfloat16(), torch.randn(H, hd, c, device=DEV).bfloat16()
+            la, at, lg = torch.randn(n, H * c, device=DEV).bfloat16(), torch.empty(n, inner, device=DEV).bfloat16(), torch.randn(n, inner, device=DEV)
+            t = graph_time(lambda: kernels.head_linear(uq, wk, qa, hd + r, w))
+            t2 = graph_time(lambda: kernels.head_linear(la, wv, at, c, hd, gate=lg))
+            t3 = graph_time(lambda: kernels.head_linear(la, wv, at, c, hd))
+            print(f"up-projections per head {H}, {n:4d} rows: key {t:6.1f} us, value with a gate {t2:6.1f} us, without {t3:6.1f} us", flush=True)
+            x, up, act = torch.randn(n, d, device=DEV).bfloat16(), torch.randn(4 * d, d, device=DEV).bfloat16(), torch.empty(n, 4 * d, device=DEV).bfloat16()
+            product = kernels.gemm_tc if n > 64 else kernels.gemm_stream
+            t, t2, t3 = (graph_time(lambda: product(x, up, act, **kw)) for kw in (dict(gelu=True), dict(relu2=True), {}))
+            print(f"up product {4 * d} x {d} with GELU, {n:4d} rows: {t:6.1f} us, with squared ReLU {t2:6.1f} us, plain {t3:6.1f} us", flush=True)
+        for n in (64, 1):
+            logits = torch.randn(n, 32768, device=DEV)
+            t, t2 = graph_time(lambda: kernels.tanh_cap_(logits, 30.0)), graph_time(lambda: kernels.scale_(logits, 1.0))
+            print(f"capped logits {n} x 32768: {t:6.1f} us, scaled {t2:6.1f} us", flush=True)
+    kernels.check_status(status)
+
+
+CASES = ("gemm_stream", "gemm_tc", "attention_decode", "attention_splits", "attention_prefill", "float32", "small", "decode_program", "layer_gemms", "latent_attention", "delta_rule", "lonorax", "tagenex", "babotar", "felovik", "lodenex")
 
 
 def main(argv) -> int:
@@ -1100,6 +1218,8 @@ def main(argv) -> int:
         bench_babotar()
     elif argv[0] == "felovik":
         bench_felovik()
+    elif argv[0] == "lodenex":
+        bench_lodenex()
     else:
         bench_attention_prefill()
     return 0

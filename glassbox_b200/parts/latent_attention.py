@@ -99,7 +99,7 @@ class LatentAttention(Mixer):
             raise ValueError("a latent attention layer without a projection of its own cannot write a cache layer")
         width, s = sum(self.input_pieces()), self.spec
         first = self.first_cols
-        freqs = self.position.inv_freq(h.device) if r else h.new_zeros(1, dtype=torch.float32)
+        freqs = self.position.inv_freq(ctx.device) if r else ctx.zeros_once("no_frequencies", 1, torch.float32)
         rot, magnitude = (self.position.rotary_dim, self.position.magnitude) if r else (0, 1.0)
         qabs = ctx.scratch("latent_q", (n, H * (c + r)))
         stores = writes_cache and self.owns_cache
