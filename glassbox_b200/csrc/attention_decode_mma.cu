@@ -112,7 +112,7 @@ static int launch_mma(const void* q, long long q_stride, void* out, long long ou
 // 1 if (head size, group size) is one this kernel is built for.
 GB_EXPORT int gb_attention_decode_mma_supported(int nh, int nkv, int hd) {
     if (nkv <= 0 || nh % nkv) return 0;
-    return (hd == 16 || hd == 32 || hd == 64 || hd == 128) && nh / nkv <= 16;
+    return (hd == 16 || hd == 32 || hd == 64 || hd == 96 || hd == 128) && nh / nkv <= 16;
 }
 
 // As gb_attention_decode_mma, with the choice of launching under programmatic stream serialisation
@@ -128,7 +128,7 @@ static int decode_mma_dispatch(const void* q, long long q_stride, void* out, lon
                                int splits, float* part_acc, float* part_ml, int* counters, int* status,
                                int pdl, int block_keys, int warps, cudaStream_t stream, const DecodeSinkTerms& terms) {
     GB_REQUIRE(gb_attention_decode_mma_supported(nh, nkv, hd),
-               "gb_attention_decode_mma: head size %d with %d heads per kv head is not built (16/32/64/128, <= 16)", hd,
+               "gb_attention_decode_mma: head size %d with %d heads per kv head is not built (16/32/64/96/128, <= 16)", hd,
                nkv > 0 ? nh / nkv : 0);
     GB_REQUIRE(page_size >= 16 && (page_size & (page_size - 1)) == 0,
                "gb_attention_decode_mma: page size %d must be a power of two >= 16", page_size);
@@ -152,6 +152,7 @@ static int decode_mma_dispatch(const void* q, long long q_stride, void* out, lon
         if (warps == 8) { GB_MMAW(64, 32, 8) }     // a small batch: one block per SM, twice the warps
         GB_MMA(64, 32)
     }
+    if (hd == 96) { GB_MMA(96, 16) }
     GB_MMA(128, 16)
 #undef GB_MMA
 #undef GB_MMAW

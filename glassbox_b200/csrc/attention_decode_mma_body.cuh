@@ -87,6 +87,13 @@ template <> struct RowLoad<4> {
         w[0] = v.x; w[1] = v.y; w[2] = v.z; w[3] = v.w;
     }
 };
+template <> struct RowLoad<6> {
+    static __device__ __forceinline__ void load(const __nv_bfloat16* p, uint32_t (&w)[6]) {
+        const uint2* q = reinterpret_cast<const uint2*>(p);      // (a share of 24 bytes starts 8-byte aligned)
+        const uint2 a = q[0], b = q[1], c = q[2];
+        w[0] = a.x; w[1] = a.y; w[2] = b.x; w[3] = b.y; w[4] = c.x; w[5] = c.y;
+    }
+};
 template <> struct RowLoad<8> {
     static __device__ __forceinline__ void load(const __nv_bfloat16* p, uint32_t (&w)[8]) {
         uint4 a = *reinterpret_cast<const uint4*>(p), b = *reinterpret_cast<const uint4*>(p + 8);

@@ -3,7 +3,7 @@
 //
 // This is the shape of the up-projections of latent attention once they are moved to the query and to the weighted sum
 // of latents: K and N are a head's sizes (tens to a few hundred), so a head's product is far too small for a launch of
-// its own. Optionally every output is multiplied by sigmoid(gate[row, h, column]), a logit per output (float32 or bfloat16).
+// its own. Optionally a rotated part behind each head's inputs is turned and carried over, and every output is multiplied by sigmoid(gate[row, h, column]), a logit per output (float32 or bfloat16).
 // One block = 64 rows x one head x up to 128 output columns (64 for narrow heads); a and w[h] are staged once in shared memory
 // (rows padded by 16 bytes so that ldmatrix meets no bank twice), each of the four warps takes 16 rows.
 #include "common.cuh"
@@ -33,11 +33,21 @@ __device__ __forceinline__ float2 hl_pair(const void* gate, int kind, size_t at)
 }
 __device__ __forceinline__ float hl_open(float v, float z) { return __fdividef(v, 1.0f + __expf(-z)); }      // v times sigmoid(z)
 
+// The rotated numbers behind a head's K inputs (dims > 0): a[row, h, K : K + dims] goes to out[row, h, N : N + dims], number i
+// turned with number i + half (i < half) by the row's position times inv_freq[i], sine and cosine times `magnitude`, the numbers
+// from 2 half on as they are. Padding rows (position < 0) are left alone.
+struct HlTurn {
+    const int* positions;
+    const float* inv_freq;
+    float magnitude;
+    int half, dims;
+};
+
 template <int BN, bool GATED>
 __global__ void __launch_bounds__(128) head_linear_kernel(const __nv_bfloat16* __restrict__ a, long long lda, long long a_head,
                                                           const __nv_bfloat16* __restrict__ w, __nv_bfloat16* __restrict__ out,
                                                           long long ldc, long long c_head, int n, int N, int K,
-                                                          const void* __restrict__ gate, long long ld_gate, int gate_kind) {
+                                                          const void* __restrict__ gate, long long ld_gate, int gate_kind, HlTurn turn) {
     extern __shared__ __align__(128) unsigned char hl_smem[];
     gb_pdl_launch_dependents();
     const int KS = K + 8;                                    // padded row, elements
@@ -104,6 +114,28 @@ __global__ void __launch_bounds__(128) head_linear_kernel(const __nv_bfloat16* _
             }
         }
     }
+    if (turn.dims > 0 && blockIdx.z == 0) {
+        const int per = turn.half + (turn.dims - 2 * turn.half);      // pairs, then numbers that pass unchanged
+        for (int idx = threadIdx.x; idx < HL_BM * per; idx += 128) {
+            const int r = idx / per, k = idx - r * per, row = m0 + r;
+            if (row >= n) break;
+            const int pos = turn.positions[row];
+            if (pos < 0) continue;
+            const __nv_bfloat16* src = ah + (size_t)row * lda + K;
+            __nv_bfloat16* dst = out + (size_t)row * ldc + (size_t)head * c_head + N;
+            if (k >= turn.half) {
+                dst[k + turn.half] = src[k + turn.half];
+                continue;
+            }
+            float sn, cs;
+            sincosf((float)pos * turn.inv_freq[k], &sn, &cs);
+            sn *= turn.magnitude;
+            cs *= turn.magnitude;
+            const float u = __bfloat162float(src[k]), v = __bfloat162float(src[k + turn.half]);
+            dst[k] = __float2bfloat16_rn(u * cs - v * sn);
+            dst[k + turn.half] = __float2bfloat16_rn(v * cs + u * sn);
+        }
+    }
     __nv_bfloat16* oh = out + (size_t)head * c_head + n0;
 #pragma unroll
     for (int nt = 0; nt < BN / 8; ++nt) {
@@ -135,7 +167,9 @@ GB_EXPORT int gb_head_linear_supported(const void* a, long long lda, long long a
 
 GB_EXPORT int gb_head_linear(const void* a, long long lda, long long a_head, const void* w, void* out, long long ldc,
                              long long c_head, int n, int heads, int N, int K, const void* gate, long long ld_gate, int gate_f32,
-                             cudaStream_t stream) {
+                             const int* positions, const float* inv_freq, float magnitude, int rot_dims, int dims, cudaStream_t stream) {
+    GB_REQUIRE(dims == 0 || (positions != nullptr && rot_dims >= 0 && rot_dims <= dims && rot_dims % 2 == 0 && (rot_dims == 0 || inv_freq != nullptr)),
+               "gb_head_linear: %d rotated numbers do not fit a part of %d", rot_dims, dims);
     GB_REQUIRE(gate == nullptr || ld_gate >= (long long)heads * N, "gb_head_linear: rows of gate logits are too short");
     GB_REQUIRE(gb_head_linear_supported(a, lda, a_head, w, out, ldc, c_head, N, K),
                "gb_head_linear: K=%d must be a multiple of 16 up to %d, N=%d even, operands aligned", K, HL_MAX_K, N);
@@ -147,7 +181,7 @@ GB_EXPORT int gb_head_linear(const void* a, long long lda, long long a_head, con
     const int bn = narrow ? HL_BN / 2 : HL_BN;
     const size_t smem = (size_t)(HL_BM + bn) * (K + 8) * sizeof(__nv_bfloat16);
     void (*kernel)(const __nv_bfloat16*, long long, long long, const __nv_bfloat16*, __nv_bfloat16*, long long, long long, int, int, int, const void*,
-                   long long, int) = narrow ? (gate ? head_linear_kernel<HL_BN / 2, true> : head_linear_kernel<HL_BN / 2, false>)
+                   long long, int, HlTurn) = narrow ? (gate ? head_linear_kernel<HL_BN / 2, true> : head_linear_kernel<HL_BN / 2, false>)
                                             : (gate ? head_linear_kernel<HL_BN, true> : head_linear_kernel<HL_BN, false>);
     static size_t allowed[4] = {48 * 1024, 48 * 1024, 48 * 1024, 48 * 1024};
     size_t& have = allowed[(narrow ? 2 : 0) + (gate ? 1 : 0)];
@@ -157,7 +191,7 @@ GB_EXPORT int gb_head_linear(const void* a, long long lda, long long a_head, con
     }
     dim3 grid(gb_ceil_div(n, HL_BM), heads, gb_ceil_div(N, bn));
     cudaError_t e = gb_launch(GB_PDL_GEMM, kernel, grid, dim3(128), smem, stream, (const __nv_bfloat16*)a, lda, a_head, (const __nv_bfloat16*)w,
-                              (__nv_bfloat16*)out, ldc, c_head, n, N, K, gate, ld_gate, kind);
+                              (__nv_bfloat16*)out, ldc, c_head, n, N, K, gate, ld_gate, kind, HlTurn{positions, inv_freq, magnitude, rot_dims / 2, dims});
     if (e != cudaSuccess) {
         gb_set_error("gb_head_linear: launch failed: %s", cudaGetErrorString(e));
         return 2;

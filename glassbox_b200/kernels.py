@@ -106,7 +106,7 @@ _SIGNATURES = {
     "gb_latent_attention_mma": [_P, _P, _P, _P, _P, _P, _I, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _LL, _F, _I, _I, _I,
                                 _P, _P],
     "gb_head_linear_supported": [_P, _LL, _LL, _P, _P, _LL, _LL, _I, _I],
-    "gb_head_linear": [_P, _LL, _LL, _P, _P, _LL, _LL, _I, _I, _I, _I, _P, _LL, _I, _P],
+    "gb_head_linear": [_P, _LL, _LL, _P, _P, _LL, _LL, _I, _I, _I, _I, _P, _LL, _I, _P, _P, _F, _I, _I, _P],
     "gb_embed_positions": [_P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _F, _P, _P],
     "gb_residual_conv": [_P, _I, _P, _I, _P, _P, _LL, _LL, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _P, _P],
     "gb_gelu_glu": [_P, _I, _LL, _P, _I, _I, _I, _P],
@@ -851,7 +851,7 @@ def attention_decode_mma(q: torch.Tensor, out: torch.Tensor, kcache: torch.Tenso
               _ptr(status), 1 if USE_PDL else 0, int(block_keys), int(warps), *terms, by_channel, float(softcap or 0.0), _stream())
         return
     assert softcap is None and chunk is None
-    if prog is not None and prog.takes_rows(n):
+    if prog is not None and prog.takes_rows(n) and hd in (16, 32, 64, 128):      # (the head sizes a program is built for)
         if not prog.takes_attention(hd, block_keys):
             prog.flush()
             prog._status = status
@@ -1139,17 +1139,30 @@ def head_linear_supported(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, a
                                                w.shape[1], w.shape[2]))
 
 
-def head_linear(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, a_head: int, c_head: int, gate: Optional[torch.Tensor] = None) -> None:
+#: up to this many rows the per-head product carries the rotated part over (8 rows, 16 and 32 heads: 4.0 and 4.5 us in one launch
+#: against 5.3 and 6.9 in two); beyond, every head's blocks would form the angles again (2,048 rows: 12.1 and 30.2 us against 10.8
+#: and 21.5) and the rotation is a launch of its own
+HEAD_TURN_MAX_ROWS = 64
+
+
+def head_linear(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, a_head: int, c_head: int, gate: Optional[torch.Tensor] = None,
+                turn=None) -> None:
     """out[row, h * c_head : h * c_head + N] = a[row, h * a_head : h * a_head + K] @ w[h]^T for every head h of
     w [heads, N, K], in one launch (bfloat16, float32 sums). ``gate`` [n, heads * N] (float32 or bfloat16 logits, rows may be
-    strided): every output is multiplied by sigmoid(gate[row, h * N + column]) first."""
+    strided): every output is multiplied by sigmoid(gate[row, h * N + column]) first. ``turn`` = (positions, inv_freq, magnitude, rot_dims, dims): the
+    ``dims`` numbers behind a head's K inputs go behind its N outputs, the first ``rot_dims`` of them rotated at the row's position
+    (number i with number i + rot_dims/2, sine and cosine times ``magnitude``)."""
+    positions, freqs, magnitude, rot, dims = turn if turn is not None else (None, None, 1.0, 0, 0)
+    _cuda(positions, freqs)
+    assert not dims or (a_head >= w.shape[2] + dims and c_head >= w.shape[1] + dims and positions.numel() >= a.shape[0])
     _cuda(a, w, out, gate)
     assert gate is None or (gate.shape == (a.shape[0], w.shape[0] * w.shape[1]) and gate.stride(1) == 1)
     heads, N, K = w.shape
     n = a.shape[0]
     assert out.shape[0] == n and a.shape[1] >= (heads - 1) * a_head + K and out.shape[1] >= (heads - 1) * c_head + N
     _call("gb_head_linear", _ptr(a), a.stride(0), a_head, _ptr(w), _ptr(out), out.stride(0), c_head, n, heads, N, K, _ptr(gate),
-          gate.stride(0) if gate is not None else 0, 1 if gate is not None and gate.dtype == torch.float32 else 0, _stream())
+          gate.stride(0) if gate is not None else 0, 1 if gate is not None and gate.dtype == torch.float32 else 0, _ptr(positions),
+          _ptr(freqs), float(magnitude), int(rot), int(dims), _stream())
 
 
 def latent_attention_mma_supported(dtype: torch.dtype, c: int, r: int, page_size: int) -> bool:

@@ -1162,9 +1162,10 @@ def bench_lodenex() -> None:
             wk, wv = torch.randn(H, c, hd, device=DEV).bfloat16(), torch.randn(H, hd, c, device=DEV).bfloat16()
             la, at, lg = torch.randn(n, H * c, device=DEV).bfloat16(), torch.empty(n, inner, device=DEV).bfloat16(), torch.randn(n, inner, device=DEV)
             t = graph_time(lambda: kernels.head_linear(uq, wk, qa, hd + r, w))
+            t4 = graph_time(lambda: kernels.head_linear(uq, wk, qa, hd + r, w, turn=(p, freqs, 1.1, r, r)))
             t2 = graph_time(lambda: kernels.head_linear(la, wv, at, c, hd, gate=lg))
             t3 = graph_time(lambda: kernels.head_linear(la, wv, at, c, hd))
-            print(f"up-projections per head {H}, {n:4d} rows: key {t:6.1f} us, value with a gate {t2:6.1f} us, without {t3:6.1f} us", flush=True)
+            print(f"up-projections per head {H}, {n:4d} rows: key {t:6.1f} us, with the query rotation {t4:6.1f} us, value with a gate {t2:6.1f} us, without {t3:6.1f} us", flush=True)
             x, up, act = torch.randn(n, d, device=DEV).bfloat16(), torch.randn(4 * d, d, device=DEV).bfloat16(), torch.empty(n, 4 * d, device=DEV).bfloat16()
             product = kernels.gemm_tc if n > 64 else kernels.gemm_stream
             t, t2, t3 = (graph_time(lambda: product(x, up, act, **kw)) for kw in (dict(gelu=True), dict(relu2=True), {}))

@@ -102,7 +102,7 @@ class LatentAttention(Mixer):
         freqs = self.position.inv_freq(ctx.device) if r else ctx.zeros_once("no_frequencies", 1, torch.float32)
         rot, magnitude = (self.position.rotary_dim, self.position.magnitude) if r else (0, 1.0)
         qabs = ctx.scratch("latent_q", (n, H * (c + r)))
-        stores = writes_cache and self.owns_cache
+        stores, turn = writes_cache and self.owns_cache, None
         if s.q_rank is not None:
             # float32 sums (rows padded to 16 bytes) up to the norms
             proj = ctx.scratch("latent_proj32", (n, -(-width // 4) * 4), torch.float32)[:, :width]
@@ -112,8 +112,11 @@ class LatentAttention(Mixer):
                                   cache.slots, cq, cache.k, c, r, rot, s.latent_eps, stores, ctx.status)
             q = ctx.scratch("latent_uq", (n, self.q_cols))
             linear(ctx, cq, self.params["w_uq"], q)
-            kernels.latent_kv_write(q, 0, qabs, cache.k, None, freqs, ctx.positions, cache.slots, H, dq, r, c, rot, s.latent_eps, False,
-                                    ctx.status, half_pairs=True, magnitude=magnitude)
+            if n <= kernels.HEAD_TURN_MAX_ROWS and dq and kernels.head_linear_supported(q, self.w_uk_t, qabs, dq + r, c + r):
+                turn = (ctx.positions, freqs, magnitude, rot, r) if r else None      # the product below carries the rotated part
+            else:
+                kernels.latent_kv_write(q, 0, qabs, cache.k, None, freqs, ctx.positions, cache.slots, H, dq, r, c, rot, s.latent_eps,
+                                        False, ctx.status, half_pairs=True, magnitude=magnitude)
         else:
             proj = q = ctx.scratch("latent_proj", (n, width))
             linear(ctx, h, self.params["w_in"], proj)
@@ -123,7 +126,7 @@ class LatentAttention(Mixer):
         gate = proj[:, width - H * dv:] if s.output_gate else None
         # the key up-projection, applied to the query: one launch for all heads where the sizes allow, else head by head
         if dq and kernels.head_linear_supported(q, self.w_uk_t, qabs, dq + r, c + r):
-            kernels.head_linear(q, self.w_uk_t, qabs, dq + r, c + r)
+            kernels.head_linear(q, self.w_uk_t, qabs, dq + r, c + r, turn=turn)
         else:
             q3 = qabs.view(n, H, c + r)
             p3 = q[:, :self.q_cols].unflatten(1, (H, dq + r))

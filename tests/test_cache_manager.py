@@ -156,6 +156,56 @@ def test_window_keeps_what_a_long_portion_needs():
     m.check_invariants()
 
 
+def chunked(pages, chunk, page_size=16, window=None, **kw):
+    return CacheManager([GroupSpec(pages, page_size, window, chunk=chunk)], share_prefixes=False, **kw)
+
+
+def test_chunks_give_pages_back_when_the_next_token_starts_a_new_one():
+    m = chunked(4, chunk=48)                       # a chunk is three pages
+    m.add_request("a")
+    for n in range(1, 101):
+        feed(m, "a", [1])
+        m.check_invariants()
+        table = m.table(0, "a")
+        first = n // 48 * 48 // 16                 # the page that holds the first key the next token can see
+        assert all(p == -1 for p in table[:first]) and all(p >= 0 for p in table[first:]), n
+    assert m.used_pages() == 1 and m.table(0, "a")[:6] == [-1] * 6 and len(m.table(0, "a")) == 7
+    m.free_request("a")
+    assert m.free_pages() == 4
+
+
+def test_a_page_that_two_chunks_share_stays_until_the_later_one_ends():
+    m = chunked(4, chunk=24)                       # chunks end in the middle of a page
+    m.add_request("a")
+    feed(m, "a", [1] * 24)                         # the next token, 24, lies on page 1: page 0 is behind it
+    assert m.table(0, "a") == [-1, 1]
+    feed(m, "a", [1] * 23)
+    assert m.table(0, "a")[0] == -1 and m.used_pages() == 2
+    feed(m, "a", [1])                              # token 48 starts a chunk and a page
+    assert m.used_pages() == 0 and m.table(0, "a") == [-1] * 3
+    feed(m, "a", [1])
+    assert m.used_pages() == 1
+
+
+def test_chunks_keep_what_a_long_portion_needs():
+    m = chunked(8, chunk=32)
+    m.add_request("a")
+    m.reserve("a", 100)                            # every row of the portion needs the keys of its own chunk
+    assert all(p >= 0 for p in m.table(0, "a")) and len(m.table(0, "a")) == 7
+    m.commit("a", [0] * 100)                       # token 100 belongs to the chunk that starts at 96
+    assert m.table(0, "a")[:6] == [-1] * 6 and m.table(0, "a")[6] >= 0
+    with pytest.raises(ValueError):
+        m.truncate("a", 90)                        # position 90 would see keys from 64 on
+    m.truncate("a", 97)
+    m.check_invariants()
+
+
+def test_chunks_switch_prefix_sharing_off_and_bound_what_a_group_holds():
+    m = CacheManager([GroupSpec(8, 16, None, chunk=32), GroupSpec(8, 16, 20), GroupSpec(8, 16)], share_prefixes=True)
+    assert not m.share_prefixes
+    assert [g.reach for g in m.groups] == [32, 20, None]
+
+
 def test_groups_have_pages_of_their_own():
     m = CacheManager([GroupSpec(8, 16, None), GroupSpec(3, 16, 16)], max_requests=4)
     m.add_request("a")
@@ -188,10 +238,10 @@ def test_state_slots():
 
 
 @pytest.mark.parametrize("seed", range(6))
-@pytest.mark.parametrize("window, share", [(None, True), (None, False), (24, False)])
-def test_random_orders_never_lose_or_double_a_page(seed, window, share):
+@pytest.mark.parametrize("window, share, chunk_size", [(None, True, None), (None, False, None), (24, False, None), (None, False, 40)])
+def test_random_orders_never_lose_or_double_a_page(seed, window, share, chunk_size):
     rng = random.Random(seed)
-    m = mgr(pages=12, share=share, window=window, max_requests=6)
+    m = mgr(pages=12, share=share, window=window, max_requests=6) if chunk_size is None else chunked(12, chunk_size, max_requests=6)
     live, next_id = {}, 0
     shared = [rng.randrange(50) for _ in range(40)]
     for _ in range(400):
@@ -217,7 +267,7 @@ def test_random_orders_never_lose_or_double_a_page(seed, window, share):
                 m.fork(parent, next_id)
                 live[next_id] = list(live[parent])
                 next_id += 1
-            elif op < 0.85 and live and window is None:
+            elif op < 0.85 and live and window is None and chunk_size is None:
                 rid = rng.choice(list(live))
                 m.truncate(rid, rng.randrange(0, m.length(rid) + 1))
                 live[rid] = []

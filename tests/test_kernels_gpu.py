@@ -397,6 +397,8 @@ MMA_CASES = [  # nh, nkv, hd, page_size, window, lens
     (32, 2, 64, 16, None, [300]),                # sixteen query heads per kv head
     (5, 5, 128, 64, 37, [300, 48, 17]),
     (2, 1, 128, 16, None, [129, 1000]),
+    (6, 2, 96, 16, None, [700, 65, 31, 32, 33]),
+    (3, 3, 96, 32, 40, [300, 39, 40, 41, 7]),
 ]
 
 
