@@ -1216,6 +1216,9 @@ def latent_attention_mma(q: torch.Tensor, out: torch.Tensor, cache: torch.Tensor
           block_tables.shape[1], _ptr(seq_first_row), _ptr(seq_start_pos), _ptr(positions), _ptr(sink), n, S,
           int(max_rows_per_seq), heads, c, r, page_size, num_pages, float(scale), int(window) if window else 0,
           1 if decode else 0, int(splits), _ptr(status), _stream())
+    if decode and splits > 1:
+        global launch_count
+        launch_count += 1
 
 
 class NormedPair:

@@ -65,8 +65,8 @@ CONFIGS = {
     ], scale=2.5, logit_cap=6.0, eps=1e-5),
     # sizes the tensor-core kernels are built for (head size 64: the flash kernel; 96, 80, 128: the tiles; latents of 64 and 128)
     "even": lambda: config(320, 128, [
-        layer(attention(8, 2, 64, 64, 64, chunk=48, cap=5.0, scaling=bands(8.0, 128, 1.0, 4.0)), 256),
-        layer(latent(4, 32, 16, 32, 64, 96, window=40, scaling=ramp(4.0, 128, 16.0, 1.0)), 192),
+        layer(attention(8, 2, 64, 64, 64, chunk=48, cap=5.0, scaling=bands(6.0, 128, 1.0, 4.0)), 288),
+        layer(latent(6, 48, 16, 48, 64, 112, window=36, scaling=ramp(3.0, 128, 16.0, 1.0)), 192),
         layer(attention(6, 3, 96, 96, 32, chunk=100, cap=4.0, scaling=bands(2.0, 300, 0.5, 6.0)), 64),
         layer(latent(20, 16, 32, 64, 128, 48, window=130), 128),
         layer(attention(2, 2, 128, 64, 128, cap=9.0), 96),

@@ -128,7 +128,7 @@ def test_what_the_parts_refuse():
 
 
 @pytest.mark.parametrize("dims, base, sc", [
-    (48, 10000.0, lu.bands(8.0, 1000, 1.0, 4.0)), (12, 500.0, lu.bands(3.0, 40, 1.0, 3.0)), (64, 1e6, lu.bands(32.0, 8192, 1.0, 4.0)),
+    (40, 10000.0, lu.bands(6.0, 1000, 1.0, 5.0)), (12, 500.0, lu.bands(3.0, 40, 1.0, 3.0)), (64, 1e6, lu.bands(32.0, 8192, 1.0, 4.0)),
     (2, 10.0, lu.bands(2.0, 10, 0.5, 2.0)), (20, 10000.0, lu.bands(4.0, 100000000, 1.0, 4.0)), (20, 10000.0, lu.bands(4.0, 1, 1.0, 4.0)), (6, 10.0, None)])
 def test_frequencies_in_bands(dims, base, sc):
     rescale = RopeBandRescaleSpec(sc["factor"], sc["original"], sc["low"], sc["high"]) if sc else None
@@ -151,7 +151,7 @@ def test_the_three_bands_of_frequencies():
 
 
 @pytest.mark.parametrize("dims, base, sc", [
-    (16, 10000.0, lu.ramp(4.0, 2000, 32.0, 1.0)), (10, 300.0, lu.ramp(2.0, 200, 16.0, 2.0)), (64, 1e6, lu.ramp(40.0, 4096, 32.0, 1.0)),
+    (24, 10000.0, lu.ramp(5.0, 2000, 32.0, 1.0)), (10, 300.0, lu.ramp(2.0, 200, 16.0, 2.0)), (64, 1e6, lu.ramp(40.0, 4096, 32.0, 1.0)),
     (2, 10.0, lu.ramp(3.0, 8, 4.0, 1.0)), (8, 10000.0, lu.ramp(3.0, 4, 32.0, 1.0)), (8, 50.0, None)])
 def test_frequencies_along_a_ramp(dims, base, sc):
     rescale = RopeRescaleSpec(sc["factor"], sc["original"], sc["fast"], sc["slow"]) if sc else None

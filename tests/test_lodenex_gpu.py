@@ -16,10 +16,10 @@ from test_felovik_gpu import _cuts, _f32, _gather, _i32, _Pages, _rounded, _scat
 pytestmark = pytest.mark.gpu
 DEV = "cuda:0"
 
-# bfloat16 against float64 on sharp models: every row within a third of the logits' spread, and close on average. Faults in which
+# bfloat16 against float64 on sharp models (the largest seen: 0.10 and 0.006 of the spread). Faults in which
 # key or token a bfloat16 kernel reads are caught by the crafted tests below and by the float32 runs of the same code, which are
 # held to 1e-4.
-BF16_REL_MAX, BF16_REL_MEAN = 0.35, 0.03
+BF16_REL_MAX, BF16_REL_MEAN = 0.2, 0.012
 
 
 def assert_logits_close(got, want, dtype, what=""):
